@@ -4,7 +4,8 @@ What a layer's mixer keeps between steps is its own business; it tells the
 cache by returning a request from ``cache_request()``:
 
 * :class:`KVRequest` — keys and values that grow with the sequence (all of
-  them, or a sliding window of the last ``window``);
+  them, or a sliding window of the last ``window``), with ``pool`` also one entry (the mean)
+  for every complete block of ``pool`` tokens, kept as long as the sequence lives;
 * :class:`StateRequest` — a tensor of fixed size per sequence;
 * ``None`` — nothing.
 
@@ -22,7 +23,7 @@ before anything is launched, in the same spirit.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Dict, List, Optional, Sequence, Tuple
 
 import numpy as np
@@ -38,12 +39,30 @@ class KVRequest:
     window: int = 0          # 0: every key is kept; W > 0: the last W keys
     shared_values: bool = False   # one tensor serves as keys and values (a cached latent)
     value_dim: int = 0       # size of a value head when it is not head_dim
+    pool: int = 0            # P > 0: beside the keys, one entry per complete block of P tokens
+
+    @property
+    def keep(self) -> int:
+        """Keys before the next position that must stay (0: all): the window's, and those of the
+        block that is not complete yet."""
+        return max(self.window, self.pool) if self.window > 0 else 0
 
 
 @dataclass(frozen=True)
 class StateRequest:
     shape: Tuple[int, ...]
     dtype: torch.dtype = torch.float32
+
+
+@dataclass
+class PoolView:
+    """A layer's entries per complete block of ``pool`` tokens; entry b of a sequence lies where
+    position b would lie in an ordinary group."""
+
+    k: torch.Tensor              # [n_blocks, num_kv_heads, block_tokens, head_dim]
+    v: torch.Tensor
+    table: torch.Tensor          # [max_slots, blocks_per_sequence] int32, device
+    pool: int
 
 
 @dataclass
@@ -55,6 +74,7 @@ class KVView:
     table: torch.Tensor          # [max_slots, blocks_per_sequence] int32, device
     block_tokens: int
     window: int
+    pool: Optional[PoolView] = None
 
 
 def _id_order(cid):
@@ -65,8 +85,10 @@ def _id_order(cid):
 
 class _KVGroup:
     def __init__(self, request: KVRequest, cache_ids: List[int], n_blocks: int,
-                 block_tokens: int, max_slots: int, blocks_per_seq: int, dtype, device):
+                 block_tokens: int, max_slots: int, blocks_per_seq: int, dtype, device,
+                 tokens_per_entry: int = 1):
         self.request = request
+        self.tokens_per_entry = tokens_per_entry     # > 1: an entry per complete run of tokens
         self.cache_ids = list(cache_ids)
         self.block_tokens = block_tokens
         self.blocks_per_seq = blocks_per_seq
@@ -85,7 +107,7 @@ class _KVGroup:
         self.dirty: set = set()
 
     def blocks_needed(self, slot: int, new_len: int) -> int:
-        want = -(-new_len // self.block_tokens)
+        want = -(-(new_len // self.tokens_per_entry) // self.block_tokens)
         return max(0, want - int(self.n_blocks_of[slot]))
 
     def grow(self, slot: int, new_len: int) -> None:
@@ -108,7 +130,7 @@ class _KVGroup:
             self.dirty.add(slot)
 
     def release_outside_window(self, slot: int, length: int) -> None:
-        w = self.request.window
+        w = self.request.keep
         if w <= 0:
             return
         first_needed_key = max(0, length - w + 1)       # the next query sits at `length`
@@ -170,6 +192,7 @@ class SequenceCache:
 
         self._kv_groups: List[_KVGroup] = []
         self._kv_of: Dict[int, Tuple[_KVGroup, int]] = {}
+        self._pool_of: Dict[int, Tuple[_KVGroup, int]] = {}
         self._state: Dict[int, torch.Tensor] = {}
         by_request: Dict[KVRequest, List[int]] = {}
         for cid in sorted(requests, key=_id_order):
@@ -195,6 +218,19 @@ class SequenceCache:
             self._kv_groups.append(g)
             for i, cid in enumerate(cids):
                 self._kv_of[cid] = (g, i)
+            if req.pool > 0:
+                # Enough for any mixture of live sequences: each may leave its last block of
+                # entries partly empty, and only one with ``pool`` tokens has an entry at all.
+                P = req.pool
+                n_pool = -(-self.max_tokens // (P * block_tokens)) \
+                    + min(self.max_slots, self.max_tokens // P)
+                pg = _KVGroup(replace(req, window=0, pool=0), cids,
+                              max(1, min(self.n_blocks, n_pool)), block_tokens, self.max_slots,
+                              max(1, -(-(self.max_len // P) // block_tokens)), dtype, self.device,
+                              tokens_per_entry=P)
+                self._kv_groups.append(pg)
+                for i, cid in enumerate(cids):
+                    self._pool_of[cid] = (pg, i)
 
     # -- slots ---------------------------------------------------------------
     def alloc_slot(self) -> int:
@@ -234,7 +270,7 @@ class SequenceCache:
             need = sum(g.blocks_needed(s, int(self.lengths[s]) + n) for s, n in entries)
             if need > g.pool.free_count:
                 raise CacheFull(f"the step needs {need} more cache blocks of {self.block_tokens} "
-                                f"tokens, only {g.pool.free_count} of {g.pool.n_blocks} are free")
+                                f"{'tokens' if g.tokens_per_entry == 1 else 'entries'}, only {g.pool.free_count} of {g.pool.n_blocks} are free")
         for g in self._kv_groups:
             for s, n in entries:
                 g.grow(s, int(self.lengths[s]) + n)
@@ -289,7 +325,11 @@ class SequenceCache:
     # -- views -----------------------------------------------------------------
     def kv_view(self, cache_id: int) -> KVView:
         g, i = self._kv_of[cache_id]
-        return KVView(g.k[i], g.v[i], g.table, g.block_tokens, g.request.window)
+        pool = None
+        if cache_id in self._pool_of:
+            pg, pi = self._pool_of[cache_id]
+            pool = PoolView(pg.k[pi], pg.v[pi], pg.table, pg.tokens_per_entry)
+        return KVView(g.k[i], g.v[i], g.table, g.block_tokens, g.request.window, pool)
 
     def state_view(self, cache_id: int) -> torch.Tensor:
         return self._state[cache_id]
@@ -315,7 +355,8 @@ class SequenceCache:
             "state_bytes": state_bytes,
             "groups": [{"num_kv_heads": g.request.num_kv_heads, "head_dim": g.request.head_dim,
                         "value_dim": g.request.value_dim or g.request.head_dim,
-                        "window": g.request.window, "layers": len(g.cache_ids)}
+                        "window": g.request.window, "layers": len(g.cache_ids),
+                        "tokens_per_entry": g.tokens_per_entry}
                        for g in self._kv_groups],
         }
 

@@ -7,6 +7,7 @@ from .rigozen import RigozenConfig, build_rigozen_spec, rigozen_config_from_dict
 from .losorax import LosoraxConfig, build_losorax_spec, losorax_config_from_dict
 from .virorax import ViroraxConfig, build_virorax_spec, virorax_config_from_dict
 from .mipurax import MipuraxConfig, build_mipurax_spec, mipurax_config_from_dict
+from .gibipel import GibipelConfig, build_gibipel_spec, gibipel_config_from_dict
 from .presets import PRESETS, preset
 
 __all__ = [
@@ -18,4 +19,5 @@ __all__ = [
     "LosoraxConfig", "build_losorax_spec", "losorax_config_from_dict",
     "ViroraxConfig", "build_virorax_spec", "virorax_config_from_dict",
     "MipuraxConfig", "build_mipurax_spec", "mipurax_config_from_dict",
+    "GibipelConfig", "build_gibipel_spec", "gibipel_config_from_dict",
 ]

@@ -15,7 +15,7 @@ extern "C" {
 // bit 1 of *fault and writes zeros.
 int cretif_embed_rows(const void* table, int table_dt, const int* ids, float* out, int T, int H,
                       int V, unsigned int* fault, const void* pos_table, const int* tok_pos, int P,
-                      void* stream);
+                      float scale, void* stream);
 
 // v = h[src] (+ delta[src]); if write_h, h[src] = v; out[r] = v * weight * rsqrt(mean(v^2)+eps).
 // src = rows ? rows[r] : r.  delta may be null.  rows and write_h exclude each other.
@@ -142,10 +142,12 @@ int cretif_rmsnorm_rows(float* x, int ld, const float* w, int R, int H, float ep
 // of its two largest logistic scores, only experts of the `keep` best groups can be chosen.
 // renorm: the chosen scores are divided by (their sum + sum_eps).
 int cretif_moe_route(const void* x, int x_dt, int ldx, const float* router_w, int E, int H,
-                     int top, int renorm, int groups, int keep, float sum_eps, int* ids,
-                     float* wts, int T, void* stream);
+                     int top, int renorm, int groups, int keep, float sum_eps, int softmax,
+                     int group_best, const float* correction, int* ids, float* wts, int T,
+                     void* stream);
 int cretif_moe_topk(const float* logits, int ld, int E, int top, int renorm, int groups, int keep,
-                    float sum_eps, int* ids, float* wts, int T, void* stream);
+                    float sum_eps, int softmax, int group_best, const float* correction, int* ids,
+                    float* wts, int T, void* stream);
 int cretif_moe_group(const int* ids, int P, int E, int* offsets, int* place, int* order,
                      int* tile_expert, int* tile_row0, int max_tiles, void* stream);
 int cretif_moe_gemm(const void* A, int a_dt, int lda, const void* W, int w_dt, void* C, int ldc,
@@ -154,14 +156,15 @@ int cretif_moe_gemm(const void* A, int a_dt, int lda, const void* W, int w_dt, v
                     const int* tile_row0, int max_tiles, int use_mma, void* stream);
 int cretif_moe_gemv(const void* A, int a_dt, int lda, const void* W, int w_dt, void* C, int ldc,
                     int N, int K, int top, int mode, int scale_at, const int* ids,
-                    const float* wts, int P, void* stream);
+                    const float* wts, int P, int experts, void* stream);
 int cretif_moe_group_padded(const int* ids, int P, int E, int tile, int* place, int* tile_expert,
                             int max_tiles, int* used, void* stream);
 int cretif_moe_gather_rows(const void* x, int ldx, void* xs, int lds, const int* place,
                            const float* wts, int top, int K, int P, void* stream);
 // place may be null: the rows are in the pairs' own order; wts may be null: no weights.
 int cretif_moe_combine(const float* rows, int ld, const int* place, int top, const float* wts,
-                       float* y, int T, int H, void* stream);
+                       float* y, int T, int H, const int* ids, int experts, const float* id_wts,
+                       const void* x, int x_dt, int ldx, void* stream);
 
 // After a decode step: ids <- sampled (if given), positions and lengths + 1.
 int cretif_advance_decode(int* tok_ids, int* tok_pos, int* seq_start, const int* sampled, int B,
@@ -251,6 +254,24 @@ int cretif_attn_simt(const void* q, int ldq, void* out, int ldo, int dt, const v
                      const int* tok_seq, const int* seq_slot, int nh, int nkv, int hd, float scale,
                      int window, int bt, int T, const float* sink, int vd, const float* bias,
                      const int* bias_edges, int bias_rows, const float* slope, void* stream);
+// The same with pooled entries: pool_k, pool_v [blocks, nkv, bt, hd or vd] and pool_table
+// [slots, pool_stride] hold one entry per complete block of `pool` tokens; a query at position p
+// sees, beside its window, the entries whose last token is at or before p - window, in the same
+// softmax.  pool_table null: none.  Here and below they need a sliding window.
+int cretif_attn_simt_pooled(const void* q, int ldq, void* out, int ldo, int dt, const void* kc,
+                            const void* vc, const int* table, int table_stride, const int* tok_pos,
+                            const int* tok_seq, const int* seq_slot, int nh, int nkv, int hd,
+                            float scale, int window, int bt, int T, const float* sink, int vd,
+                            const float* bias, const int* bias_edges, int bias_rows,
+                            const float* slope, const void* pool_k, const void* pool_v,
+                            const int* pool_table, int pool_stride, int pool, void* stream);
+// The entries themselves (head_ops.cu): for every sequence, those whose block is completed by this
+// step's tokens -- the means (32-bit sums in the order of the positions) of the block's rows as the
+// cache holds them.
+int cretif_pool_kv(const void* kc, const void* vc, int dt, const int* table, int table_stride,
+                   void* pool_k, void* pool_v, const int* pool_table, int pool_stride, int pool,
+                   const int* cu_seqlens, const int* seq_start, const int* seq_slot, int nkv, int hd,
+                   int vd, int bt, int B, int max_new, unsigned int* fault, void* stream);
 
 // Decode attention (one query token per sequence), bfloat16, keys split into n_splits <= 64
 // ranges per (sequence, kv head); part_o/part_ml are float32 scratch of the sizes that
@@ -297,6 +318,15 @@ int cretif_attn_decode_mma_bias(const void* q, int ldq, void* out, int ldo, cons
                                 const float* bias_near, const float* bias_far, int n_far,
                                 int head_groups, const float* bias_slope, unsigned int* fault,
                                 void* stream);
+// ... and with pooled entries (see cretif_attn_simt_pooled; pool_blocks blocks of them).
+int cretif_attn_decode_mma_pooled(
+    const void* q, int ldq, void* out, int ldo, const void* kc, const void* vc, long long n_blocks,
+    const int* table, int table_stride, const int* tok_pos, const int* tok_seq, const int* seq_slot,
+    int nh, int nkv, int hd, float scale, int window, int bt, int B, int n_splits, float* part_o,
+    float* part_ml, int* counters, const float* sink, const float* bias_near, const float* bias_far,
+    int n_far, int head_groups, const float* bias_slope, const void* pool_k, const void* pool_v,
+    long long pool_blocks, const int* pool_table, int pool_stride, int pool, unsigned int* fault,
+    void* stream);
 
 // Fused decode projections (see decode_fused.cu).  H is the float32 residual stream; when it
 // is given, x = bf16(rmsnorm(H[rows])) is computed in the kernel, else X (bfloat16) is read.
@@ -361,6 +391,15 @@ int cretif_attn_prefill_tc_bias(const void* qkv, int ldq, int T, void* out, int 
                                 const float* sink, const float* bias_near, const float* bias_far,
                                 int n_far, const float* bias_slope, unsigned int* fault,
                                 void* stream);
+// ... and with pooled entries (see cretif_attn_simt_pooled), without a bias or a slope.
+int cretif_attn_prefill_tc_pooled(
+    const void* qkv, int ldq, int T, void* out, int ldo, const void* kc, const void* vc,
+    long long n_blocks, const int* table, int table_stride, const int* cu_seqlens,
+    const int* seq_start, const int* seq_slot, int nh, int nkv, int hd, float scale, int window,
+    int bt, int B, int max_new, const float* sink, const float* bias_near, const float* bias_far,
+    int n_far, const float* bias_slope, const void* pool_k, const void* pool_v,
+    long long pool_blocks, const int* pool_table, int pool_stride, int pool, unsigned int* fault,
+    void* stream);
 
 // Per-head work of an attention whose projections are normed head by head (head_ops.cu).
 // proj rows [q (nh hd) | k (nkv hd) | v (nkv vd) | ...] (float32 or bfloat16): + bias (null for
@@ -383,9 +422,33 @@ int cretif_activation(const void* in, int ldi, int in_dt, void* out, int ldo, in
                       int width, int kind, void* stream);
 // z <- cap * tanh(z / cap) in place.
 int cretif_softcap(float* z, long long total, float cap, void* stream);
+// z <- factor * z, in place.
+int cretif_scale(float* z, long long total, float factor, void* stream);
 // h += alpha * y over `total` elements (y float32 or bfloat16).
 int cretif_axpy_rows(float* h, const void* y, int y_dt, float alpha, long long total,
                      void* stream);
+
+// The same with the norms over the whole query and key projections (wq [nh hd], wk [nkv hd]), float32
+// rows, v times v_scale; pool_table non-null (one token a sequence): the pooled entry of a block that
+// a token completes is written too (see cretif_pool_kv).
+int cretif_projnorm_rope_kv_append(
+    const float* proj, int ldp, const float* bias, const float* wq, const float* wk, float eps,
+    const float* cos_t, const float* sin_t, int pairing, int rot_dim, const int* tok_pos,
+    const int* tok_seq, const int* seq_slot, int nh, int nkv, int hd, int vd, float v_scale,
+    void* q_out, int ldq, int dt, const int* table, int table_stride, void* kc, void* vc, int bt,
+    int write_cache, void* pool_k, void* pool_v, const int* pool_table, int pool_stride, int pool,
+    int T, unsigned int* fault, void* stream);
+
+// Matrix memory with exponential gates (matrix_memory.cu): proj rows (float32) [q (H d) | k (H d) |
+// v (H e) | gate (H e) | z_i (H) | z_f (H) | ...] -> out [T, H e], the normed and gated read-outs; a
+// slot's state is [S (H d e) | n (H d) | m (H)].  Scratch: o_raw [T, H e], den and ref [T, H] float32,
+// gates [3, H, T] float64.  form: 0 chooses, 1 token by token, 2 chunks of 64 tokens.
+int cretif_matrix_memory(const float* proj, int ldp, const float* bias_i, const float* bias_f,
+                         float cap, float q_scale, float* state, long long state_stride,
+                         const int* cu_seqlens, const int* seq_slot, const int* tok_seq, int B, int H,
+                         int d, int e, const float* norm_w, float eps, float* o_raw, float* den,
+                         float* ref, double* gates, void* out, int out_dt, int ldo, int write_state,
+                         int T, int form, void* stream);
 
 // Retention (retention.cu).  proj rows (float32): [q (H d) | k (H d) | ...]; prep rows: the
 // rotated q and the rotated k times k_scale.  state points at the first sequence slot's

@@ -23,7 +23,8 @@ static int launch_dm(const CUtensorMap& mk, const CUtensorMap& mv, const void* q
                      const int* seq_slot, int nh, int nkv, float scale_log2, int window,
                      float* part_o, float* part_ml, void* out, int ldo, int* counters,
                      unsigned int* fault, dim3 grid, cudaStream_t st, const float* sink,
-                     DistanceBias bias) {
+                     DistanceBias bias, const CUtensorMap& mpk, const CUtensorMap& mpv,
+                     const PooledKeys& pooled) {
   // Few CTAs (at most two per SM) walk many tiles each: a deeper ring keeps more of the cache
   // in flight per CTA, as long as two CTAs still fit an SM.
   static int sm_count = 0;
@@ -69,7 +70,7 @@ static int launch_dm(const CUtensorMap& mk, const CUtensorMap& mv, const void* q
   cudaError_t e = cudaLaunchKernelEx(
       &cfg, attn_decode_mma_kernel<HD16, CLUSTER>, mk, mv, (const __nv_bfloat16*)q, ldq, table,
       table_stride, tok_pos, tok_seq, seq_slot, nh, nkv, scale_log2, window, part_o, part_ml,
-      (__nv_bfloat16*)out, ldo, counters, fault, g_dm_stamps, n_stages, sink, bias);
+      (__nv_bfloat16*)out, ldo, counters, fault, g_dm_stamps, n_stages, sink, bias, mpk, mpv, pooled);
   return e == cudaSuccess ? launch_status() : (int)e;
 }
 
@@ -121,7 +122,26 @@ extern "C" int cretif_attn_decode_mma_bias(const void* q, int ldq, void* out, in
                                            const float* bias_near, const float* bias_far,
                                            int n_far, int head_groups, const float* bias_slope,
                                            unsigned int* fault, void* stream) {
+  return cretif_attn_decode_mma_pooled(
+      q, ldq, out, ldo, kc, vc, n_blocks, table, table_stride, tok_pos, tok_seq, seq_slot, nh, nkv,
+      hd, scale, window, bt, B, n_splits, part_o, part_ml, counters, sink, bias_near, bias_far,
+      n_far, head_groups, bias_slope, nullptr, nullptr, 0, nullptr, 0, 0, fault, stream);
+}
+
+// pool_k, pool_v (blocks like kc and vc, pool_blocks of them), pool_table [slots, pool_stride]: the
+// entries per complete block of `pool` tokens (pool_table null: none; they need a sliding window).
+extern "C" int cretif_attn_decode_mma_pooled(
+    const void* q, int ldq, void* out, int ldo, const void* kc, const void* vc, long long n_blocks,
+    const int* table, int table_stride, const int* tok_pos, const int* tok_seq, const int* seq_slot,
+    int nh, int nkv, int hd, float scale, int window, int bt, int B, int n_splits, float* part_o,
+    float* part_ml, int* counters, const float* sink, const float* bias_near, const float* bias_far,
+    int n_far, int head_groups, const float* bias_slope, const void* pool_k, const void* pool_v,
+    long long pool_blocks, const int* pool_table, int pool_stride, int pool, unsigned int* fault,
+    void* stream) {
   if (B <= 0) return kOk;
+  if (pool_table && (!pool_k || !pool_v || pool <= 0 || window <= 0 || pool_blocks <= 0))
+    return kBadArgument;
+  const PooledKeys pooled{pool_k, pool_v, pool_table, pool_stride, pool > 0 ? pool : 1, pool_blocks};
   if ((bias_near != nullptr) != (bias_far != nullptr) || (bias_near && n_far < 1) ||
       head_groups < 1 || B % head_groups || (bias_near && bias_slope))
     return kBadArgument;
@@ -130,12 +150,18 @@ extern "C" int cretif_attn_decode_mma_bias(const void* q, int ldq, void* out, in
       bt != kDmTile || n_splits <= 0 || n_splits > kDmTile || nkv > 65535 || B > 65535 ||
       ldq % 2)
     return kBadArgument;
-  if (((uintptr_t)kc | (uintptr_t)vc) & 15 || ((uintptr_t)q & 3)) return kMisaligned;
-  const long long cache_rows = n_blocks * nkv * kDmTile;
-  if (cache_rows > 0x7fffffffLL) return kBadArgument;
+  if (((uintptr_t)kc | (uintptr_t)vc | (uintptr_t)pool_k | (uintptr_t)pool_v) & 15 ||
+      ((uintptr_t)q & 3))
+    return kMisaligned;
+  const long long cache_rows = n_blocks * nkv * kDmTile, pool_rows = pool_blocks * nkv * kDmTile;
+  if (cache_rows > 0x7fffffffLL || pool_rows > 0x7fffffffLL) return kBadArgument;
   CUtensorMap mk, mv;
   if (make_tile_map_bf16(&mk, kc, (int)cache_rows, hd, hd, kDmTile)) return kBadArgument;
   if (make_tile_map_bf16(&mv, vc, (int)cache_rows, hd, hd, kDmTile)) return kBadArgument;
+  CUtensorMap mpk = mk, mpv = mv;               // (not read without entries)
+  if (pool_table && (make_tile_map_bf16(&mpk, pool_k, (int)pool_rows, hd, hd, kDmTile) ||
+                     make_tile_map_bf16(&mpv, pool_v, (int)pool_rows, hd, hd, kDmTile)))
+    return kBadArgument;
   const float scale_log2 = scale * 1.4426950408889634f;
   dim3 grid(n_splits, nkv, B);
   cudaStream_t st = (cudaStream_t)stream;
@@ -147,10 +173,12 @@ extern "C" int cretif_attn_decode_mma_bias(const void* q, int ldq, void* out, in
     return cluster                                                                            \
                ? launch_dm<N, true>(mk, mv, q, ldq, table, table_stride, tok_pos, tok_seq,    \
                                     seq_slot, nh, nkv, scale_log2, window, part_o, part_ml,   \
-                                    out, ldo, counters, fault, grid, st, sink, bias)          \
+                                    out, ldo, counters, fault, grid, st, sink, bias, mpk,     \
+                                    mpv, pooled)                                              \
                : launch_dm<N, false>(mk, mv, q, ldq, table, table_stride, tok_pos, tok_seq,   \
                                      seq_slot, nh, nkv, scale_log2, window, part_o, part_ml,  \
-                                     out, ldo, counters, fault, grid, st, sink, bias)
+                                     out, ldo, counters, fault, grid, st, sink, bias, mpk,    \
+                                     mpv, pooled)
   switch (hd / 16) {
     CRETIF_DM(1); CRETIF_DM(2); CRETIF_DM(3); CRETIF_DM(4);
     CRETIF_DM(5); CRETIF_DM(6); CRETIF_DM(7); CRETIF_DM(8);

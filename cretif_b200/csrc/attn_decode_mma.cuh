@@ -16,6 +16,9 @@
 // scratch and are merged by the CTA that finishes last, as in attn_decode.cu (same scratch,
 // same counters).
 //
+// With pooled entries (PooledKeys, common.cuh) the tiles of the entries that the query sees come
+// before the tiles of its window in one list, which the ranges share out.
+//
 // The reference walks positions serially with one block per head (src/attention.cu:410-494).
 #pragma once
 
@@ -115,7 +118,9 @@ __device__ __forceinline__ void attn_decode_mma_item(
     int ldo, int* __restrict__ counters, unsigned int* __restrict__ fault, int split,
     int n_splits, int kvh, int b, uint32_t& it_base, unsigned long long* stamps = nullptr,
     int n_stages = kDmStages, const float* sink = nullptr,
-    DistanceBias bias = DistanceBias{nullptr, nullptr, 0, 1, nullptr}) {
+    DistanceBias bias = DistanceBias{nullptr, nullptr, 0, 1, nullptr},
+    const CUtensorMap* map_pk = nullptr, const CUtensorMap* map_pv = nullptr,
+    PooledKeys pooled = PooledKeys{nullptr, nullptr, nullptr, 0, 1, 0}) {
   if (bias.head_groups > 1) {           // this item's heads start at head0 of the model's
     const int head0 = (b % bias.head_groups) * nh;
     if (sink) sink += head0;
@@ -171,10 +176,15 @@ __device__ __forceinline__ void attn_decode_mma_item(
   const int slot = seq_slot[tok_seq[b]];
   const int* tab = table + (size_t)slot * table_stride;
   const int first_key = first_visible_key(pos, window);
-  const int first_tile = first_key / kDmTile, n_tiles = pos / kDmTile + 1;
+  const int first_tile = first_key / kDmTile;
+  // tiles 0 .. pool_tiles - 1 of the item's list hold pooled entries, the rest the window's keys
+  const int n_pooled = pooled.table ? visible_pooled(pos, window, pooled.pool) : 0;
+  const int pool_tiles = (n_pooled + kDmTile - 1) / kDmTile;
+  const int* ptab = pooled.table + (size_t)slot * pooled.table_stride;
+  const int shift = first_tile - pool_tiles;             // list index + shift = the window's tile
   // the tiles are dealt out evenly: the first (tiles % ranges) ranges take one more
-  const int span = n_tiles - first_tile, per = span / n_splits, extra = span - per * n_splits;
-  const int t_begin = first_tile + split * per + min(split, extra);
+  const int span = pos / kDmTile + 1 - shift, per = span / n_splits, extra = span - per * n_splits;
+  const int t_begin = split * per + min(split, extra);
   const int my_tiles = per + (split < extra ? 1 : 0);
   if (stamping && my_tiles >= 0) stamp(threadIdx.x >> 5, 1);
 
@@ -198,7 +208,8 @@ __device__ __forceinline__ void attn_decode_mma_item(
     // divided, per tile)
     int st = (int)(it_base % (uint32_t)n_stages), turn = (int)(it_base / (uint32_t)n_stages);
     for (int i0 = 0; i0 < my_tiles; i0 += 32) {
-      const int mine = i0 + lane < my_tiles ? tab[t_begin + i0 + lane] : 0;
+      const int at = t_begin + i0 + lane;
+      const int mine = i0 + lane < my_tiles ? (at < pool_tiles ? ptab[at] : tab[at + shift]) : 0;
       const int n = min(32, my_tiles - i0);
       if (stamping && mine >= -1) stamp(threadIdx.x >> 5, 2);
       bool go = true;
@@ -206,7 +217,7 @@ __device__ __forceinline__ void attn_decode_mma_item(
         const int i = i0 + j;
         const int blk = __shfl_sync(0xffffffffu, mine, j);
         const int s = st;
-        if (!waited && (i >= n_stages || t_begin + i == n_tiles - 1)) {
+        if (!waited && (i >= n_stages || t_begin + i == span - 1)) {
           asm volatile("griddepcontrol.wait;" ::: "memory");
           waited = true;
         }
@@ -216,11 +227,14 @@ __device__ __forceinline__ void attn_decode_mma_item(
           } else {
             if (blk < 0) atomicOr(fault, kFaultBlockTable);
             const int row = (max(blk, 0) * nkv + kvh) * kDmTile;
+            const bool entries = t_begin + i < pool_tiles;
+            const CUtensorMap* mk = entries ? map_pk : map_k;
+            const CUtensorMap* mv = entries ? map_pv : map_v;
             tc::mbar_expect_tx(&full[s], 2u * kTileBytes);
 #pragma unroll
             for (int sub = 0; sub < kSub; ++sub) {
-              tc::tma_load_2d(ktiles + s * kTileBytes + sub * kDmTile * 128, map_k, 64 * sub, row, &full[s]);
-              tc::tma_load_2d(vtiles + s * kTileBytes + sub * kDmTile * 128, map_v, 64 * sub, row, &full[s]);
+              tc::tma_load_2d(ktiles + s * kTileBytes + sub * kDmTile * 128, mk, 64 * sub, row, &full[s]);
+              tc::tma_load_2d(vtiles + s * kTileBytes + sub * kDmTile * 128, mv, 64 * sub, row, &full[s]);
             }
           }
         }
@@ -280,20 +294,22 @@ __device__ __forceinline__ void attn_decode_mma_item(
         }
       }
       // ---- online softmax of row r over this thread's 4 keys (and the quad's 16)
-      const int key0 = (t_begin + i) * kDmTile + warp * 16;
+      const bool entries = t_begin + i < pool_tiles;
+      const int key0 = (t_begin + i + (entries ? 0 : shift)) * kDmTile + warp * 16;
+      const int key_lo = entries ? 0 : first_key, key_hi = entries ? n_pooled - 1 : pos;
       float t4[4];
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int key = key0 + n * 8 + 2 * c + e;
-          const bool valid = key <= pos && key >= first_key;
+          const bool valid = key <= key_hi && key >= key_lo;
           float sv = sacc[n][e] * scale_log2;
-          if (bias.near_ && valid && r < g) {
+          if (bias.near_ && valid && r < g && !entries) {
             const int head = kvh * g + r, dist = pos - key;
             sv += dist >= bias.n_far ? __ldg(bias.far_ + head)
                                      : __ldg(bias.near_ + (size_t)head * bias.n_far + dist);
-          } else if (bias.slope_ && valid && r < g) {
+          } else if (bias.slope_ && valid && r < g && !entries) {
             sv -= __ldg(bias.slope_ + kvh * g + r) * (float)(pos - key);
           }
           t4[n * 2 + e] = valid ? sv : -INFINITY;
@@ -545,7 +561,9 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap map_k,
                        int window, float* __restrict__ part_o, float* __restrict__ part_ml,
                        __nv_bfloat16* __restrict__ out, int ldo, int* __restrict__ counters,
                        unsigned int* __restrict__ fault, unsigned long long* stamps,
-                       int n_stages, const float* __restrict__ sink, DistanceBias bias) {
+                       int n_stages, const float* __restrict__ sink, DistanceBias bias,
+                       const __grid_constant__ CUtensorMap map_pk,
+                       const __grid_constant__ CUtensorMap map_pv, PooledKeys pooled) {
   extern __shared__ unsigned char smem_raw[];
   if (kStamps && stamps && blockIdx.x + blockIdx.y + blockIdx.z == 0 && threadIdx.x == 0) {
     unsigned long long t;
@@ -562,7 +580,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap map_k,
                                       tok_seq, seq_slot, nh, nkv, scale_log2, window, part_o,
                                       part_ml, out, ldo, counters, fault, blockIdx.x, gridDim.x,
                                       blockIdx.y, blockIdx.z, it_base, stamps, n_stages, sink,
-                                      bias);
+                                      bias, &map_pk, &map_pv, pooled);
 }
 
 }  // namespace cretif

@@ -23,6 +23,9 @@
 // call (src/attention.cu:644-728); nothing of that exists here.
 //
 // Queries of the next sequence that fall into a tile's 128 rows are computed and dropped.
+//
+// POOLED: the entries per complete block of tokens (PooledKeys, common.cuh) that any of the tile's
+// queries sees are walked first, 128 a step like keys, each row masked to its own number of them.
 #include <cuda.h>
 #include <cuda_runtime.h>
 
@@ -87,7 +90,7 @@ __device__ __forceinline__ uint64_t smem_desc_mn_sw128(const void* tile, uint32_
   return d;
 }
 
-template <int HDMAX>
+template <int HDMAX, bool POOLED = false>
 __global__ void __launch_bounds__(kPfThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                        const __grid_constant__ CUtensorMap map_k,
@@ -98,7 +101,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                        int window, unsigned int* __restrict__ fault,
                        unsigned long long* stamps, const float* __restrict__ sink,
                        const float* __restrict__ bias_near, const float* __restrict__ bias_far,
-                       int n_far, const float* __restrict__ bias_slope) {
+                       int n_far, const float* __restrict__ bias_slope,
+                       const __grid_constant__ CUtensorMap map_pk,
+                       const __grid_constant__ CUtensorMap map_pv, const PooledKeys pooled) {
   // bias_near [nh, n_far], bias_far [nh] (both times log2 e, may be null): what is added to the
   // scaled score of the key n positions back, for n < n_far and for every n beyond.
   // bias_slope [nh] (times log2 e, may be null; not together with the table): n times it is
@@ -149,7 +154,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
   const int pos_first = start + q0, pos_last = start + q0 + rows_here - 1;
   const int key_lo = first_visible_key(pos_first, window);
   const int blk_lo = key_lo / kPfBlk, blk_hi = pos_last / kPfBlk;      // cache blocks, inclusive
-  const int n_tiles = (blk_hi - blk_lo + 2) / 2;                        // steps of two blocks
+  // the first pool_tiles steps walk blocks of pooled entries, the others the tokens' blocks
+  const int pool_blks =
+      POOLED ? (visible_pooled(pos_last, window, pooled.pool) + kPfBlk - 1) / kPfBlk : 0;
+  const int pool_tiles = POOLED ? (pool_blks + 1) / 2 : 0;
+  const int n_tiles = pool_tiles + (blk_hi - blk_lo + 2) / 2;           // steps of two blocks
   // Tensor memory: two score tiles (the product of step j + 1 runs under the softmax of
   // step j) and two tiles of P V.
   constexpr uint32_t kTmemCols = 512;
@@ -196,13 +205,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         for (int half = 0; half < 2; ++half) {
           // a step past the last block loads that block again: its keys are masked, and the
           // operand tile holds finite numbers instead of whatever was in shared memory
-          const int blk = tab[min(blk_lo + 2 * j + half, blk_hi)];
+          const bool entries = POOLED && j < pool_tiles;
+          const int blk = entries ? pooled.table[(size_t)slot * pooled.table_stride +
+                                                 min(2 * j + half, pool_blks - 1)]
+                                  : tab[min(blk_lo + 2 * (j - pool_tiles) + half, blk_hi)];
           if (blk < 0) atomicOr(fault, kFaultBlockTable);
           const int row = (max(blk, 0) * nkv + kvh) * kPfBlk;
+          const CUtensorMap* mk = entries ? &map_pk : &map_k;
+          const CUtensorMap* mv = entries ? &map_pv : &map_v;
           for (int sub = 0; sub < n_sub; ++sub) {
             const int off = (s * n_sub + sub) * kPfBK * 128 + half * kPfBlk * 128;
-            tc::tma_load_2d(smem + L.k + off, &map_k, 64 * sub, row, &kv_full[s]);
-            tc::tma_load_2d(smem + L.v + off, &map_v, 64 * sub, row, &kv_full[s]);
+            tc::tma_load_2d(smem + L.k + off, mk, 64 * sub, row, &kv_full[s]);
+            tc::tma_load_2d(smem + L.v + off, mv, 64 * sub, row, &kv_full[s]);
           }
         }
       }
@@ -267,6 +281,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
     // a step needs masks if it reaches past the first row's position or starts before the
     // last row's window
     const int lo_key_last = first_visible_key(start + q0 + kPfBQ - 1, window);
+    // entries that the row and the tile's first row see
+    const int n_mine = POOLED ? visible_pooled(q_pos, window, pooled.pool) : 0;
+    const int n_first = POOLED ? visible_pooled(pos_first, window, pooled.pool) : 0;
     const uint32_t lane_addr = tmem + ((uint32_t)(quad * 32) << 16);
     const int ocols = hd >> 1, obase = half * ocols;     // this thread's output columns
     float o[HDMAX / 2];
@@ -328,17 +345,19 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
       tc::tmem_load_32(lane_addr + s_col + 32, sb);
       tc::tmem_load_wait();
       if (warp == 2) stamp(j, 2);
-      const int key0 = (blk_lo + 2 * j) * kPfBlk + half * 64;
+      const bool entries = POOLED && j < pool_tiles;
+      const int key0 = (entries ? 2 * j : blk_lo + 2 * (j - pool_tiles)) * kPfBlk + half * 64;
       // Raw scores stay in their registers; only steps that touch the diagonal, the
       // sequence's end or a window's edge pay for masking (uniform for the whole CTA).
       float t[64];
-      const bool masked = key0 + 63 > pos_first || key0 < lo_key_last;
+      const bool masked = entries ? key0 + 63 >= n_first : key0 + 63 > pos_first || key0 < lo_key_last;
       if (masked) {
+        const int hi = entries ? n_mine - 1 : q_pos, lo = entries ? 0 : lo_key;
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
           const int key = key0 + c;
           const float sv = __uint_as_float(c < 32 ? sa[c] : sb[c - 32]);
-          t[c] = (key <= q_pos && key >= lo_key) ? sv : -INFINITY;
+          t[c] = (key <= hi && key >= lo) ? sv : -INFINITY;
         }
       } else {
 #pragma unroll
@@ -953,7 +972,28 @@ extern "C" int cretif_attn_prefill_tc_bias(const void* qkv, int ldq, int T, void
                                            const float* bias_far, int n_far,
                                            const float* bias_slope, unsigned int* fault,
                                            void* stream) {
+  return cretif_attn_prefill_tc_pooled(qkv, ldq, T, out, ldo, kc, vc, n_blocks, table, table_stride,
+                                       cu_seqlens, seq_start, seq_slot, nh, nkv, hd, scale, window,
+                                       bt, B, max_new, sink, bias_near, bias_far, n_far, bias_slope,
+                                       nullptr, nullptr, 0, nullptr, 0, 0, fault, stream);
+}
+
+// pool_k, pool_v (blocks like kc and vc, pool_blocks of them), pool_table [slots, pool_stride]: the
+// entries per complete block of `pool` tokens (pool_table null: none; they need a sliding window and
+// come without a bias or a slope).
+extern "C" int cretif_attn_prefill_tc_pooled(
+    const void* qkv, int ldq, int T, void* out, int ldo, const void* kc, const void* vc,
+    long long n_blocks, const int* table, int table_stride, const int* cu_seqlens,
+    const int* seq_start, const int* seq_slot, int nh, int nkv, int hd, float scale, int window,
+    int bt, int B, int max_new, const float* sink, const float* bias_near, const float* bias_far,
+    int n_far, const float* bias_slope, const void* pool_k, const void* pool_v,
+    long long pool_blocks, const int* pool_table, int pool_stride, int pool, unsigned int* fault,
+    void* stream) {
   if (B <= 0 || T <= 0) return kOk;
+  if (pool_table && (!pool_k || !pool_v || pool <= 0 || window <= 0 || pool_blocks <= 0 ||
+                     bias_near || bias_slope))
+    return kBadArgument;
+  const PooledKeys pooled{pool_k, pool_v, pool_table, pool_stride, pool > 0 ? pool : 1, pool_blocks};
   if ((bias_near != nullptr) != (bias_far != nullptr) || (bias_near && (n_far < 1 || n_far > 8192)) ||
       (bias_near && bias_slope))
     return kBadArgument;
@@ -961,13 +1001,19 @@ extern "C" int cretif_attn_prefill_tc_bias(const void* qkv, int ldq, int T, void
       !(scale > 0.f) || max_new <= 0 || B > 65535 || ldq % 8 || ldo % 8 ||
       (max_new + kPfBQ - 1) / kPfBQ > 65535)
     return kBadArgument;
-  if (((uintptr_t)qkv | (uintptr_t)kc | (uintptr_t)vc | (uintptr_t)out) & 15) return kMisaligned;
-  const long long cache_rows = n_blocks * nkv * kPfBlk;
-  if (cache_rows > 0x7fffffffLL) return kBadArgument;
+  if (((uintptr_t)qkv | (uintptr_t)kc | (uintptr_t)vc | (uintptr_t)out | (uintptr_t)pool_k |
+       (uintptr_t)pool_v) & 15)
+    return kMisaligned;
+  const long long cache_rows = n_blocks * nkv * kPfBlk, pool_rows = pool_blocks * nkv * kPfBlk;
+  if (cache_rows > 0x7fffffffLL || pool_rows > 0x7fffffffLL) return kBadArgument;
   CUtensorMap map_q, map_k, map_v;
   if (make_tile_map_bf16(&map_q, qkv, T, ldq, ldq, kPfBQ)) return kBadArgument;
   if (make_tile_map_bf16(&map_k, kc, (int)cache_rows, hd, hd, kPfBlk)) return kBadArgument;
   if (make_tile_map_bf16(&map_v, vc, (int)cache_rows, hd, hd, kPfBlk)) return kBadArgument;
+  CUtensorMap map_pk = map_k, map_pv = map_v;    // (not read without entries)
+  if (pool_table && (make_tile_map_bf16(&map_pk, pool_k, (int)pool_rows, hd, hd, kPfBlk) ||
+                     make_tile_map_bf16(&map_pv, pool_v, (int)pool_rows, hd, hd, kPfBlk)))
+    return kBadArgument;
   const int n_sub = (hd + 63) / 64;
   const PfSmem L(n_sub);
   cudaStream_t st = (cudaStream_t)stream;
@@ -1024,32 +1070,28 @@ extern "C" int cretif_attn_prefill_tc_bias(const void* qkv, int ldq, int T, void
     return e == cudaSuccess ? launch_status() : (int)e;
   }
   count_variant(kVarPrefillAttn);
+#define CRETIF_PF(HDMAX, POOLED)                                                                   \
+  do {                                                                                             \
+    static int configured = 0;                                                                     \
+    if (smem_bytes > configured) {                                                                 \
+      e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HDMAX, POOLED>,                              \
+                               cudaFuncAttributeMaxDynamicSharedMemorySize, smem_bytes);           \
+      if (e != cudaSuccess) return (int)e;                                                         \
+      configured = smem_bytes;                                                                     \
+    }                                                                                              \
+    e = cudaLaunchKernelEx(&cfg, attn_prefill_tc_kernel<HDMAX, POOLED>, map_q, map_k, map_v,       \
+                           (__nv_bfloat16*)out, ldo, table, table_stride, cu_seqlens, seq_start,   \
+                           seq_slot, nh, nkv, hd, scale_log2, window, fault, g_pf_stamps, sink,    \
+                           bias_near, bias_far, n_far, bias_slope, map_pk, map_pv, pooled);        \
+    if (e != cudaSuccess) return (int)e;                                                           \
+  } while (0)
   if (hd <= 64) {
-    static int configured = 0;
-    if (smem_bytes > configured) {
-      e = cudaFuncSetAttribute(attn_prefill_tc_kernel<64>,
-                               cudaFuncAttributeMaxDynamicSharedMemorySize, smem_bytes);
-      if (e != cudaSuccess) return (int)e;
-      configured = smem_bytes;
-    }
-    e = cudaLaunchKernelEx(&cfg, attn_prefill_tc_kernel<64>, map_q, map_k, map_v,
-                           (__nv_bfloat16*)out, ldo, table, table_stride, cu_seqlens, seq_start,
-                           seq_slot, nh, nkv, hd, scale_log2, window, fault, g_pf_stamps, sink,
-                           bias_near, bias_far, n_far, bias_slope);
-    if (e != cudaSuccess) return (int)e;
+    if (pool_table) CRETIF_PF(64, true);
+    else CRETIF_PF(64, false);
   } else {
-    static int configured = 0;
-    if (smem_bytes > configured) {
-      e = cudaFuncSetAttribute(attn_prefill_tc_kernel<128>,
-                               cudaFuncAttributeMaxDynamicSharedMemorySize, smem_bytes);
-      if (e != cudaSuccess) return (int)e;
-      configured = smem_bytes;
-    }
-    e = cudaLaunchKernelEx(&cfg, attn_prefill_tc_kernel<128>, map_q, map_k, map_v,
-                           (__nv_bfloat16*)out, ldo, table, table_stride, cu_seqlens, seq_start,
-                           seq_slot, nh, nkv, hd, scale_log2, window, fault, g_pf_stamps, sink,
-                           bias_near, bias_far, n_far, bias_slope);
-    if (e != cudaSuccess) return (int)e;
+    if (pool_table) CRETIF_PF(128, true);
+    else CRETIF_PF(128, false);
   }
+#undef CRETIF_PF
   return launch_status();
 }

@@ -24,6 +24,11 @@
 // Slope by distance: slope[heads]; a key n positions back has slope[h] * n taken off its scaled
 // score.  The mask is first_visible_key(pos, window): every key, a sliding window, or the
 // query's own chunk of positions.
+//
+// Pooled entries (PooledKeys, common.cuh): the entries that a query sees are walked like keys, after
+// the tokens and in the same softmax; bias and slope are the tokens' only.
+#include <type_traits>
+
 #include "api.h"
 #include "common.cuh"
 
@@ -42,7 +47,7 @@ attn_simt_kernel(const T* __restrict__ q, int ldq, T* __restrict__ out, int ldo,
                  const int* __restrict__ seq_slot, int nh, int nkv, int hd, float scale,
                  int window, int bt, int T_tokens, const float* __restrict__ sink, int vd,
                  const float* __restrict__ bias, const int* __restrict__ bias_edges,
-                 int bias_rows, const float* __restrict__ slope) {
+                 int bias_rows, const float* __restrict__ slope, const PooledKeys pooled) {
   __shared__ float qs[kMaxHd];
   __shared__ float bias_s[kMaxBiasRows];
   __shared__ int edge_s[kMaxBiasRows];
@@ -72,78 +77,87 @@ attn_simt_kernel(const T* __restrict__ q, int ldq, T* __restrict__ out, int ldo,
 #pragma unroll
   for (int i = 0; i < kMaxHd / 32; ++i) acc[i] = 0.f;
 
-  for (int base = first + 32 * warp; base <= pos; base += 32 * kWarps) {
-    const int key = base + lane;
-    bool valid = key <= pos;
-    float s = -INFINITY;
-    unsigned long long row = 0;
-    const int blk = valid ? tab[key / bt] : -1;
-    valid = blk >= 0;                 // a position without a block counts as masked
-    if (valid) {
-      row = ((unsigned long long)blk * nkv + kvh) * bt + (key % bt);
-      const T* kp = kc + row * hd;
-      float dot = 0.f;
-      if ((hd & 7) == 0) {
+  // Keys lo .. hi of one block cache join the softmax.  TOKENS: the sequence's own keys (a bias or
+  // slope by distance applies), else its pooled entries.
+  auto walk = [&](auto tokens, int lo, int hi, const T* kbase, const T* vbase, const int* tbl) {
+    constexpr bool TOKENS = decltype(tokens)::value;
+    for (int base = lo + 32 * warp; base <= hi; base += 32 * kWarps) {
+      const int key = base + lane;
+      bool valid = key <= hi;
+      float s = -INFINITY;
+      unsigned long long row = 0;
+      const int blk = valid ? tbl[key / bt] : -1;
+      valid = blk >= 0;                 // a position without a block counts as masked
+      if (valid) {
+        row = ((unsigned long long)blk * nkv + kvh) * bt + (key % bt);
+        const T* kp = kbase + row * hd;
+        float dot = 0.f;
+        if ((hd & 7) == 0) {
 #pragma unroll 4
-        for (int d = 0; d < hd; d += 8) {
-          float kv[8];
-          load8(kp + d, kv);
+          for (int d = 0; d < hd; d += 8) {
+            float kv[8];
+            load8(kp + d, kv);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) dot = fmaf(qs[d + e], kv[e], dot);
+            for (int e = 0; e < 8; ++e) dot = fmaf(qs[d + e], kv[e], dot);
+          }
+        } else {                        // a head size that is no multiple of 8: element by element
+          for (int d = 0; d < hd; ++d) dot = fmaf(qs[d], to_float(kp[d]), dot);
         }
-      } else {                        // a head size that is no multiple of 8: element by element
-        for (int d = 0; d < hd; ++d) dot = fmaf(qs[d], to_float(kp[d]), dot);
+        s = dot * scale;
+        if (TOKENS && slope) s -= tilt * (float)(pos - key);
+        if (TOKENS && bias) {
+          // the last row whose edge is at or below the distance
+          const int n = pos - key;
+          int lo = 0, hi = bias_rows - 1;
+          while (lo < hi) {
+            const int mid = (lo + hi + 1) >> 1;
+            if (edge_s[mid] <= n) lo = mid; else hi = mid - 1;
+          }
+          s += bias_s[lo];
+        }
       }
-      s = dot * scale;
-      if (slope) s -= tilt * (float)(pos - key);
-      if (bias) {
-        // the last row whose edge is at or below the distance
-        const int n = pos - key;
-        int lo = 0, hi = bias_rows - 1;
-        while (lo < hi) {
-          const int mid = (lo + hi + 1) >> 1;
-          if (edge_s[mid] <= n) lo = mid; else hi = mid - 1;
+      const float m_new = fmaxf(m, warp_max(s));
+      const float p = valid ? expf(s - m_new) : 0.f;
+      const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);   // nothing summed yet
+      l = l * corr + warp_sum(p);
+#pragma unroll
+      for (int i = 0; i < kMaxHd / 32; ++i) acc[i] *= corr;
+      m = m_new;
+      // Values: keys in ascending order, eight at a time so that their loads travel together
+      // (a decode step has one warp per head and nothing else to hide a load behind).  A key
+      // with p = 0 (masked, or underflowed) adds nothing and is not read.
+      const int n_valid = min(32, hi + 1 - base);
+      constexpr int kAhead = 8;
+      for (int j0 = 0; j0 < n_valid; j0 += kAhead) {
+        float pj[kAhead];
+        const T* vp[kAhead];
+#pragma unroll
+        for (int u = 0; u < kAhead; ++u) {
+          const int j = min(j0 + u, 31);
+          const float pu = __shfl_sync(0xffffffffu, p, j);
+          const unsigned long long ru = __shfl_sync(0xffffffffu, row, j);
+          pj[u] = j0 + u < n_valid ? pu : 0.f;
+          vp[u] = vbase + ru * vd;
         }
-        s += bias_s[lo];
+#pragma unroll
+        for (int i = 0; i < kMaxHd / 32; ++i) {
+          const int d = lane + 32 * i;
+          if (d < vd) {
+            float v[kAhead];
+#pragma unroll
+            for (int u = 0; u < kAhead; ++u) v[u] = pj[u] != 0.f ? to_float(vp[u][d]) : 0.f;
+#pragma unroll
+            for (int u = 0; u < kAhead; ++u)
+              if (pj[u] != 0.f) acc[i] = fmaf(pj[u], v[u], acc[i]);
+          }
+        }
       }
     }
-    const float m_new = fmaxf(m, warp_max(s));
-    const float p = valid ? expf(s - m_new) : 0.f;
-    const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);   // nothing summed yet
-    l = l * corr + warp_sum(p);
-#pragma unroll
-    for (int i = 0; i < kMaxHd / 32; ++i) acc[i] *= corr;
-    m = m_new;
-    // Values: keys in ascending order, eight at a time so that their loads travel together
-    // (a decode step has one warp per head and nothing else to hide a load behind).  A key
-    // with p = 0 (masked, or underflowed) adds nothing and is not read.
-    const int n_valid = min(32, pos + 1 - base);
-    constexpr int kAhead = 8;
-    for (int j0 = 0; j0 < n_valid; j0 += kAhead) {
-      float pj[kAhead];
-      const T* vp[kAhead];
-#pragma unroll
-      for (int u = 0; u < kAhead; ++u) {
-        const int j = min(j0 + u, 31);
-        const float pu = __shfl_sync(0xffffffffu, p, j);
-        const unsigned long long ru = __shfl_sync(0xffffffffu, row, j);
-        pj[u] = j0 + u < n_valid ? pu : 0.f;
-        vp[u] = vc + ru * vd;
-      }
-#pragma unroll
-      for (int i = 0; i < kMaxHd / 32; ++i) {
-        const int d = lane + 32 * i;
-        if (d < vd) {
-          float v[kAhead];
-#pragma unroll
-          for (int u = 0; u < kAhead; ++u) v[u] = pj[u] != 0.f ? to_float(vp[u][d]) : 0.f;
-#pragma unroll
-          for (int u = 0; u < kAhead; ++u)
-            if (pj[u] != 0.f) acc[i] = fmaf(pj[u], v[u], acc[i]);
-        }
-      }
-    }
-  }
+  };
+  walk(std::true_type{}, first, pos, kc, vc, tab);
+  if (pooled.table)
+    walk(std::false_type{}, 0, visible_pooled(pos, window, pooled.pool) - 1, (const T*)pooled.k,
+         (const T*)pooled.v, pooled.table + (size_t)slot * pooled.table_stride);
   // the warps' results meet in shared memory; warp 0 folds them in the warps' order
   if (lane == 0) {
     part_m[warp] = m;
@@ -203,7 +217,22 @@ extern "C" int cretif_attn_simt(const void* q, int ldq, void* out, int ldo, int 
                                 const float* sink, int vd, const float* bias,
                                 const int* bias_edges, int bias_rows, const float* slope,
                                 void* stream) {
+  return cretif_attn_simt_pooled(q, ldq, out, ldo, dt, kc, vc, table, table_stride, tok_pos, tok_seq,
+                                 seq_slot, nh, nkv, hd, scale, window, bt, T, sink, vd, bias,
+                                 bias_edges, bias_rows, slope, nullptr, nullptr, nullptr, 0, 0, stream);
+}
+
+// pool_k, pool_v [blocks, nkv, bt, hd or vd], pool_table [slots, pool_stride]: the entries per
+// complete block of `pool` tokens (pool_table null: none; they need a sliding window).
+extern "C" int cretif_attn_simt_pooled(
+    const void* q, int ldq, void* out, int ldo, int dt, const void* kc, const void* vc,
+    const int* table, int table_stride, const int* tok_pos, const int* tok_seq, const int* seq_slot,
+    int nh, int nkv, int hd, float scale, int window, int bt, int T, const float* sink, int vd,
+    const float* bias, const int* bias_edges, int bias_rows, const float* slope, const void* pool_k,
+    const void* pool_v, const int* pool_table, int pool_stride, int pool, void* stream) {
   if (T <= 0) return kOk;
+  if (pool_table && (!pool_k || !pool_v || pool <= 0 || window <= 0)) return kBadArgument;
+  const PooledKeys pooled{pool_k, pool_v, pool_table, pool_stride, pool, 0};
   if (nh <= 0 || nkv <= 0 || nh % nkv || hd <= 0 || hd > kMaxHd || bt <= 0 ||
       vd <= 0 || vd > kMaxHd)
     return kBadArgument;
@@ -216,12 +245,12 @@ extern "C" int cretif_attn_simt(const void* q, int ldq, void* out, int ldo, int 
     attn_simt_kernel<float><<<blocks, kWarps * 32, 0, st>>>(
         (const float*)q, ldq, (float*)out, ldo, (const float*)kc, (const float*)vc, table,
         table_stride, tok_pos, tok_seq, seq_slot, nh, nkv, hd, scale, window, bt, T, sink, vd, bias,
-        bias_edges, bias_rows, slope);
+        bias_edges, bias_rows, slope, pooled);
   else if (dt == kBF16)
     attn_simt_kernel<__nv_bfloat16><<<blocks, kWarps * 32, 0, st>>>(
         (const __nv_bfloat16*)q, ldq, (__nv_bfloat16*)out, ldo, (const __nv_bfloat16*)kc,
         (const __nv_bfloat16*)vc, table, table_stride, tok_pos, tok_seq, seq_slot, nh, nkv, hd,
-        scale, window, bt, T, sink, vd, bias, bias_edges, bias_rows, slope);
+        scale, window, bt, T, sink, vd, bias, bias_edges, bias_rows, slope, pooled);
   else
     return kBadDType;
   return launch_status();

@@ -182,6 +182,25 @@ __host__ __device__ __forceinline__ int first_visible_key(int pos, int window) {
   return 0;
 }
 
+// Pooled keys and values: one entry (a mean) per complete block of `pool` tokens, in a block cache
+// of its own that is laid out like the tokens'.  A query at position pos with a sliding window
+// sees, beside its window's tokens, entry b if the block's last token lies before the window:
+// b * pool + pool - 1 <= pos - window.  That is the first visible_pooled(pos, ..) entries, a number
+// that never decreases with pos.  table null: there are none.
+struct PooledKeys {
+  const void* k;
+  const void* v;
+  const int* table;
+  int table_stride;
+  int pool;
+  long long n_blocks;         // blocks of the entries' cache
+};
+
+__host__ __device__ __forceinline__ int visible_pooled(int pos, int window, int pool) {
+  const int before = pos - window + 1;          // tokens that lie before the window
+  return before > 0 ? before / pool : 0;
+}
+
 inline int launch_status() {
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : static_cast<int>(e);

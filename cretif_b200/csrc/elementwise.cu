@@ -17,7 +17,7 @@ __global__ void embed_rows_kernel(const T* __restrict__ table, const int* __rest
                                   float* __restrict__ out, int H, int V,
                                   unsigned int* __restrict__ fault,
                                   const T* __restrict__ pos_table, const int* __restrict__ tok_pos,
-                                  int P) {
+                                  int P, float scale) {
   const int t = blockIdx.x;
   const int id = ids[t];
   float* row = out + (size_t)t * H;
@@ -32,10 +32,10 @@ __global__ void embed_rows_kernel(const T* __restrict__ table, const int* __rest
   const T* src = table + (size_t)id * H;
   if (pos_table) {
     const T* pv = pos_table + (size_t)pos * H;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) row[i] = to_float(src[i]) + to_float(pv[i]);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) row[i] = to_float(src[i]) * scale + to_float(pv[i]);
     return;
   }
-  for (int i = threadIdx.x; i < H; i += blockDim.x) row[i] = to_float(src[i]);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) row[i] = to_float(src[i]) * scale;
 }
 
 // ---------------------------------------------------------------- residual + RMSNorm
@@ -312,18 +312,18 @@ using namespace cretif;
 
 extern "C" int cretif_embed_rows(const void* table, int table_dt, const int* ids, float* out,
                                  int T, int H, int V, unsigned int* fault, const void* pos_table,
-                                 const int* tok_pos, int P, void* stream) {
+                                 const int* tok_pos, int P, float scale, void* stream) {
   if (T <= 0) return kOk;
   if (H <= 0 || V <= 0 || (pos_table && (!tok_pos || P <= 0))) return kBadArgument;
   cudaStream_t st = (cudaStream_t)stream;
   const int threads = H >= 256 ? 256 : 64;
   if (table_dt == kF32)
     embed_rows_kernel<float><<<T, threads, 0, st>>>((const float*)table, ids, out, H, V, fault,
-                                                    (const float*)pos_table, tok_pos, P);
+                                                    (const float*)pos_table, tok_pos, P, scale);
   else if (table_dt == kBF16)
     embed_rows_kernel<__nv_bfloat16><<<T, threads, 0, st>>>(
         (const __nv_bfloat16*)table, ids, out, H, V, fault, (const __nv_bfloat16*)pos_table,
-        tok_pos, P);
+        tok_pos, P, scale);
   else
     return kBadDType;
   return launch_status();

@@ -11,6 +11,14 @@
 //   q, k:  channels (i, partner(i)) of the first rot_dim are rotated by pos * f_j
 //          (pairing 0: partner i + rot_dim/2; 1: i ^ 1), cos/sin from a 32-bit table
 //   q -> q_out, k -> key cache, v -> value cache at the token's position.
+//
+// projnorm_rope_kv_append: the same with the norms over the WHOLE query and the whole key projection
+// (a weight per channel), from float32 rows, a CTA per token; v is multiplied by v_scale before it is
+// stored, so that a factor on the attention's output costs nothing.
+//
+// Pooled entries (PooledKeys in common.cuh): pool_kv writes the means of the blocks of tokens that
+// the step completes; a step of one token a sequence does it at the end of
+// projnorm_rope_kv_append instead.
 #include "api.h"
 #include "common.cuh"
 
@@ -116,6 +124,189 @@ headnorm_rope_kv_append_kernel(const TI* __restrict__ proj, int ldp,
   }
 }
 
+// The mean of `pool` consecutive cached rows' channel c, from position p0: a 32-bit sum in the order
+// of the positions.
+template <typename T>
+__device__ __forceinline__ float pooled_mean(const T* cache, const int* tab, int p0, int pool, int nkv,
+                                             int kvh, int bt, int n, int c) {
+  float sum = 0.f;
+#pragma unroll 4
+  for (int r = 0; r < pool; ++r) {
+    const int p = p0 + r, blk = max(tab[p / bt], 0);
+    sum += to_float(cache[(((size_t)blk * nkv + kvh) * bt + p % bt) * n + c]);
+  }
+  return sum / (float)pool;
+}
+
+// A sequence's entry e (its block of tokens is complete) -> the entries' cache, by the threads
+// tid, tid + threads, ... of a CTA, for the key/value heads kv0 .. kv1 - 1.
+template <typename T>
+__device__ __forceinline__ void write_entry(const T* kc, const T* vc, const int* tab, T* pk, T* pv,
+                                            const int* ptab, int pool, int e, int nkv, int kv0,
+                                            int kv1, int hd, int vd, int bt, int tid, int threads,
+                                            unsigned int* fault) {
+  const int blk = ptab[e / bt];
+  if (blk < 0) {
+    if (tid == 0) atomicOr(fault, kFaultBlockTable);
+    return;
+  }
+  const int per = hd + vd;
+  for (int idx = tid; idx < (kv1 - kv0) * per; idx += threads) {
+    const int kvh = kv0 + idx / per, c = idx % per;
+    const size_t row = ((size_t)blk * nkv + kvh) * bt + e % bt;
+    if (c < hd)
+      pk[row * hd + c] = from_float<T>(pooled_mean(kc, tab, e * pool, pool, nkv, kvh, bt, hd, c));
+    else
+      pv[row * vd + c - hd] =
+          from_float<T>(pooled_mean(vc, tab, e * pool, pool, nkv, kvh, bt, vd, c - hd));
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+pool_kv_kernel(const T* kc, const T* vc, const int* __restrict__ table, int table_stride, T* pk, T* pv,
+               const int* __restrict__ pool_table, int pool_stride, int pool,
+               const int* __restrict__ cu_seqlens, const int* __restrict__ seq_start,
+               const int* __restrict__ seq_slot, int nkv, int hd, int vd, int bt,
+               unsigned int* __restrict__ fault) {
+  const int b = blockIdx.z, kvh = blockIdx.y;
+  const int start = seq_start[b], end = start + cu_seqlens[b + 1] - cu_seqlens[b];
+  const int e = start / pool + blockIdx.x;
+  if (e >= end / pool) return;
+  const int slot = seq_slot[b];
+  write_entry(kc, vc, table + (size_t)slot * table_stride, pk, pv,
+              pool_table + (size_t)slot * pool_stride, pool, e, nkv, kvh, kvh + 1, hd, vd, bt,
+              (int)threadIdx.x, (int)blockDim.x, fault);
+}
+
+// VEC: four channels a thread (head size, rotated part and addresses allow it).
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
+                               const float* __restrict__ bias, const float* __restrict__ wq,
+                               const float* __restrict__ wk, float eps,
+                               const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                               int pairing, int rot_dim, const int* __restrict__ tok_pos,
+                               const int* __restrict__ tok_seq, const int* __restrict__ seq_slot,
+                               int nh, int nkv, int hd, int vd, float v_scale,
+                               T* __restrict__ q_out, int ldq, const int* __restrict__ table,
+                               int table_stride, T* kc, T* vc, int bt, int write_cache, T* pk, T* pv,
+                               const int* __restrict__ pool_table, int pool_stride, int pool,
+                               unsigned int* __restrict__ fault) {
+  extern __shared__ __align__(16) float row_s[];       // q | k with the bias
+  __shared__ float sums[8][2];
+  const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int pos = tok_pos[t];
+  const float* row = proj + (size_t)t * ldp;
+  const int nq = nh * hd, nk = nkv * hd, nqk = nq + nk;
+  float ssq = 0.f, ssk = 0.f;
+  if (VEC) {
+    for (int i = 4 * tid; i < nqk; i += 4 * 256) {
+      float4 v = *reinterpret_cast<const float4*>(row + i);
+      if (bias) {
+        const float4 b4 = *reinterpret_cast<const float4*>(bias + i);
+        v.x += b4.x; v.y += b4.y; v.z += b4.z; v.w += b4.w;
+      }
+      *reinterpret_cast<float4*>(row_s + i) = v;
+      const float s4 = v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      if (i < nq) ssq += s4; else ssk += s4;
+    }
+  } else {
+    for (int i = tid; i < nqk; i += 256) {
+      const float v = row[i] + (bias ? bias[i] : 0.f);
+      row_s[i] = v;
+      if (i < nq) ssq += v * v; else ssk += v * v;
+    }
+  }
+  int slot = 0, blk = -1;
+  if (write_cache) {
+    slot = seq_slot[tok_seq[t]];
+    blk = table[(size_t)slot * table_stride + pos / bt];
+    if (blk < 0 && tid == 0) atomicOr(fault, kFaultBlockTable);
+  }
+  ssq = warp_sum(ssq);
+  ssk = warp_sum(ssk);
+  if (lane == 0) { sums[warp][0] = ssq; sums[warp][1] = ssk; }
+  __syncthreads();
+  ssq = ssk = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) { ssq += sums[w][0]; ssk += sums[w][1]; }
+  const float fq = 1.0f / sqrtf(ssq / (float)nq + eps);
+  const float fk = nk ? 1.0f / sqrtf(ssk / (float)nk + eps) : 0.f;
+  const int half = rot_dim >> 1;
+  const float* c = cos_t + (size_t)pos * half;
+  const float* s = sin_t + (size_t)pos * half;
+  const int n_write = write_cache && blk >= 0 ? nqk : nq;
+  auto normed = [&](int idx) {
+    return idx < nq ? row_s[idx] * fq * wq[idx] : row_s[idx] * fk * wk[idx - nq];
+  };
+  auto target = [&](int idx, int i) {              // where channel i of the head of column idx goes
+    if (idx < nq) return q_out + (size_t)t * ldq + idx;
+    const int kvh = (idx - nq) / hd;
+    return kc + (((size_t)blk * nkv + kvh) * bt + pos % bt) * hd + i;
+  };
+  if (VEC) {
+    for (int idx = 4 * tid; idx < n_write; idx += 4 * 256) {
+      const int i = idx % hd;
+      float v[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) v[u] = normed(idx + u);
+      if (i < rot_dim) {
+        if (pairing) {
+          const int j = i >> 1;
+          const float c0 = c[j], s0 = s[j], c1 = c[j + 1], s1 = s[j + 1];
+          const float a = v[0], b = v[1], d = v[2], e = v[3];
+          v[0] = a * c0 - b * s0; v[1] = b * c0 + a * s0;
+          v[2] = d * c1 - e * s1; v[3] = e * c1 + d * s1;
+        } else {
+          const bool first = i < half;
+          const int j = first ? i : i - half;
+#pragma unroll
+          for (int u = 0; u < 4; ++u) {
+            const float other = normed(idx + u + (first ? half : -half));
+            v[u] = first ? v[u] * c[j + u] - other * s[j + u] : v[u] * c[j + u] + other * s[j + u];
+          }
+        }
+      }
+      T* dst = target(idx, i);
+      if constexpr (sizeof(T) == 2) {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+        uint2 u2;
+        u2.x = *reinterpret_cast<uint32_t*>(&lo);
+        u2.y = *reinterpret_cast<uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>(dst) = u2;
+      } else {
+        *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+      }
+    }
+  } else {
+    for (int idx = tid; idx < n_write; idx += 256) {
+      const int i = idx % hd;
+      float v = normed(idx);
+      if (i < rot_dim) {
+        const bool first = pairing ? !(i & 1) : i < half;
+        const int j = pairing ? i >> 1 : (first ? i : i - half);
+        const int partner = pairing ? i ^ 1 : (first ? i + half : i - half);
+        const float other = normed(idx - i + partner);
+        v = first ? v * c[j] - other * s[j] : v * c[j] + other * s[j];
+      }
+      *target(idx, i) = from_float<T>(v);
+    }
+  }
+  if (!write_cache || blk < 0) return;
+  for (int idx = tid; idx < nkv * vd; idx += 256) {
+    const int kvh = idx / vd, i = idx - kvh * vd;
+    const float v = row[nqk + idx] + (bias ? bias[nqk + idx] : 0.f);
+    vc[(((size_t)blk * nkv + kvh) * bt + pos % bt) * vd + i] = from_float<T>(v * v_scale);
+  }
+  if (pool_table && (pos + 1) % pool == 0) {       // (one token a sequence: this one ends a block)
+    __syncthreads();
+    write_entry<T>(kc, vc, table + (size_t)slot * table_stride, pk, pv,
+                   pool_table + (size_t)slot * pool_stride, pool, pos / pool, nkv, 0, nkv, hd, vd, bt,
+                   tid, 256, fault);
+  }
+}
+
 // o[t, h, :] *= sigmoid(g[t, h]): a gate per head from a float32 column of the projections.
 template <typename T>
 __global__ void gate_heads_kernel(T* __restrict__ o, int ldo, const float* __restrict__ g, int ldg,
@@ -193,6 +384,11 @@ __global__ void softcap_kernel(float* __restrict__ z, long long total, float cap
   if (idx < total) z[idx] = cap * tanhf(z[idx] / cap);
 }
 
+__global__ void scale_kernel(float* __restrict__ z, long long total, float factor) {
+  const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx < total) z[idx] *= factor;
+}
+
 // h += alpha * y, 32-bit (y float32 or bfloat16).
 template <typename TY>
 __global__ void axpy_rows_kernel(float* __restrict__ h, const TY* __restrict__ y, float alpha,
@@ -246,6 +442,87 @@ extern "C" int cretif_headnorm_rope_kv_append(
     return kBadDType;
 #undef CRETIF_HN_T
 #undef CRETIF_HN
+  return launch_status();
+}
+
+// proj float32; pool_table non-null: the step brings one token a sequence and the entry of a block
+// that a token completes is written here.
+extern "C" int cretif_projnorm_rope_kv_append(
+    const float* proj, int ldp, const float* bias, const float* wq, const float* wk, float eps,
+    const float* cos_t, const float* sin_t, int pairing, int rot_dim, const int* tok_pos,
+    const int* tok_seq, const int* seq_slot, int nh, int nkv, int hd, int vd, float v_scale,
+    void* q_out, int ldq, int dt, const int* table, int table_stride, void* kc, void* vc, int bt,
+    int write_cache, void* pool_k, void* pool_v, const int* pool_table, int pool_stride, int pool,
+    int T, unsigned int* fault, void* stream) {
+  if (T <= 0) return kOk;
+  if (nh <= 0 || nkv < 0 || hd <= 0 || vd <= 0 || ldq < nh * hd || rot_dim < 0 || rot_dim > hd ||
+      (rot_dim & 1) || !wq || (nkv && !wk) || ldp < (nh + nkv) * hd + nkv * vd)
+    return kBadArgument;
+  if (rot_dim > 0 && (!cos_t || !sin_t)) return kBadArgument;
+  if (write_cache && (bt <= 0 || nkv <= 0 || !kc || !vc || !table || !tok_seq || !seq_slot))
+    return kBadArgument;
+  if (pool_table && (!write_cache || pool <= 0 || !pool_k || !pool_v)) return kBadArgument;
+  const size_t smem = sizeof(float) * (size_t)(nh + nkv) * hd;
+  if (smem > 200 * 1024) return kBadArgument;
+  const bool vec = hd % 4 == 0 && ldp % 4 == 0 && ldq % 4 == 0 &&
+                   (pairing ? rot_dim % 4 == 0 : rot_dim % 8 == 0) &&
+                   (((uintptr_t)proj | (uintptr_t)bias | (uintptr_t)q_out | (uintptr_t)kc) & 15) == 0;
+  cudaStream_t st = (cudaStream_t)stream;
+#define CRETIF_PN(TT, VEC)                                                                        \
+  do {                                                                                            \
+    if (smem > 40 * 1024) {                                                                       \
+      cudaError_t err = cudaFuncSetAttribute(projnorm_rope_kv_append_kernel<TT, VEC>,             \
+                                             cudaFuncAttributeMaxDynamicSharedMemorySize,         \
+                                             (int)smem);                                          \
+      if (err != cudaSuccess) return (int)err;                                                    \
+    }                                                                                             \
+    projnorm_rope_kv_append_kernel<TT, VEC><<<T, 256, smem, st>>>(                                \
+        proj, ldp, bias, wq, wk, eps, cos_t, sin_t, pairing, rot_dim, tok_pos, tok_seq, seq_slot, \
+        nh, nkv, hd, vd, v_scale, (TT*)q_out, ldq, table, table_stride, (TT*)kc, (TT*)vc, bt,     \
+        write_cache, (TT*)pool_k, (TT*)pool_v, pool_table, pool_stride, pool, fault);             \
+  } while (0)
+  if (dt == kF32) {
+    if (vec) CRETIF_PN(float, true);
+    else CRETIF_PN(float, false);
+  } else if (dt == kBF16) {
+    if (vec) CRETIF_PN(__nv_bfloat16, true);
+    else CRETIF_PN(__nv_bfloat16, false);
+  } else {
+    return kBadDType;
+  }
+#undef CRETIF_PN
+  return launch_status();
+}
+
+extern "C" int cretif_pool_kv(const void* kc, const void* vc, int dt, const int* table,
+                              int table_stride, void* pool_k, void* pool_v, const int* pool_table,
+                              int pool_stride, int pool, const int* cu_seqlens, const int* seq_start,
+                              const int* seq_slot, int nkv, int hd, int vd, int bt, int B,
+                              int max_new, unsigned int* fault, void* stream) {
+  if (B <= 0 || max_new <= 0) return kOk;
+  if (pool <= 0 || nkv <= 0 || nkv > 65535 || B > 65535 || hd <= 0 || vd <= 0 || bt <= 0 || !table ||
+      !pool_table || !pool_k || !pool_v)
+    return kBadArgument;
+  // (n new tokens complete at most ceil(n / pool) blocks)
+  const dim3 grid((max_new + pool - 1) / pool, nkv, B);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (dt == kF32)
+    pool_kv_kernel<float><<<grid, 128, 0, st>>>(
+        (const float*)kc, (const float*)vc, table, table_stride, (float*)pool_k, (float*)pool_v,
+        pool_table, pool_stride, pool, cu_seqlens, seq_start, seq_slot, nkv, hd, vd, bt, fault);
+  else if (dt == kBF16)
+    pool_kv_kernel<__nv_bfloat16><<<grid, 128, 0, st>>>(
+        (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, table, table_stride,
+        (__nv_bfloat16*)pool_k, (__nv_bfloat16*)pool_v, pool_table, pool_stride, pool, cu_seqlens,
+        seq_start, seq_slot, nkv, hd, vd, bt, fault);
+  else
+    return kBadDType;
+  return launch_status();
+}
+
+extern "C" int cretif_scale(float* z, long long total, float factor, void* stream) {
+  if (total <= 0) return kOk;
+  scale_kernel<<<(unsigned)((total + 255) / 256), 256, 0, (cudaStream_t)stream>>>(z, total, factor);
   return launch_status();
 }
 

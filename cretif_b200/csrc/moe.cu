@@ -4,8 +4,11 @@
 // slice of two grouped matrix products (gate|up with the activation in the epilogue, down):
 //
 // * moe_route (a CTA per token): router logits z = W_r x in 32-bit (W_r float32; x as stored),
-//   score s = 1 / (1 + e^-z), the `top` largest (ties: the lower index), weights = the scores
-//   as they are, or divided by their sum when asked.
+//   score s = 1 / (1 + e^-z) or the softmax over all outputs, the `top` largest choices (a choice is
+//   the score, plus a correction per output where there is one; ties: the lower index), weights =
+//   the scores as they are, or divided by their sum when asked.
+// * Router outputs beyond the E experts are identities: such a pair has no rows in the products (its
+//   place is -1), and moe_combine adds the weight times the token's own input row.
 // * moe_group (one CTA): counts per expert, offsets, each pair's place in the sorted list and
 //   the list of row tiles (expert, first row) that the products walk.  The number of tiles is at
 //   most ceil(pairs / 64) + E, which the host knows, so the grid does not depend on the routing
@@ -37,17 +40,20 @@ namespace {
 constexpr int kTile = 64;
 constexpr int kMaxExpertsPerLane = 8;            // E <= 256
 
-// How a token's experts are chosen.  groups > 1: the experts form that many equal groups of
-// neighbours, a group's score is the sum of its two largest logistic scores, and only experts of
-// the `keep` best groups can be chosen.  renorm: the chosen scores are divided by their sum plus
-// sum_eps.
+// How a token's experts are chosen.  softmax: the scores are the softmax of the logits, else their
+// logistic function.  correction [E] (may be null): added to the scores for the choice only.
+// groups > 1: the experts form that many equal groups of neighbours, a group's score is the sum of
+// its two largest choice scores (group_best: the largest alone), and only experts of the `keep` best
+// groups can be chosen.  renorm: the chosen scores are divided by their sum plus sum_eps.
 struct RouteRule {
   int top, renorm, groups, keep;
   float sum_eps;
+  int softmax, group_best;
+  const float* correction;
 };
 
-// Warp-wide: the `top` largest of E logits (ties: the lower index) among the experts of the groups
-// that are kept, their logistic scores as weights, written for token t.  `scratch`: E floats and
+// Warp-wide: the `top` largest choices of E outputs (ties: the lower index) among those of the groups
+// that are kept, their scores as weights, written for token t.  `scratch`: E floats and
 // `groups` ints of shared memory that belong to this warp.
 __device__ __forceinline__ void select_top(const float* logits, int E, const RouteRule rule,
                                            int* __restrict__ ids, float* __restrict__ wts, int t,
@@ -59,6 +65,33 @@ __device__ __forceinline__ void select_top(const float* logits, int E, const Rou
     const int e = lane + 32 * m;
     z[m] = e < E ? logits[e] : -INFINITY;
   }
+  // sc: the scores; z from here on: what the choice compares (the logits order like their logistic
+  // scores, so without a correction they are compared as they are)
+  float sc[kMaxExpertsPerLane];
+  if (rule.softmax) {
+    float mx = -INFINITY, sum = 0.f;
+#pragma unroll
+    for (int m = 0; m < kMaxExpertsPerLane; ++m) mx = fmaxf(mx, z[m]);
+    mx = warp_max(mx);
+#pragma unroll
+    for (int m = 0; m < kMaxExpertsPerLane; ++m) {
+      sc[m] = lane + 32 * m < E ? expf(z[m] - mx) : 0.f;
+      sum += sc[m];
+    }
+    sum = warp_sum(sum);
+#pragma unroll
+    for (int m = 0; m < kMaxExpertsPerLane; ++m) sc[m] /= sum;
+  } else {
+#pragma unroll
+    for (int m = 0; m < kMaxExpertsPerLane; ++m) sc[m] = 1.0f / (1.0f + expf(-z[m]));
+  }
+  if (rule.correction) {
+#pragma unroll
+    for (int m = 0; m < kMaxExpertsPerLane; ++m) {
+      const int e = lane + 32 * m;
+      if (e < E) z[m] = sc[m] + rule.correction[e];
+    }
+  }
   if (rule.groups > 1) {
     const int per = E / rule.groups;
     int* kept = reinterpret_cast<int*>(scratch + E);
@@ -66,11 +99,11 @@ __device__ __forceinline__ void select_top(const float* logits, int E, const Rou
 #pragma unroll
     for (int m = 0; m < kMaxExpertsPerLane; ++m) {
       const int e = lane + 32 * m;
-      if (e < E) scratch[e] = 1.0f / (1.0f + expf(-z[m]));
+      if (e < E) scratch[e] = rule.correction ? z[m] : sc[m];
     }
     for (int g = lane; g < rule.groups; g += 32) kept[g] = 0;
     __syncwarp();
-    // lane g % 32 scores group g: its two largest scores, summed
+    // lane g % 32 scores group g by its largest or its two largest choice scores
     float gs[kMaxExpertsPerLane];
 #pragma unroll
     for (int m = 0; m < kMaxExpertsPerLane; ++m) {
@@ -82,7 +115,7 @@ __device__ __forceinline__ void select_top(const float* logits, int E, const Rou
           const float v = scratch[g * per + i];
           if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
         }
-        gs[m] = per > 1 ? a + b : a;
+        gs[m] = per > 1 && !rule.group_best ? a + b : a;
       }
     }
     for (int k = 0; k < rule.keep; ++k) {
@@ -131,12 +164,17 @@ __device__ __forceinline__ void select_top(const float* logits, int E, const Rou
       const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
       if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
     }
+    if (best_e >= E) best_e = k;                 // (nothing comparable left: not a number)
+    float s = 0.f;
     if ((best_e & 31) == lane) {
 #pragma unroll
       for (int m = 0; m < kMaxExpertsPerLane; ++m)
-        if (m == (best_e >> 5)) z[m] = -INFINITY;
+        if (m == (best_e >> 5)) {
+          z[m] = -INFINITY;
+          s = sc[m];
+        }
     }
-    const float s = 1.0f / (1.0f + expf(-best));
+    s = __shfl_sync(0xffffffffu, s, best_e & 31);
     total += s;
     if (lane == k % 32 && k < 32) { my_w = s; my_id = best_e; }
     if (k >= 32 && lane == 0) {                  // more than 32 choices: written one by one
@@ -223,7 +261,8 @@ moe_group_kernel(const int* __restrict__ ids, int P, int E, int* __restrict__ of
   int* start = sh + 2 * E;
   for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = cursor[e] = 0;
   __syncthreads();
-  for (int p = threadIdx.x; p < P; p += blockDim.x) atomicAdd(&counts[ids[p]], 1);
+  for (int p = threadIdx.x; p < P; p += blockDim.x)
+    if (ids[p] < E) atomicAdd(&counts[ids[p]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int at = 0, n_tiles = 0;
@@ -244,6 +283,10 @@ moe_group_kernel(const int* __restrict__ ids, int P, int E, int* __restrict__ of
   __syncthreads();
   for (int p = threadIdx.x; p < P; p += blockDim.x) {
     const int e = ids[p];
+    if (e >= E) {                                // an identity: no row in the products
+      place[p] = -1;
+      continue;
+    }
     const int at = start[e] + atomicAdd(&cursor[e], 1);
     place[p] = at;
     if (order) order[at] = p;
@@ -257,6 +300,7 @@ moe_gather_rows_kernel(const __nv_bfloat16* __restrict__ x, int ldx,
                        __nv_bfloat16* __restrict__ xs, int lds, const int* __restrict__ place,
                        const float* __restrict__ wts, int top, int K, int vec) {
   const int p = blockIdx.x;
+  if (place[p] < 0) return;
   const __nv_bfloat16* src = x + (size_t)(p / top) * ldx;
   __nv_bfloat16* dst = xs + (size_t)place[p] * lds;
   const float s = wts ? wts[p] : 1.f;
@@ -504,11 +548,12 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 moe_gemv_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, void* Cv, int ldc, int N,
                 int K, int top, int mode, int scale_at, const int* __restrict__ ids,
-                const float* __restrict__ wts, int vec) {
+                const float* __restrict__ wts, int vec, int experts) {
   extern __shared__ __align__(16) unsigned char gemv_smem[];
   T* xs = reinterpret_cast<T*>(gemv_smem);
   const int p = blockIdx.y;
   const int e = ids[p];
+  if (e >= experts) return;                      // an identity (moe_combine reads no row of it)
   const float s = scale_at ? wts[p] : 1.f;
   const T* arow = A + (size_t)(mode != 1 ? p / top : p) * lda;
   if (vec) {
@@ -559,15 +604,24 @@ moe_gemv_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, void*
   }
 }
 
+// Identity pairs (ids[pair] >= experts): id_wts[pair] times the token's row of x instead of a row of
+// the products.  wts: weights that the products have not applied yet.
+template <typename TX>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ rows, int ld, const int* __restrict__ place, int top,
-                   const float* __restrict__ wts, float* __restrict__ y, int T, int H) {
+                   const float* __restrict__ wts, float* __restrict__ y, int T, int H,
+                   const int* __restrict__ ids, int experts, const float* __restrict__ id_wts,
+                   const TX* __restrict__ x, int ldx) {
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= (long long)T * H) return;
   const int t = (int)(idx / H), c = (int)(idx - (long long)t * H);
   float acc = 0.f;
   for (int k = 0; k < top; ++k) {
     const size_t pair = (size_t)t * top + k;
+    if (ids && ids[pair] >= experts) {
+      acc += id_wts[pair] * to_float(x[(size_t)t * ldx + c]);
+      continue;
+    }
     const float v = rows[(place ? (size_t)place[pair] : pair) * ld + c];
     acc += wts ? wts[pair] * v : v;
   }
@@ -588,12 +642,13 @@ static bool route_rule_ok(int E, int top, int groups, int keep) {
 
 extern "C" int cretif_moe_route(const void* x, int x_dt, int ldx, const float* router_w, int E,
                                 int H, int top, int renorm, int groups, int keep, float sum_eps,
-                                int* ids, float* wts, int T, void* stream) {
+                                int softmax, int group_best, const float* correction, int* ids,
+                                float* wts, int T, void* stream) {
   if (T <= 0) return kOk;
   if (E <= 0 || E > 32 * kMaxExpertsPerLane || H <= 0 || top <= 0 || top > E || ldx < H)
     return kBadArgument;
   if (!route_rule_ok(E, top, groups, keep)) return kBadArgument;
-  const RouteRule rule{top, renorm, groups, keep, sum_eps};
+  const RouteRule rule{top, renorm, groups, keep, sum_eps, softmax, group_best, correction};
   cudaStream_t st = (cudaStream_t)stream;
   const int vec = H % 4 == 0 && ldx % 4 == 0 && (((uintptr_t)x | (uintptr_t)router_w) & 15) == 0;
   if (x_dt == kF32)
@@ -609,12 +664,12 @@ extern "C" int cretif_moe_route(const void* x, int x_dt, int ldx, const float* r
 
 // ids/wts from logits [T, ld >= E] that a matrix product computed.
 extern "C" int cretif_moe_topk(const float* logits, int ld, int E, int top, int renorm, int groups,
-                               int keep, float sum_eps, int* ids, float* wts, int T,
-                               void* stream) {
+                               int keep, float sum_eps, int softmax, int group_best,
+                               const float* correction, int* ids, float* wts, int T, void* stream) {
   if (T <= 0) return kOk;
   if (E <= 0 || E > kMaxExperts || top <= 0 || top > E || ld < E) return kBadArgument;
   if (!route_rule_ok(E, top, groups, keep)) return kBadArgument;
-  const RouteRule rule{top, renorm, groups, keep, sum_eps};
+  const RouteRule rule{top, renorm, groups, keep, sum_eps, softmax, group_best, correction};
   moe_topk_kernel<<<(unsigned)((T + 7) / 8), 256, 0, (cudaStream_t)stream>>>(logits, ld, E, rule,
                                                                              ids, wts, T);
   return launch_status();
@@ -706,7 +761,7 @@ extern "C" int cretif_moe_gemm(const void* A, int a_dt, int lda, const void* W, 
 // with C's rows indexed by the pair.
 extern "C" int cretif_moe_gemv(const void* A, int a_dt, int lda, const void* W, int w_dt, void* C,
                                int ldc, int N, int K, int top, int mode, int scale_at,
-                               const int* ids, const float* wts, int P, void* stream) {
+                               const int* ids, const float* wts, int P, int experts, void* stream) {
   if (P <= 0) return kOk;
   if (N <= 0 || K <= 0 || lda < K || ldc < N || top <= 0 || mode < 0 || mode >= 2 + kUnaryKinds ||
       scale_at < 0 || scale_at > 2 || P > 65535 || a_dt != w_dt)
@@ -725,7 +780,7 @@ extern "C" int cretif_moe_gemv(const void* A, int a_dt, int lda, const void* W, 
       if (err != cudaSuccess) return (int)err;
     }
     moe_gemv_kernel<float><<<grid, 256, smem, st>>>((const float*)A, lda, (const float*)W, C, ldc,
-                                                    N, K, top, mode, scale_at, ids, wts, vec);
+                                                    N, K, top, mode, scale_at, ids, wts, vec, experts);
   } else if (a_dt == kBF16) {
     if (smem > 48 * 1024) {
       cudaError_t err = cudaFuncSetAttribute(moe_gemv_kernel<bf16>,
@@ -733,18 +788,29 @@ extern "C" int cretif_moe_gemv(const void* A, int a_dt, int lda, const void* W, 
       if (err != cudaSuccess) return (int)err;
     }
     moe_gemv_kernel<bf16><<<grid, 256, smem, st>>>((const bf16*)A, lda, (const bf16*)W, C, ldc, N,
-                                                   K, top, mode, scale_at, ids, wts, vec);
+                                                   K, top, mode, scale_at, ids, wts, vec, experts);
   } else {
     return kBadDType;
   }
   return launch_status();
 }
 
+// ids non-null: pairs whose id is `experts` or more are identities (see moe_combine_kernel).
 extern "C" int cretif_moe_combine(const float* rows, int ld, const int* place, int top,
-                                  const float* wts, float* y, int T, int H, void* stream) {
+                                  const float* wts, float* y, int T, int H, const int* ids,
+                                  int experts, const float* id_wts, const void* x, int x_dt, int ldx,
+                                  void* stream) {
   if (T <= 0) return kOk;
-  if (H <= 0 || ld < H || top <= 0) return kBadArgument;
+  if (H <= 0 || ld < H || top <= 0 || (ids && (!id_wts || !x || ldx < H))) return kBadArgument;
   const unsigned blocks = (unsigned)(((long long)T * H + 255) / 256);
-  moe_combine_kernel<<<blocks, 256, 0, (cudaStream_t)stream>>>(rows, ld, place, top, wts, y, T, H);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (x_dt == kF32)
+    moe_combine_kernel<float><<<blocks, 256, 0, st>>>(rows, ld, place, top, wts, y, T, H, ids, experts,
+                                                      id_wts, (const float*)x, ldx);
+  else if (x_dt == kBF16)
+    moe_combine_kernel<__nv_bfloat16><<<blocks, 256, 0, st>>>(
+        rows, ld, place, top, wts, y, T, H, ids, experts, id_wts, (const __nv_bfloat16*)x, ldx);
+  else
+    return kBadDType;
   return launch_status();
 }

@@ -115,9 +115,9 @@ def _rows(t: torch.Tensor, name: str) -> int:
 
 
 # ------------------------------------------------------------------ elementwise
-def embed_rows(table, ids, out, fault, positions=None, tok_pos=None) -> None:
-    """``positions`` [P, H] (same type as ``table``) with ``tok_pos``: a learned vector per
-    position is added to each token's row."""
+def embed_rows(table, ids, out, fault, positions=None, tok_pos=None, scale: float = 1.0) -> None:
+    """A token's row times ``scale``; ``positions`` [P, H] (same type as ``table``) with
+    ``tok_pos``: a learned vector per position is added to it."""
     _need(table, "table", dim=2); _need(ids, "ids", torch.int32, 1)
     _need(out, "out", torch.float32, 2); _need(fault, "fault", torch.int32)
     T, (V, H) = ids.numel(), table.shape
@@ -131,7 +131,8 @@ def embed_rows(table, ids, out, fault, positions=None, tok_pos=None) -> None:
             raise KernelError(f"embed_rows: positions must be a contiguous [P, {H}] table with "
                               "a position per token")
     _check(lib().cretif_embed_rows(_p(table), _dt(table), _p(ids), _p(out), T, H, V, _p(fault),
-                                   _p(positions), _p(tok_pos), P, _stream()), "embed_rows")
+                                   _p(positions), _p(tok_pos), P, ctypes.c_float(scale), _stream()),
+           "embed_rows")
 
 
 def add_rmsnorm(h, delta, weight, out, eps: float, rows=None, write_h: bool = True) -> None:
@@ -407,6 +408,97 @@ def headnorm_rope_kv_append(proj, bias, wq, wk, eps: float, cos, sin, pairing: i
         int(write_cache), T, _p(fault), _stream()), "headnorm_rope_kv_append")
 
 
+def projnorm_rope_kv_append(proj, bias, wq, wk, eps: float, cos, sin, pairing: int, rot_dim: int,
+                            tok_pos, tok_seq, seq_slot, nh: int, nkv: int, hd: int, vd: int, q_out,
+                            table=None, kc=None, vc=None, block_tokens: int = 64,
+                            write_cache: bool = True, fault=None, v_scale: float = 1.0,
+                            pool=None) -> None:
+    """``headnorm_rope_kv_append`` with the norms over the whole query and the whole key projection
+    (``wq`` [nh hd], ``wk`` [nkv hd] float32), float32 ``proj``, and v times ``v_scale``.  ``pool``
+    (a PoolView; steps of one token a sequence): the entry of a block of tokens that a token
+    completes is written too."""
+    _need(proj, "proj", torch.float32, 2); _need(q_out, "q_out", dim=2)
+    _need(wq, "wq", torch.float32, 1)
+    T = proj.shape[0]
+    n_in = (nh + nkv) * hd + nkv * vd
+    if q_out.shape[0] != T or q_out.shape[1] < nh * hd or proj.shape[1] < n_in:
+        raise KernelError("projnorm_rope_kv_append: proj or q_out too narrow")
+    if wq.numel() != nh * hd or not wq.is_contiguous():
+        raise KernelError("projnorm_rope_kv_append: wq has a number per query column")
+    if nkv:
+        _need(wk, "wk", torch.float32, 1)
+        if wk.numel() != nkv * hd or not wk.is_contiguous():
+            raise KernelError("projnorm_rope_kv_append: wk has a number per key column")
+    if bias is not None:
+        _need(bias, "bias", torch.float32, 1)
+        if bias.numel() < n_in or not bias.is_contiguous():
+            raise KernelError("projnorm_rope_kv_append: the bias has a number per q, k and v column")
+    if rot_dim:
+        _need(cos, "cos", torch.float32, 2); _need(sin, "sin", torch.float32, 2)
+        if cos.shape[1] != rot_dim // 2 or not cos.is_contiguous() or not sin.is_contiguous():
+            raise KernelError("projnorm_rope_kv_append: cos/sin must be contiguous "
+                              "[positions, rot_dim/2]")
+    else:
+        cos = sin = None
+    _need(tok_pos, "tok_pos", torch.int32, 1)
+    if write_cache:
+        _need(tok_seq, "tok_seq", torch.int32, 1); _need(seq_slot, "seq_slot", torch.int32, 1)
+        _need(table, "table", torch.int32, 2)
+        _need(kc, "k cache", q_out.dtype, 4); _need(vc, "v cache", q_out.dtype, 4)
+        if (tuple(kc.shape[1:]) != (nkv, block_tokens, hd) or not kc.is_contiguous()
+                or tuple(vc.shape[1:]) != (nkv, block_tokens, vd) or not vc.is_contiguous()):
+            raise KernelError("projnorm_rope_kv_append: caches must be contiguous [blocks, "
+                              f"{nkv}, {block_tokens}, {hd}] and [..., {vd}]")
+        _need_pool(pool, kc, vc)
+    if fault is None:
+        fault = fault_word(proj.device)
+    _check(lib().cretif_projnorm_rope_kv_append(
+        _p(proj), _rows(proj, "proj"), _p(bias), _p(wq), _p(wk), ctypes.c_float(eps), _p(cos),
+        _p(sin), pairing, rot_dim, _p(tok_pos), _p(tok_seq), _p(seq_slot), nh, nkv, hd, vd,
+        ctypes.c_float(v_scale), _p(q_out), _rows(q_out, "q_out"), _dt(q_out), _p(table),
+        table.stride(0) if table is not None else 0, _p(kc), _p(vc), block_tokens,
+        int(write_cache), *_pool_args(pool if write_cache else None), T, _p(fault), _stream()),
+        "projnorm_rope_kv_append")
+
+
+def _need_pool(pool, kc, vc) -> None:
+    """A PoolView's tensors are laid out like the caches they stand beside."""
+    if pool is None:
+        return
+    _need(pool.k, "pooled keys", kc.dtype, 4); _need(pool.v, "pooled values", vc.dtype, 4)
+    _need(pool.table, "pool table", torch.int32, 2)
+    if (pool.k.shape[1:] != kc.shape[1:] or pool.v.shape[1:] != vc.shape[1:] or pool.pool < 1
+            or not pool.k.is_contiguous() or not pool.v.is_contiguous()):
+        raise KernelError("pooled entries must be laid out like the keys and values")
+
+
+def _pool_args(pool, blocks: bool = False):
+    """(k, v[, blocks], table, its stride, tokens an entry) of a PoolView, or of none."""
+    if pool is None:
+        return (None, None) + ((ctypes.c_longlong(0),) if blocks else ()) + (None, 0, 0)
+    return (_p(pool.k), _p(pool.v)) \
+        + ((ctypes.c_longlong(pool.k.shape[0]),) if blocks else ()) \
+        + (_p(pool.table), pool.table.stride(0), pool.pool)
+
+
+def pool_kv(kc, vc, table, pool, cu_seqlens, seq_start, seq_slot, nkv: int, hd: int, vd: int,
+            block_tokens: int, B: int, max_new: int, fault) -> None:
+    """The pooled entries of every block of ``pool.pool`` tokens that the step's tokens (already in
+    the cache) complete: the means of the block's rows."""
+    _need(kc, "k cache", dim=4); _need(vc, "v cache", kc.dtype, 4); _need(table, "table", torch.int32, 2)
+    if (tuple(kc.shape[1:]) != (nkv, block_tokens, hd) or not kc.is_contiguous()
+            or tuple(vc.shape[1:]) != (nkv, block_tokens, vd) or not vc.is_contiguous()):
+        raise KernelError("pool_kv: the caches' sizes do not fit")
+    _need_pool(pool, kc, vc)
+    for name, t in (("cu_seqlens", cu_seqlens), ("seq_start", seq_start), ("seq_slot", seq_slot)):
+        _need(t, name, torch.int32, 1)
+    pk, pv, ptab, pstride, P = _pool_args(pool)
+    _check(lib().cretif_pool_kv(
+        _p(kc), _p(vc), _dt(kc), _p(table), table.stride(0), pk, pv, ptab, pstride, P,
+        _p(cu_seqlens), _p(seq_start), _p(seq_slot), nkv, hd, vd, block_tokens, B, max_new,
+        _p(fault), _stream()), "pool_kv")
+
+
 def latent_in(proj, q_rank: int, rank: int, rot: int, wq, wc, eps: float, cos, sin, pairing: int,
               tok_pos, tok_seq, seq_slot, cq_out, table=None, kc=None, block_tokens: int = 64,
               write_cache: bool = True, fault=None, rot_dims: Optional[int] = None) -> None:
@@ -513,6 +605,15 @@ def activation(x, out, kind: str) -> None:
                                    _stream()), "activation")
 
 
+def scale_in_place(z, factor: float) -> None:
+    """z <- factor * z, float32."""
+    _need(z, "z", torch.float32)
+    if not z.is_contiguous():
+        raise KernelError("scale_in_place: z must be contiguous")
+    _check(lib().cretif_scale(_p(z), ctypes.c_longlong(z.numel()), ctypes.c_float(factor),
+                              _stream()), "scale")
+
+
 def softcap(z, cap: float) -> None:
     """``z <- cap * tanh(z / cap)`` in place (float32, contiguous)."""
     _need(z, "z", torch.float32)
@@ -572,6 +673,42 @@ def retention_recurrence(prep, v, decay, state, cu_seqlens, seq_slot, B: int, H:
         ctypes.c_longlong(state.stride(0)), _p(cu_seqlens), _p(seq_slot), B, H, d, e, _p(o_raw),
         int(write_state), T, {"auto": 0, "token": 1, "chunk": 2}[form], _stream()),
         "retention_recurrence")
+
+
+def matrix_memory(proj, bias_i, bias_f, cap: float, q_scale: float, state, cu_seqlens, seq_slot,
+                  tok_seq, B: int, H: int, d: int, e: int, norm_w, eps: float, out,
+                  write_state: bool = True, form: str = "auto") -> None:
+    """The matrix memory with exponential gates over the step's tokens of every (sequence, head), from
+    and to ``state`` (view [slots, >= H·d·(e+1) + H] float32: S, n and m), then the division, the
+    per-head RMS norm times ``norm_w`` [H·e] times sigmoid of the gate columns -> ``out`` [T, H·e].
+    ``proj`` rows (float32): [q | k | v | gate | input gate (H) | forget gate (H)].  ``form``:
+    ``"token"`` walks the tokens one by one, ``"chunk"`` takes 64 at a time as matrix products
+    (refused where sizes or addresses rule out 16-byte accesses), ``"auto"`` takes chunks where the
+    step brings 16 tokens a sequence or more and they are allowed."""
+    _need(proj, "proj", torch.float32, 2); _need(state, "state", torch.float32, 2)
+    _need(out, "out", dim=2)
+    for name, t, n in (("bias_i", bias_i, H), ("bias_f", bias_f, H), ("norm_w", norm_w, H * e)):
+        _need(t, name, torch.float32, 1)
+        if t.numel() != n or not t.is_contiguous():
+            raise KernelError(f"matrix_memory: {name} has {n} numbers")
+    for name, t in (("cu_seqlens", cu_seqlens), ("seq_slot", seq_slot), ("tok_seq", tok_seq)):
+        _need(t, name, torch.int32, 1)
+    T = proj.shape[0]
+    if (state.stride(1) != 1 or state.shape[1] < H * d * (e + 1) + H or out.shape[0] != T
+            or out.shape[1] < H * e or proj.shape[1] < 2 * H * (d + e) + 2 * H
+            or tok_seq.numel() < T):
+        raise KernelError("matrix_memory: the sizes do not fit")
+    n_o = T * H * e
+    scratch = torch.empty(n_o + 2 * T * H, dtype=torch.float32, device=proj.device)
+    chunks = form == "chunk" or (form == "auto" and T >= 16 * B)
+    gates = torch.empty(3 * H * T, dtype=torch.float64, device=proj.device) if chunks else None
+    _check(lib().cretif_matrix_memory(
+        _p(proj), _rows(proj, "proj"), _p(bias_i), _p(bias_f), ctypes.c_float(cap),
+        ctypes.c_float(q_scale), _p(state), ctypes.c_longlong(state.stride(0)), _p(cu_seqlens),
+        _p(seq_slot), _p(tok_seq), B, H, d, e, _p(norm_w), ctypes.c_float(eps), _p(scratch),
+        _p(scratch[n_o:]), _p(scratch[n_o + T * H:]), _p(gates), _p(out), _dt(out),
+        _rows(out, "out"), int(write_state), T, {"auto": 0, "token": 1, "chunk": 2}[form],
+        _stream()), "matrix_memory", kernels=3 if chunks else 2)
 
 
 def heads_out_norm(o_raw, gate, norm_w, eps: float, out, H: int, e: int,
@@ -763,12 +900,23 @@ def _route_rule(E: int, top: int, groups: int, keep: int) -> None:
                           f"{keep} hold {top} experts")
 
 
+def _correction(correction, E: int) -> None:
+    if correction is not None:
+        _need(correction, "correction", torch.float32, 1)
+        if correction.numel() != E or not correction.is_contiguous():
+            raise KernelError("routing: the correction has a number per router output")
+
+
 def moe_route(x, router_w, top: int, ids, wts, renorm: bool = False, groups: int = 0,
-              keep: int = 0, sum_eps: float = 0.0) -> None:
-    """ids/wts [T, top]: the ``top`` experts with the largest sigmoid(router_w · x) per token.
+              keep: int = 0, sum_eps: float = 0.0, softmax: bool = False, group_best: bool = False,
+              correction=None) -> None:
+    """ids/wts [T, top]: the ``top`` experts with the largest scores per token, a score being
+    sigmoid(router_w · x) or (``softmax``) its share of the softmax over all outputs.
+    ``correction`` (float32 [E]) is added to the scores for the choice, not for the weights.
     ``groups`` > 1: the experts form that many equal groups of neighbours, a group's score is
-    the sum of its two largest scores, and only experts of the ``keep`` best groups can be
-    chosen.  ``renorm``: the weights are divided by (their sum + ``sum_eps``)."""
+    the sum of its two largest choice scores (``group_best``: the largest), and only experts of the
+    ``keep`` best groups can be chosen.  ``renorm``: the weights are divided by (their sum +
+    ``sum_eps``)."""
     _need(x, "x", dim=2); _need(router_w, "router_w", torch.float32, 2)
     _need(ids, "ids", torch.int32, 2); _need(wts, "wts", torch.float32, 2)
     T, H = x.shape
@@ -779,13 +927,16 @@ def moe_route(x, router_w, top: int, ids, wts, renorm: bool = False, groups: int
     if not 0 < top <= E or E > 256:
         raise KernelError(f"moe_route: {top} of {E} experts (at most 256) cannot be chosen")
     _route_rule(E, top, groups, keep)
+    _correction(correction, E)
     _check(lib().cretif_moe_route(_p(x), _dt(x), _rows(x, "x"), _p(router_w), E, H, top,
                                   int(renorm), int(groups), int(keep), ctypes.c_float(sum_eps),
+                                  int(softmax), int(group_best), _p(correction),
                                   _p(ids), _p(wts), T, _stream()), "moe_route")
 
 
 def moe_topk(logits, top: int, ids, wts, renorm: bool = False, groups: int = 0, keep: int = 0,
-             sum_eps: float = 0.0) -> None:
+             sum_eps: float = 0.0, softmax: bool = False, group_best: bool = False,
+             correction=None) -> None:
     """``moe_route``'s choice from router logits [T, E] (float32) that a matrix product left."""
     _need(logits, "logits", torch.float32, 2); _need(ids, "ids", torch.int32, 2)
     _need(wts, "wts", torch.float32, 2)
@@ -794,14 +945,17 @@ def moe_topk(logits, top: int, ids, wts, renorm: bool = False, groups: int = 0, 
             or not wts.is_contiguous() or not 0 < top <= E or E > 256):
         raise KernelError("moe_topk: sizes do not fit")
     _route_rule(E, top, groups, keep)
+    _correction(correction, E)
     _check(lib().cretif_moe_topk(_p(logits), _rows(logits, "logits"), E, top, int(renorm),
-                                 int(groups), int(keep), ctypes.c_float(sum_eps), _p(ids),
-                                 _p(wts), T, _stream()), "moe_topk")
+                                 int(groups), int(keep), ctypes.c_float(sum_eps), int(softmax),
+                                 int(group_best), _p(correction), _p(ids), _p(wts), T, _stream()),
+           "moe_topk")
 
 
 def moe_group(ids, experts: int, offsets, place, order, tile_expert, tile_row0) -> None:
     """Sort the (token, choice) pairs by expert: ``offsets`` [E + 1], ``place`` [P] (a pair's
-    row in the sorted list), ``order`` [P] (its inverse) and the list of 64-row tiles."""
+    row in the sorted list), ``order`` [P] (its inverse) and the list of 64-row tiles.  Pairs whose
+    id is ``experts`` or more (identities) have no row: their place is -1."""
     for name, t in (("ids", ids), ("offsets", offsets), ("place", place), ("order", order),
                     ("tile_expert", tile_expert), ("tile_row0", tile_row0)):
         _need(t, name, torch.int32)
@@ -845,7 +999,8 @@ def moe_gemm(a, w, c, top: int, mode: int, scale_at: int, wts, order, offsets, t
 
 def moe_gemv(a, w, c, top: int, mode: int, scale_at: int, ids, wts) -> None:
     """``moe_gemm`` for a handful of pairs, in the pairs' own order (nothing is sorted): a CTA
-    per pair and 16 output columns streams the expert's rows once."""
+    per pair and 16 output columns streams the expert's rows once.  Pairs whose id is no expert's
+    (identities) are left out."""
     _need(a, "a", dim=2); _need(w, "w", a.dtype, 3); _need(c, "c", dim=2)
     _need(ids, "ids", torch.int32); _need(wts, "wts", torch.float32)
     K, N, P = a.shape[1], c.shape[1], ids.numel()
@@ -855,7 +1010,7 @@ def moe_gemv(a, w, c, top: int, mode: int, scale_at: int, ids, wts) -> None:
         raise KernelError("moe_gemv: sizes or element types do not fit")
     _check(lib().cretif_moe_gemv(
         _p(a), _dt(a), _rows(a, "a"), _p(w), _dt(w), _p(c), _rows(c, "c"), N, K, top, mode,
-        scale_at, _p(ids), _p(wts), P, _stream()), "moe_gemv")
+        scale_at, _p(ids), _p(wts), P, w.shape[0], _stream()), "moe_gemv")
 
 
 MOE_TC_TILE = 128
@@ -946,10 +1101,11 @@ def gemm_tc_grouped(a, w, c, tile_expert, used) -> None:
         _p(used), _p(fault_word(a.device)), _stream()), "gemm_tc_grouped")
 
 
-def moe_combine(rows, place, top: int, y, wts=None) -> None:
+def moe_combine(rows, place, top: int, y, wts=None, identity=None) -> None:
     """y[t] = the sum of the token's ``top`` rows of ``rows`` (float32), in their order, each
     times its weight when ``wts`` is given; ``place`` None: the rows are in the pairs' own
-    order."""
+    order.  ``identity`` (``(ids, experts, weights, x)``): a pair whose id is ``experts`` or more has
+    no row of its own and adds its weight times the token's row of ``x``."""
     _need(rows, "rows", torch.float32, 2); _need(y, "y", torch.float32, 2)
     if place is not None:
         _need(place, "place", torch.int32)
@@ -957,21 +1113,33 @@ def moe_combine(rows, place, top: int, y, wts=None) -> None:
     if (rows.shape[1] != H or (place is not None and place.numel() != T * top)
             or rows.shape[0] < T * top or not y.is_contiguous()):
         raise KernelError("moe_combine: sizes do not fit")
+    ids = id_wts = x = None
+    experts = ldx = x_dt = 0
+    if identity is not None:
+        ids, experts, id_wts, x = identity
+        _need(ids, "ids", torch.int32); _need(id_wts, "weights", torch.float32); _need(x, "x", dim=2)
+        if (ids.numel() != T * top or id_wts.numel() != T * top or tuple(x.shape) != (T, H)
+                or not ids.is_contiguous() or not id_wts.is_contiguous()):
+            raise KernelError("moe_combine: the identities' sizes do not fit")
+        ldx, x_dt = _rows(x, "x"), _dt(x)
     _check(lib().cretif_moe_combine(_p(rows), _rows(rows, "rows"), _p(place), top, _p(wts), _p(y),
-                                    T, H, _stream()), "moe_combine")
+                                    T, H, _p(ids), int(experts), _p(id_wts), _p(x), x_dt, ldx,
+                                    _stream()), "moe_combine")
 
 
 # ------------------------------------------------------------------ attention
 def attn_simt(q, out, kc, vc, table, tok_pos, tok_seq, seq_slot, nh: int, nkv: int, hd: int,
               scale: float, window: int, block_tokens: int, sink=None, vd: int = 0, bias=None,
-              bias_edges=None, slope=None) -> None:
+              bias_edges=None, slope=None, pool=None) -> None:
     """``window`` > 0: a sliding window of that many keys; < 0: chunks of ``-window`` positions
     counted from 0, a query sees the keys of its own chunk; 0: every earlier key.  ``slope``
     (float32 [heads], optional): the key n positions back has ``slope[h] * n`` taken off its
     scaled score.  ``sink`` (float32 [heads], optional): exp(sink_h) joins head h's softmax denominator
     without a key or a value.  ``vd``: size of a value head when it is not ``hd``.  ``bias``
     (float32 [rows, heads]) with ``bias_edges`` (int32 [rows], ascending from 0): the key n
-    positions back adds ``bias[r, h]`` to its scaled score, r the last row with edge <= n."""
+    positions back adds ``bias[r, h]`` to its scaled score, r the last row with edge <= n.  ``pool``
+    (a PoolView; with a sliding window): the entries whose last token lies ``window`` or more
+    positions back join the softmax, without bias or slope."""
     _need(q, "q", dim=2); _need(out, "out", q.dtype, 2)
     _need(kc, "k cache", q.dtype, 4); _need(vc, "v cache", q.dtype, 4)
     T = q.shape[0]
@@ -1001,11 +1169,18 @@ def attn_simt(q, out, kc, vc, table, tok_pos, tok_seq, seq_slot, nh: int, nkv: i
         _need(slope, "slope", torch.float32, 1)
         if slope.numel() != nh or not slope.is_contiguous():
             raise KernelError("attention: the slope has one number per query head")
-    _check(lib().cretif_attn_simt(
+    _need_window_pool(pool, kc, vc, window)
+    _check(lib().cretif_attn_simt_pooled(
         _p(q), _rows(q, "q"), _p(out), _rows(out, "out"), _dt(q), _p(kc), _p(vc), _p(table),
         table.stride(0), _p(tok_pos), _p(tok_seq), _p(seq_slot), nh, nkv, hd,
         ctypes.c_float(scale), window, block_tokens, T, _p(sink), vd, _p(bias), _p(bias_edges),
-        rows, _p(slope), _stream()), "attn_simt")
+        rows, _p(slope), *_pool_args(pool), _stream()), "attn_simt")
+
+
+def _need_window_pool(pool, kc, vc, window: int) -> None:
+    if pool is not None and window <= 0:
+        raise KernelError("attention: pooled entries need a sliding window")
+    _need_pool(pool, kc, vc)
 
 
 # ------------------------------------------------------------------ sampling
@@ -1175,8 +1350,9 @@ def decode_plan(B: int, nkv: int, max_context: int, device, hd: int = 64):
 def attn_decode(q, out, kc, vc, table, tok_pos, tok_seq, seq_slot, nh: int, nkv: int, hd: int,
                 scale: float, window: int, block_tokens: int, n_splits: int, fault,
                 cluster: bool = False, sink=None, bias_near=None, bias_far=None,
-                head_groups: int = 1, bias_slope=None) -> None:
-    """``bias_slope`` (float32 [heads], times log2 e; tensor-core kernel only, not with the
+                head_groups: int = 1, bias_slope=None, pool=None) -> None:
+    """``pool`` (a PoolView; tensor-core kernel only): as in ``attn_simt``.
+    ``bias_slope`` (float32 [heads], times log2 e; tensor-core kernel only, not with the
     table): the key n positions back has n times it taken off its scaled score.
     ``head_groups`` = G > 1 (tensor-core kernel only): more than eight query heads on a
     key/value head in ONE launch; the rows of ``q``, ``out``, ``tok_pos`` and ``tok_seq`` are
@@ -1212,30 +1388,34 @@ def attn_decode(q, out, kc, vc, table, tok_pos, tok_seq, seq_slot, nh: int, nkv:
     if (tuple(kc.shape[1:]) != (nkv, block_tokens, hd) or not kc.is_contiguous()
             or not vc.is_contiguous()):
         raise KernelError("attn_decode: cache must be contiguous [blocks, kv_heads, 64, head_dim]")
+    _need_window_pool(pool, kc, vc, window)
+    if pool is not None and (hd > 128 or _decode_simt_only):
+        raise KernelError("attn_decode: pooled entries need head_dim <= 128")
     if n_splits > 64:
         raise KernelError("attn_decode: at most 64 ranges per (sequence, kv head)")
     if cluster:
         if hd > 128 or _decode_simt_only or n_splits > CLUSTER_MAX_RANGES:
             raise KernelError("attn_decode: the cluster merge takes head sizes up to 128 and at "
                               f"most {CLUSTER_MAX_RANGES} ranges")
-        _check(lib().cretif_attn_decode_mma_bias(
+        _check(lib().cretif_attn_decode_mma_pooled(
             _p(q), _rows(q, "q"), _p(out), _rows(out, "out"), _p(kc), _p(vc),
             ctypes.c_longlong(kc.shape[0]), _p(table), table.stride(0), _p(tok_pos), _p(tok_seq),
             _p(seq_slot), nh, nkv, hd, ctypes.c_float(scale), window, block_tokens, B, n_splits,
             None, None, None, _p(sink), _p(bias_near), _p(bias_far), n_far, head_groups,
-            _p(bias_slope), _p(fault), _stream()),
+            _p(bias_slope), *_pool_args(pool, True), _p(fault), _stream()),
             "attn_decode_mma")
         return
     part_o = torch.empty((B, nh, n_splits, hd), dtype=torch.float32, device=q.device)
     part_ml = torch.empty((B, nh, n_splits, 2), dtype=torch.float32, device=q.device)
     counters = _decode_counters(q.device, B * nkv)
     if hd <= 128 and not _decode_simt_only:
-        _check(lib().cretif_attn_decode_mma_bias(
+        _check(lib().cretif_attn_decode_mma_pooled(
             _p(q), _rows(q, "q"), _p(out), _rows(out, "out"), _p(kc), _p(vc),
             ctypes.c_longlong(kc.shape[0]), _p(table), table.stride(0), _p(tok_pos), _p(tok_seq),
             _p(seq_slot), nh, nkv, hd, ctypes.c_float(scale), window, block_tokens, B, n_splits,
             _p(part_o), _p(part_ml), _p(counters), _p(sink), _p(bias_near), _p(bias_far), n_far,
-            head_groups, _p(bias_slope), _p(fault), _stream()), "attn_decode_mma")
+            head_groups, _p(bias_slope), *_pool_args(pool, True), _p(fault), _stream()),
+            "attn_decode_mma")
         return
     _check(lib().cretif_attn_decode(
         _p(q), _rows(q, "q"), _p(out), _rows(out, "out"), _p(kc), _p(vc), _p(table),
@@ -1309,8 +1489,8 @@ def set_dependent_launch(on: bool) -> bool:
 
 
 def fused_norm_linear(h, norm_w, eps: float, w, out, rows=None, accumulate: bool = False,
-                      unary: Optional[str] = None) -> None:
-    """out (+)= bf16(rmsnorm(h[rows])) · wᵀ in one kernel (decode-sized row counts); ``unary``
+                      unary: Optional[str] = None, alpha: float = 1.0) -> None:
+    """out (+)= alpha · bf16(rmsnorm(h[rows])) · wᵀ in one kernel (decode-sized row counts); ``unary``
     (a key of ACTIVATIONS; stores only) is applied to the 32-bit sums."""
     _need(h, "h", torch.float32, 2); _need(norm_w, "norm weight", torch.float32, 1)
     _need(w, "w", torch.bfloat16, 2); _need(out, "out", dim=2)
@@ -1321,7 +1501,7 @@ def fused_norm_linear(h, norm_w, eps: float, w, out, rows=None, accumulate: bool
         raise KernelError("fused_norm_linear: shapes do not fit")
     _check(lib().cretif_fused_linear(None, 0, _p(h), _p(norm_w), _p(rows), ctypes.c_float(eps),
                                      _p(w), _rows(w, "w"), _p(out), _dt(out), _rows(out, "out"),
-                                     int(accumulate), ctypes.c_float(1.0),
+                                     int(accumulate), ctypes.c_float(alpha),
                                      0 if unary is None else 1 + ACTIVATIONS[unary], M, N, K,
                                      _p(fault_word(h.device)), _stream()), "fused_norm_linear")
 
@@ -1461,12 +1641,14 @@ def attn_prefill_supported(hd: int, block_tokens: int) -> bool:
 
 def attn_prefill(qkv, out, kc, vc, table, cu_seqlens, seq_start, seq_slot, nh: int, nkv: int,
                  hd: int, scale: float, window: int, block_tokens: int, B: int, max_new: int,
-                 fault, sink=None, bias_near=None, bias_far=None, bias_slope=None) -> None:
+                 fault, sink=None, bias_near=None, bias_far=None, bias_slope=None,
+                 pool=None) -> None:
     """Causal attention of whole prompts; ``qkv`` rows start with the query heads.  ``sink``
     (float32 [heads], optional): exp(sink_h) joins head h's softmax denominator.  ``bias_near``
     [heads, n_far] with ``bias_far`` [heads] (float32, times log2 e): what the key n positions
     back adds to its scaled score, for n < n_far and for every n beyond.  ``bias_slope`` (float32
-    [heads], times log2 e; not with the table): n times it is taken off that score instead."""
+    [heads], times log2 e; not with the table): n times it is taken off that score instead.
+    ``pool`` (a PoolView; without bias and slope): as in ``attn_simt``."""
     n_far = 0
     if bias_near is not None:
         _need(bias_near, "bias_near", torch.float32, 2); _need(bias_far, "bias_far", torch.float32, 1)
@@ -1489,9 +1671,10 @@ def attn_prefill(qkv, out, kc, vc, table, cu_seqlens, seq_start, seq_slot, nh: i
     if (tuple(kc.shape[1:]) != (nkv, block_tokens, hd) or not kc.is_contiguous()
             or not vc.is_contiguous()):
         raise KernelError("attn_prefill: cache must be contiguous [blocks, kv_heads, 64, head_dim]")
-    _check(lib().cretif_attn_prefill_tc_bias(
+    _need_window_pool(pool, kc, vc, window)
+    _check(lib().cretif_attn_prefill_tc_pooled(
         _p(qkv), _rows(qkv, "qkv"), qkv.shape[0], _p(out), _rows(out, "out"), _p(kc), _p(vc),
         ctypes.c_longlong(kc.shape[0]), _p(table), table.stride(0), _p(cu_seqlens), _p(seq_start),
         _p(seq_slot), nh, nkv, hd, ctypes.c_float(scale), window, block_tokens, B, max_new,
-        _p(sink), _p(bias_near), _p(bias_far), n_far, _p(bias_slope), _p(fault), _stream()),
-        "attn_prefill_tc")
+        _p(sink), _p(bias_near), _p(bias_far), n_far, _p(bias_slope), *_pool_args(pool, True),
+        _p(fault), _stream()), "attn_prefill_tc")

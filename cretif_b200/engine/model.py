@@ -140,22 +140,32 @@ class Model:
     def cache_requests(self) -> Dict[Tuple, Any]:
         """cache id → what its part keeps between steps.  A cache id is (index of the schedule
         entry, index of the branch in its layer) for the branch's part and (entry, branch,
-        "shift") for a shift in front of it.  A part may ask for keys and values, for a state of
+        "shift") for a shift in front of it; a mixer made of several (``sub_mixers``) keeps one for
+        each, (entry, branch, its name).  A part may ask for keys and values, for a state of
         fixed size, or for both (a tuple).  An entry that borrows (``ScheduleEntry.cache``) reads
         the owner's keys and values and asks for none; states are always an entry's own."""
         out = {}
         for i, entry in enumerate(self.spec.schedule):
             for k, br in enumerate(self.layers[entry.layer].branches):
-                if hasattr(br.part, "cache_request"):
-                    reqs = br.part.cache_request()
+                for cid, part in self._keepers(i, k, br.part):
+                    if not hasattr(part, "cache_request"):
+                        continue
+                    reqs = part.cache_request()
                     reqs = list(reqs) if isinstance(reqs, (tuple, list)) else [reqs]
                     reqs = [r for r in reqs if r is not None
                             and not (entry.cache is not None and isinstance(r, KVRequest))]
                     if reqs:
-                        out[(i, k)] = reqs[0] if len(reqs) == 1 else tuple(reqs)
+                        out[cid] = reqs[0] if len(reqs) == 1 else tuple(reqs)
                 if br.shift is not None:
                     out[(i, k, "shift")] = br.shift.cache_request()
         return out
+
+    @staticmethod
+    def _keepers(i: int, k: int, part):
+        """(cache id, part) of everything that keeps something in branch k of entry i."""
+        if hasattr(part, "sub_mixers"):
+            return [((i, k, name), sub) for name, sub in part.sub_mixers()]
+        return [((i, k), part)]
 
     def layer_caches(self, i: int, cache) -> List[Optional[LayerCache]]:
         """What each branch of schedule entry ``i`` is handed: its own keys/values or those of
@@ -173,12 +183,19 @@ class Model:
                 theirs = [j for j, b in enumerate(
                     self.layers[self.spec.schedule[owner].layer].branches) if b.role == "mixer"]
                 cid = (owner, theirs[mine.index(k)])
-            kv = cache.kv_view(cid) if cache.has_kv(cid) else None
-            state = cache.state_view((i, k)) if cache.has_state((i, k)) else None
             shift = cache.state_view((i, k, "shift")) if cache.has_state((i, k, "shift")) else None
-            views.append(None if kv is None and state is None and shift is None
-                         else LayerCache(kv=kv, state=state, writes=entry.cache is None,
-                                         shift_state=shift))
+
+            def view(tail=(), shift=None):
+                kv = cache.kv_view(cid + tail) if cache.has_kv(cid + tail) else None
+                own = (i, k) + tail
+                state = cache.state_view(own) if cache.has_state(own) else None
+                return None if kv is None and state is None and shift is None else LayerCache(
+                    kv=kv, state=state, writes=entry.cache is None, shift_state=shift)
+            if hasattr(br.part, "sub_mixers"):
+                views.append(LayerCache(writes=entry.cache is None, shift_state=shift, subs={
+                    name: view((name,)) for name, _ in br.part.sub_mixers()}))
+            else:
+                views.append(view(shift=shift))
         return views
 
     # -- one step ------------------------------------------------------------------

@@ -32,6 +32,18 @@ its own run of ``chunk`` positions, runs counted from position 0 of the sequence
 for query i, with ``slope_h = 2^(-x (h + 1) / heads)``.  Both belong to the family whose
 projections are handled head by head, which also serves a layer without key and value tensors of
 its own (``own_kv: False``).
+
+``pool`` (P tokens; with a sliding ``window``) keeps, beside the window, one key and value for every
+block of P tokens: the means of the block's rows as the cache holds them.  A query sees the blocks
+that lie wholly before its window, in the same softmax as the window's tokens; tokens that have left
+the window and whose block has not left it yet are not seen.  ``qk_norm`` together with biases, a
+position encoding, values of another size or ``pool`` is one kernel between the input product and
+the attention as well, and there ``out_scale`` (a factor on the layer's output) is applied to the
+values as they are stored.
+
+A mixer that can stand beside another one on the same input (parts/parallel.py) offers ``w_in``,
+``w_out`` and ``mix(proj, ctx, cache, out)``: what lies between its input and its output product.
+The head-by-head family does.
 """
 from __future__ import annotations
 
@@ -91,7 +103,7 @@ FAST_BIAS_MAX_DISTANCES = 4096
 
 
 def run_attention(q, o, ctx, kv, nh, nkv, hd, scale, window, dtype, sink=None, vd=0, bias=None,
-                  bias_edges=None, bias_dense=None, slope=None, slope_log2e=None):
+                  bias_edges=None, bias_dense=None, slope=None, slope_log2e=None, pool=None):
     """Causal (windowed) attention of the step's queries ``q`` [T, nh·hd] over the cache view
     ``kv`` into ``o``, with the kernel that fits the step: the decode kernels when every
     sequence brings one token, the prompt kernel otherwise, the plain kernel for float32 and
@@ -101,14 +113,19 @@ def run_attention(q, o, ctx, kv, nh, nkv, hd, scale, window, dtype, sink=None, v
     (near [heads, n_far], far [heads]), times log2 e, as the tensor-core kernels do.  ``window``
     below zero stands for chunks of ``-window`` positions.  ``slope`` [heads]: a multiple of the
     distance taken off the scores; the plain kernel takes it as it is, the fast kernels work in
-    powers of two and take ``slope_log2e``, the same numbers times log2 e."""
+    powers of two and take ``slope_log2e``, the same numbers times log2 e.  ``pool`` (a PoolView):
+    the entries per block of tokens that are seen beside the window."""
     vd = vd or hd
     fast = (not _force_plain and dtype == torch.bfloat16 and (sink is None or hd <= 128)
             and vd == hd and not (bias is not None and slope is not None)
             and (bias is None or (bias_dense is not None and hd <= 128))
-            and (slope is None or (slope_log2e is not None and hd <= 128)))
+            and (slope is None or (slope_log2e is not None and hd <= 128))
+            and (pool is None or (hd <= 128 and bias is None and slope is None)))
     near, far = bias_dense if (bias is not None and bias_dense is not None) else (None, None)
     tilt = slope_log2e if slope is not None else None
+    # what a decode step's keys are shared out by: with pooled entries, the keys it really reads
+    context = ctx.max_context if pool is None else min(
+        ctx.max_context, window + 64 + ctx.max_context // pool.pool)
     if fast:
         if ctx.is_decode and ops.attn_decode_supported(hd, kv.block_tokens, min(nh // nkv, 8)) \
                 and (nh // nkv <= 8 or nkv == 1):
@@ -124,34 +141,35 @@ def run_attention(q, o, ctx, kv, nh, nkv, hd, scale, window, dtype, sink=None, v
                     ctx.extras[key] = tuple(t.repeat_interleave(G).contiguous()
                                             for t in (ctx.tok_pos, ctx.tok_seq))
                 pos_g, seq_g = ctx.extras[key]
-                splits, cluster = ops.decode_plan(ctx.B * G, 1, ctx.max_context, q.device, hd)
+                splits, cluster = ops.decode_plan(ctx.B * G, 1, context, q.device, hd)
                 ops.attn_decode(q.view(ctx.B * G, 8 * hd), o.view(ctx.B * G, 8 * hd), kv.k, kv.v,
                                 kv.table, pos_g, seq_g, ctx.seq_slot, 8, 1, hd, scale, window,
                                 kv.block_tokens, splits, ctx.fault, cluster, sink=sink,
-                                bias_near=near, bias_far=far, head_groups=G, bias_slope=tilt)
+                                bias_near=near, bias_far=far, head_groups=G, bias_slope=tilt,
+                                pool=pool)
                 return
             # ... else eight at a time
             step = nh if nh // nkv <= 8 else 8
             for h0 in range(0, nh, step):
                 n = min(step, nh - h0)
-                splits, cluster = ops.decode_plan(ctx.B, nkv, ctx.max_context, q.device, hd)
+                splits, cluster = ops.decode_plan(ctx.B, nkv, context, q.device, hd)
                 ops.attn_decode(q[:, h0 * hd:], o[:, h0 * hd:], kv.k, kv.v, kv.table,
                                 ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, n, nkv, hd, scale,
                                 window, kv.block_tokens, splits, ctx.fault, cluster,
                                 sink=None if sink is None else sink[h0:h0 + n],
                                 bias_near=None if near is None else near[h0:h0 + n],
                                 bias_far=None if far is None else far[h0:h0 + n],
-                                bias_slope=None if tilt is None else tilt[h0:h0 + n])
+                                bias_slope=None if tilt is None else tilt[h0:h0 + n], pool=pool)
             return
         if not ctx.is_decode and ops.attn_prefill_supported(hd, kv.block_tokens):
             ops.attn_prefill(q, o, kv.k, kv.v, kv.table, ctx.cu_seqlens, ctx.seq_start,
                              ctx.seq_slot, nh, nkv, hd, scale, window, kv.block_tokens, ctx.B,
                              ctx.max_new, ctx.fault, sink=sink, bias_near=near, bias_far=far,
-                             bias_slope=tilt)
+                             bias_slope=tilt, pool=pool)
             return
     ops.attn_simt(q, o, kv.k, kv.v, kv.table, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot,
                   nh, nkv, hd, scale, window, kv.block_tokens, sink=sink, vd=vd, bias=bias,
-                  bias_edges=bias_edges, slope=slope)
+                  bias_edges=bias_edges, slope=slope, pool=pool)
 
 
 @register_part("mixer", "attention")
@@ -161,7 +179,8 @@ class Attention(Part):
     (tensor names of q, k, v, o relative to the layer's prefix).  Optional: ``qk_norm``
     (``{"eps", "q": name, "k": name}``: RMS norm over the whole q and k projections),
     ``values`` (``"keys"``: no value projection, the un-normed keys are the values; needs
-    ``qk_norm`` or no position encoding), ``sink`` (name of a [heads] tensor)."""
+    ``qk_norm`` or no position encoding), ``sink`` (name of a [heads] tensor); ``pool``,
+    ``out_scale`` and the families' options as the module describes them."""
 
     graph_safe = True
 
@@ -194,9 +213,9 @@ class Attention(Part):
         if self.values_are_keys and self.qk_norm is None:
             raise ValueError("attention: values taken from the keys need qk_norm (the kernel "
                              "that norms the keys stores both)")
-        if self.qk_norm is not None and (params.get("position") or {}).get("kind", "none") != "none":
-            raise ValueError("attention: qk_norm over the whole projection is built without a "
-                             "position encoding only")
+        has_position = (params.get("position") or {}).get("kind", "none") != "none"
+        if self.values_are_keys and has_position:
+            raise ValueError("attention: keys as values are built without a position encoding only")
         self.sink = None
         # -- the convolved family
         self.vd = int(params.get("value_dim") or self.hd)
@@ -212,9 +231,23 @@ class Attention(Part):
         # the family that norms head by head without a convolution
         self.slope_spec = params.get("distance_slope")
         self.slope = self.slope_log2e = None
+        # pooled blocks beside a window, a factor on the output
+        self.pool = int(params.get("pool") or 0)
+        self.out_scale = float(params.get("out_scale", 1.0))
+        if self.pool < 0 or (self.pool and not (self.window > 0 and self.own_kv
+                                                and self.conv is None
+                                                and self.slope_spec is None
+                                                and self.distance_bias is None)):
+            raise ValueError("attention: pooled blocks need a sliding window, keys of the layer's own "
+                             "and no convolution, bias or slope by distance")
         self.headwise = self.conv is None and bool(
             self.bias_names or self.head_gate or self.head_norm or self.vd != self.hd
-            or self.chunk or self.slope_spec or not self.own_kv)
+            or self.chunk or self.slope_spec or not self.own_kv or self.pool
+            or self.out_scale != 1.0 or (self.qk_norm is not None and has_position))
+        # norms over the whole projections in the kernel that stores keys and values
+        self.whole_norm = self.headwise and self.qk_norm is not None
+        if self.out_scale != 1.0 and not self.whole_norm:
+            raise ValueError("attention: out_scale is built together with qk_norm")
         extras = [k for k in ("query_gain", "distance_bias") if params.get(k)] \
             + ([] if self.own_kv or self.headwise else ["own_kv"]) \
             + ([] if self.headwise else
@@ -226,9 +259,11 @@ class Attention(Part):
         if self.conv is not None and (self.bias_names or self.head_gate):
             raise ValueError("attention: bias and head_gate are built without a convolution")
         if self.headwise:
-            if self.qk_norm is not None or self.values_are_keys:
-                raise ValueError("attention: projections normed head by head take no norm over "
-                                 "the whole projection and no keys as values")
+            if self.values_are_keys or (self.qk_norm is not None
+                                        and (self.head_norm is not None or not self.own_kv)):
+                raise ValueError("attention: this family takes no keys as values, and a norm over the "
+                                 "whole projections only instead of one by head and with keys of the "
+                                 "layer's own")
             if self.head_norm is not None and not (self.head_norm.get("q")
                                                    and self.head_norm.get("k")):
                 raise ValueError("attention: head_norm without a convolution names its two "
@@ -353,7 +388,8 @@ class Attention(Part):
         # (a chunked mask keeps every block: another layer may read these keys with a mask of
         # its own)
         kv = KVRequest(self.nkv, self.hd, self.window,
-                       value_dim=0 if self.vd == self.hd else self.vd) if self.own_kv else None
+                       value_dim=0 if self.vd == self.hd else self.vd,
+                       pool=self.pool) if self.own_kv else None
         if self.conv is None or self.taps == 1:
             return kv
         # the last taps - 1 projected rows of every convolved channel
@@ -388,11 +424,30 @@ class Attention(Part):
             return None
         return linear_few(o, self.w_o, out_dtype=torch.float32)
 
-    def _forward_headwise(self, x, ctx, cache, into=None, alpha: float = 1.0, proj=None):
-        """One product for q|k|v|gates with 32-bit sums (``proj``, where the caller made it
-        already), one kernel for bias, head norms, rotation and the cache write, attention, the
-        per-head gate, output product."""
-        from .linear import linear_few, linear_scaled_add
+    # -- what a mixer offers that shares its products with another one -----------------
+    @property
+    def w_in(self):
+        return self.w_qkv
+
+    @w_in.setter
+    def w_in(self, w):
+        self.w_qkv = w
+
+    @property
+    def w_out(self):
+        return self.w_o
+
+    @w_out.setter
+    def w_out(self, w):
+        self.w_o = w
+
+    @property
+    def can_mix(self) -> bool:
+        return self.headwise
+
+    def mix(self, proj, ctx, cache, out) -> None:
+        """From the input product's rows (32-bit sums) to the output product's: bias, norms, rotation
+        and the cache write in one kernel, pooled entries, attention, the per-head gate."""
         kv = cache.kv
         rot = getattr(self.position, "rotary_table", None)
         if rot is not None:
@@ -403,23 +458,41 @@ class Attention(Part):
         else:
             raise ValueError("attention: projections normed head by head take a rotary position "
                              "encoding or none")
-        proj = linear_few(x, self.w_qkv, out_dtype=torch.float32) if proj is None else proj
-        q = torch.empty((ctx.T, self.q_dim), dtype=self.dtype, device=proj.device)
         if kv is None:
             raise ValueError("attention: this layer reads another entry's keys and values, but "
                              "the schedule gives it none")
+        q = torch.empty((ctx.T, self.q_dim), dtype=self.dtype, device=proj.device)
         own = self.own_kv
-        ops.headnorm_rope_kv_append(
-            proj, self.in_bias, self.q_head_w, self.k_head_w,
-            float(self.head_norm["eps"]) if self.head_norm else 0.0, cos, sin, pairing, rot_dim,
-            ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, self.nh, self.nkv if own else 0, self.hd,
-            self.vd, q, table=kv.table, kc=kv.k, vc=kv.v, block_tokens=kv.block_tokens,
-            write_cache=cache.writes and own, fault=ctx.fault)
-        o = torch.empty((ctx.T, self.o_dim), dtype=self.dtype, device=proj.device)
-        self.attend(q, o, ctx, kv)
+        writes = cache.writes and own
+        pool = kv.pool if self.pool else None
+        common = dict(table=kv.table, kc=kv.k, vc=kv.v, block_tokens=kv.block_tokens,
+                      write_cache=writes, fault=ctx.fault)
+        if self.whole_norm:
+            ops.projnorm_rope_kv_append(
+                proj, self.in_bias, self.q_norm_w, self.k_norm_w, self.qk_eps, cos, sin, pairing,
+                rot_dim, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, self.nh, self.nkv, self.hd, self.vd,
+                q, v_scale=self.out_scale, pool=pool if ctx.is_decode else None, **common)
+        else:
+            ops.headnorm_rope_kv_append(
+                proj, self.in_bias, self.q_head_w, self.k_head_w,
+                float(self.head_norm["eps"]) if self.head_norm else 0.0, cos, sin, pairing, rot_dim,
+                ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, self.nh, self.nkv if own else 0, self.hd,
+                self.vd, q, **common)
+        if pool is not None and writes and not (self.whole_norm and ctx.is_decode):
+            ops.pool_kv(kv.k, kv.v, kv.table, pool, ctx.cu_seqlens, ctx.seq_start, ctx.seq_slot,
+                        self.nkv, self.hd, self.vd, kv.block_tokens, ctx.B, ctx.max_new, ctx.fault)
+        self.attend(q, out, ctx, kv)
         if self.head_gate:
-            ops.gate_heads(o, proj[:, self.q_dim + (self.kv_dim + self.v_dim if own else 0):],
+            ops.gate_heads(out, proj[:, self.q_dim + (self.kv_dim + self.v_dim if own else 0):],
                            self.nh, self.vd)
+
+    def _forward_headwise(self, x, ctx, cache, into=None, alpha: float = 1.0, proj=None):
+        """One product for q|k|v|gates with 32-bit sums (``proj``, where the caller made it
+        already), ``mix``, output product."""
+        from .linear import linear_few, linear_scaled_add
+        proj = linear_few(x, self.w_qkv, out_dtype=torch.float32) if proj is None else proj
+        o = torch.empty((ctx.T, self.o_dim), dtype=self.dtype, device=proj.device)
+        self.mix(proj, ctx, cache, o)
         if into is not None:
             linear_scaled_add(o, self.w_o, into, alpha)
             return None
@@ -539,7 +612,7 @@ class Attention(Part):
         run_attention(q, o, ctx, kv, self.nh, self.nkv, self.hd, self.scale, self.mask,
                       self.dtype, self.sink, vd=self.vd, bias=self.bias,
                       bias_edges=self.bias_edges, bias_dense=self.bias_dense, slope=self.slope,
-                      slope_log2e=self.slope_log2e)
+                      slope_log2e=self.slope_log2e, pool=kv.pool if self.pool else None)
 
     def weight_bytes(self):
         return (self.w_qkv.numel() + self.w_o.numel()) * self.w_qkv.element_size()

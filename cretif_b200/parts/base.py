@@ -101,6 +101,7 @@ class LayerCache:
     state: Optional[torch.Tensor] = None   # [max_slots, *shape]
     writes: bool = True               # False: the visit borrows another visit's keys and values
     shift_state: Optional[torch.Tensor] = None   # [max_slots, H]: the branch's shift, if any
+    subs: Dict[str, "LayerCache"] = field(default_factory=dict)   # of a mixer made of several
 
 
 class Part:

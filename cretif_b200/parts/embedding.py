@@ -23,7 +23,8 @@ class TokenEmbedding(Part):
     Optional ``positions`` (``{"name", "rows"}``): a learned vector per position, a table of
     ``rows`` positions, added to the token's row as it is (32-bit sum).  Optional ``norm``
     (``{"name", "eps", "offset"}``): an RMS norm of the gathered row, its weight stored as the
-    factor minus ``offset``, in 32-bit, before the first layer reads the stream."""
+    factor minus ``offset``, in 32-bit, before the first layer reads the stream.  Optional ``scale``:
+    a factor on the token's row (32-bit)."""
 
     graph_safe = True
 
@@ -57,7 +58,8 @@ class TokenEmbedding(Part):
     def forward(self, ids, ctx):
         h = torch.empty((ids.numel(), self.hidden_size), dtype=torch.float32, device=ids.device)
         ops.embed_rows(self.table, ids, h, ctx.fault, positions=self.positions,
-                       tok_pos=ctx.tok_pos if self.positions is not None else None)
+                       tok_pos=ctx.tok_pos if self.positions is not None else None,
+                       scale=float(self.params.get("scale", 1.0)))
         if self.norm_weight is not None:
             ops.rmsnorm_rows(h, self.norm_weight, self.norm_eps)
         return h
@@ -71,7 +73,7 @@ class TokenEmbedding(Part):
 @register_part("head", "linear_head")
 class LinearHead(Part):
     """params: ``tied`` (share the embedding matrix), ``name``, ``vocab_size``; optional
-    ``softcap`` c: the logits leave as ``c * tanh(logits / c)``."""
+    ``scale``: a factor on the logits; ``softcap`` c: they leave as ``c * tanh(logits / c)``."""
 
     graph_safe = True
 
@@ -87,7 +89,14 @@ class LinearHead(Part):
     def tie(self, embedding: TokenEmbedding) -> None:
         self.weight = embedding.table
 
-    def _capped(self, logits):
+    @property
+    def scale(self) -> float:
+        return float(self.params.get("scale", 1.0))
+
+    def _capped(self, logits, scaled: bool = False):
+        """``scaled``: the product has applied the factor already."""
+        if not scaled and self.scale != 1.0 and logits.numel():
+            ops.scale_in_place(logits, self.scale)
         cap = self.params.get("softcap")
         if cap and logits.numel():
             ops.softcap(logits, float(cap))
@@ -108,8 +117,8 @@ class LinearHead(Part):
             return None
         logits = torch.empty((R, self.weight.shape[0]), dtype=torch.float32, device=h.device)
         norm_w, eps = rms()
-        ops.fused_norm_linear(h, norm_w, eps, self.weight, logits, rows=rows)
-        return self._capped(logits)
+        ops.fused_norm_linear(h, norm_w, eps, self.weight, logits, rows=rows, alpha=self.scale)
+        return self._capped(logits, scaled=True)
 
     def weight_bytes(self):
         if self.params.get("tied") or self.weight is None:

@@ -11,7 +11,11 @@ Options: ``gated: False`` makes an expert ``down(act(up x))`` with ``activation`
 kernels' unary activations; ``groups`` (``{"count", "keep"}``) lets the experts form ``count``
 equal groups of neighbours, scores a group by the sum of its two largest scores and allows only
 experts of the ``keep`` best groups; ``sum_eps`` is added to the sum that ``renormalize`` divides
-by; ``shared`` (``{"intermediate_size", "names"}``) is one more expert of the same form that every
+by; ``scores: "softmax"`` takes the softmax over all router outputs instead of the logistic
+function; ``correction`` names a tensor with a number per router output that is added to the scores
+for the choice alone; a group's score is then that of its choice scores, and ``groups`` may say
+``"score": "best"`` for the largest instead of the sum of two; ``identities`` appends that many router
+outputs that are no experts: their output is the input itself; ``shared`` (``{"intermediate_size", "names"}``) is one more expert of the same form that every
 token uses with weight one.
 
 The step's (token, choice) pairs are sorted by expert on the device and each expert's rows
@@ -53,13 +57,20 @@ class RoutedExperts(Part):
     """params: ``num_experts``, ``top``, ``intermediate_size`` (of one expert), ``weight_on``
     ("input" | "output"), ``renormalize`` (default False), ``names``: ``router`` and the
     patterns ``gate``, ``up``, ``down`` with ``{e}`` for the expert's number.  Optional:
-    ``gated`` (default True), ``activation``, ``groups``, ``sum_eps``, ``shared``."""
+    ``gated`` (default True), ``activation``, ``groups``, ``sum_eps``, ``scores`` ("sigmoid" |
+    "softmax"), ``correction``, ``identities``, ``shared``."""
 
     graph_safe = True
 
     def __init__(self, params, hidden_size, dtype, device):
         super().__init__(params, hidden_size, dtype, device)
         self.E = int(params["num_experts"])
+        self.identities = int(params.get("identities") or 0)
+        self.outputs = self.E + self.identities              # of the router
+        self.softmax = params.get("scores", "sigmoid") == "softmax"
+        if params.get("scores", "sigmoid") not in ("sigmoid", "softmax") or self.identities < 0:
+            raise ValueError("routed_experts: scores must be 'sigmoid' or 'softmax' and identities "
+                             "not below zero")
         self.top = int(params["top"])
         self.inter = int(params["intermediate_size"])
         self.weight_on = params.get("weight_on", "output")
@@ -67,9 +78,11 @@ class RoutedExperts(Part):
         if self.weight_on not in ("input", "output"):
             raise ValueError(f"routed_experts: weight_on must be 'input' or 'output', got "
                              f"{self.weight_on!r}")
-        if not 0 < self.top <= self.E or self.E > 256:
-            raise ValueError(f"routed_experts: {self.top} of {self.E} experts (at most 256) "
+        if self.E <= 0 or not 0 < self.top <= self.outputs or self.outputs > 256:
+            raise ValueError(f"routed_experts: {self.top} of {self.outputs} experts (at most 256) "
                              "cannot be chosen")
+        if self.identities and self.weight_on == "input":
+            raise ValueError("routed_experts: identities are built with the weight on the output")
         self.gated = bool(params.get("gated", True))
         self.activation = params.get("activation", "silu")
         if self.gated and self.activation != "silu":
@@ -80,9 +93,12 @@ class RoutedExperts(Part):
         groups = params.get("groups") or {}
         self.groups = int(groups.get("count", 0) or 0)
         self.keep = int(groups.get("keep", 0) or 0)
-        if self.groups > 1 and (self.E % self.groups or not 1 <= self.keep <= self.groups
-                                or self.keep * (self.E // self.groups) < self.top):
-            raise ValueError(f"routed_experts: {self.E} experts do not form {self.groups} equal "
+        self.group_best = groups.get("score", "two") == "best"
+        if groups.get("score", "two") not in ("two", "best"):
+            raise ValueError("routed_experts: a group's score is 'two' or 'best'")
+        if self.groups > 1 and (self.outputs % self.groups or not 1 <= self.keep <= self.groups
+                                or self.keep * (self.outputs // self.groups) < self.top):
+            raise ValueError(f"routed_experts: {self.outputs} experts do not form {self.groups} equal "
                              f"groups of which {self.keep} hold {self.top} experts")
         self.sum_eps = float(params.get("sum_eps", 0.0))
         self.shared = None
@@ -96,7 +112,10 @@ class RoutedExperts(Part):
     @classmethod
     def weight_specs(cls, params, hidden_size):
         E, F, n = params["num_experts"], params["intermediate_size"], params["names"]
-        out = {"router": (n["router"], WeightSpec((E, hidden_size), init=(0.0, 0.5)))}
+        outputs = E + int(params.get("identities") or 0)
+        out = {"router": (n["router"], WeightSpec((outputs, hidden_size), init=(0.0, 0.5)))}
+        if params.get("correction"):
+            out["correction"] = (params["correction"], WeightSpec((outputs,), init=(0.0, 0.05)))
         for e in range(E):
             if params.get("gated", True):
                 out[f"gate{e}"] = (n["gate"].format(e=e), WeightSpec((F, hidden_size)))
@@ -116,9 +135,11 @@ class RoutedExperts(Part):
         self.router = self._vector32(tensors["router"])            # 32-bit logits
         # Many tokens: the logits are a matrix product (32-bit sums of exact products) whenever
         # the stored router is exact in the compute type, which a bfloat16 checkpoint's is.
-        self.router_matrix = self._matrix(tensors["router"])
-        if not torch.equal(self.router_matrix.float(), self.router):
+        self.router_matrix = self._stacked([tensors["router"]])
+        if not torch.equal(self.router_matrix[:self.outputs].float(), self.router):
             self.router_matrix = None
+        self.correction = (self._vector32(tensors["correction"]) if "correction" in tensors
+                           else None)
         if self.shared is not None:
             self.shared.load({k[len("shared_"):]: v for k, v in tensors.items()
                               if k.startswith("shared_")})
@@ -148,12 +169,10 @@ class RoutedExperts(Part):
         if self.router_matrix is not None and (T > ROUTE_BY_PRODUCT
                                                or self.dtype == torch.bfloat16):
             from .linear import linear_few
-            logits = linear_few(x, self.router_matrix, out_dtype=torch.float32)
-            ops.moe_topk(logits, self.top, ids, wts, renorm=self.renorm, groups=self.groups,
-                         keep=self.keep, sum_eps=self.sum_eps)
+            logits = linear_few(x, self.router_matrix, out_dtype=torch.float32)[:, :self.outputs]
+            ops.moe_topk(logits, self.top, ids, wts, **self._rule())
         else:
-            ops.moe_route(x, self.router, self.top, ids, wts, renorm=self.renorm,
-                          groups=self.groups, keep=self.keep, sum_eps=self.sum_eps)
+            ops.moe_route(x, self.router, self.top, ids, wts, **self._rule())
         y = torch.empty((T, H), dtype=torch.float32, device=dev)
         if self.gated:
             self._gated_experts(x, ids, wts, y)
@@ -162,6 +181,15 @@ class RoutedExperts(Part):
         if self.shared is not None:
             self.shared.forward(x, ctx, into=y)
         return y
+
+    def _rule(self) -> dict:
+        return dict(renorm=self.renorm, groups=self.groups, keep=self.keep, sum_eps=self.sum_eps,
+                    softmax=self.softmax, group_best=self.group_best, correction=self.correction)
+
+    def _combine(self, rows, place, y, x, ids, wts, scaled: bool):
+        """The choices summed; ``scaled``: the rows carry their weights already."""
+        ops.moe_combine(rows, place, self.top, y, wts=None if scaled else wts,
+                        identity=(ids, self.E, wts, x) if self.identities else None)
 
     def _plain_experts(self, x, ids, wts, y):
         """Experts without a gate: the activation sits in the first product's epilogue."""
@@ -174,7 +202,7 @@ class RoutedExperts(Part):
             rows = torch.empty((P, H), dtype=torch.float32, device=dev)
             ops.moe_gemv(x, self.w_up, act, self.top, mode, 1 if on_input else 0, ids, wts)
             ops.moe_gemv(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, ids, wts)
-            ops.moe_combine(rows, None, self.top, y)
+            self._combine(rows, None, y, x, ids, wts, True)
             return
         if self.dtype == torch.bfloat16 and ops.moe_tc_supported(x, self.w_up, self.w_down,
                                                                  gated=False):
@@ -189,7 +217,7 @@ class RoutedExperts(Part):
             ops.gemm_tc_act_grouped(xs, self.w_up, act, tile_expert, used, self.activation)
             rows = torch.empty((rows_pad, H), dtype=torch.float32, device=dev)
             ops.gemm_tc_grouped(act, self.w_down, rows, tile_expert, used)
-            ops.moe_combine(rows, place, self.top, y, wts=None if on_input else wts)
+            self._combine(rows, place, y, x, ids, wts, on_input)
             return
         tiles = ops.moe_max_tiles(P, self.E)
         idx = torch.empty(self.E + 1 + 2 * P + 2 * tiles, dtype=torch.int32, device=dev)
@@ -204,7 +232,7 @@ class RoutedExperts(Part):
                      tile_expert, tile_row0)
         ops.moe_gemm(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, wts, order,
                      offsets, tile_expert, tile_row0)
-        ops.moe_combine(rows, place, self.top, y)
+        self._combine(rows, place, y, x, ids, wts, True)
 
     def _gated_experts(self, x, ids, wts, y):
         T, H = x.shape
@@ -216,7 +244,7 @@ class RoutedExperts(Part):
             rows = torch.empty((P, H), dtype=torch.float32, device=dev)
             ops.moe_gemv(x, self.w_gu, act, self.top, 0, 1 if on_input else 0, ids, wts)
             ops.moe_gemv(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, ids, wts)
-            ops.moe_combine(rows, None, self.top, y)
+            self._combine(rows, None, y, x, ids, wts, True)
             return
         if self.w_gu_blocks is not None and ops.moe_tc_supported(x, self.w_gu_blocks, self.w_down):
             # many pairs, bfloat16: the tcgen05 product in its grouped mode over rows sorted
@@ -232,7 +260,7 @@ class RoutedExperts(Part):
             ops.gemm_tc_silu_grouped(xs, self.w_gu_blocks, act, tile_expert, used)
             rows = torch.empty((rows_pad, H), dtype=torch.float32, device=dev)
             ops.gemm_tc_grouped(act, self.w_down, rows, tile_expert, used)
-            ops.moe_combine(rows, place, self.top, y, wts=None if on_input else wts)
+            self._combine(rows, place, y, x, ids, wts, on_input)
             return
         tiles = ops.moe_max_tiles(P, self.E)
         idx = torch.empty(self.E + 1 + 2 * P + 2 * tiles, dtype=torch.int32, device=dev)
@@ -247,7 +275,7 @@ class RoutedExperts(Part):
                      tile_expert, tile_row0)
         ops.moe_gemm(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, wts, order,
                      offsets, tile_expert, tile_row0)
-        ops.moe_combine(rows, place, self.top, y)
+        self._combine(rows, place, y, x, ids, wts, True)
 
     def weight_bytes(self):
         # (the blocked copy of gate|up serves the many-pairs path and is not counted twice)

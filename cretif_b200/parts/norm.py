@@ -22,17 +22,22 @@ from .base import Part, register_part
 @register_part("norm", "rmsnorm")
 class RMSNorm(Part):
     """params: ``eps``; ``name`` (tensor name relative to the prefix); ``offset`` (default 0:
-    added to the stored weight)."""
+    added to the stored weight); ``scalar`` (default False: the weight is one number, the same for
+    every channel)."""
 
     graph_safe = True
 
     @classmethod
     def weight_specs(cls, params, hidden_size):
         mean = 1.0 - float(params.get("offset", 0.0))
-        return {"weight": (params["name"], WeightSpec((hidden_size,), init=(mean, 0.02)))}
+        shape = () if params.get("scalar") else (hidden_size,)
+        return {"weight": (params["name"], WeightSpec(shape, init=(mean, 0.02)))}
 
     def load(self, tensors):
-        self.weight = self._vector32(tensors["weight"])
+        weight = tensors["weight"]
+        if self.params.get("scalar"):          # the kernels read a weight per channel
+            weight = weight.reshape(1).expand(self.hidden_size)
+        self.weight = self._vector32(weight)
         offset = float(self.params.get("offset", 0.0))
         if offset:
             self.weight = (self.weight + offset).contiguous()

@@ -10,6 +10,10 @@ function).  Angles, cosines and sines are computed once on the host in 64-bit an
 kept as a 32-bit table ``[positions, rotary_dim/2]`` that every kernel reads, so a
 position's rotation is the same in every step shape.
 
+``scaling`` stretches long wavelengths: with l = 2 pi / f the wavelength of a pair's frequency f,
+f is kept where l < original/high, divided by ``factor`` where l > original/low, and between the two
+blended, ``(1 - s) f / factor + s f`` with ``s = (original/l - low) / (high - low)``.
+
 ``none``: queries and keys stay as they are.
 
 Interface of a position part: ``prepare(max_positions)`` builds what depends on the longest
@@ -22,6 +26,7 @@ that offers it promises that ``encode`` is exactly that rotation.
 """
 from __future__ import annotations
 
+import math
 from typing import Dict, Tuple
 
 import torch
@@ -32,11 +37,28 @@ from .base import Part, register_part
 _TABLES: Dict[Tuple, Tuple[torch.Tensor, torch.Tensor]] = {}
 
 
-def rotary_table(theta: float, rot_dim: int, positions: int, device):
-    key = (float(theta), rot_dim, positions, str(device))
+SCALING_KEYS = ("factor", "low", "high", "original")
+
+
+def stretched_frequencies(freq: torch.Tensor, scaling) -> torch.Tensor:
+    """``scaling`` (factor, low, high, original) applied to the frequencies (float64)."""
+    factor, low, high, original = (float(scaling[k]) for k in SCALING_KEYS)
+    if not (factor > 0 and original > 0 and 0 < low < high):
+        raise ValueError(f"rotary scaling needs factor > 0, original > 0 and 0 < low < high, got "
+                         f"{dict(scaling)}")
+    turns = original * freq / (2.0 * math.pi)          # of the pair over `original` positions
+    s = ((turns - low) / (high - low)).clamp(0.0, 1.0)
+    return (1.0 - s) * freq / factor + s * freq
+
+
+def rotary_table(theta: float, rot_dim: int, positions: int, device, scaling=None):
+    key = (float(theta), rot_dim, positions, str(device),
+           tuple(float(scaling[k]) for k in SCALING_KEYS) if scaling else None)
     if key not in _TABLES:
         j = torch.arange(rot_dim // 2, dtype=torch.float64)
         freq = 1.0 / torch.pow(torch.tensor(float(theta), dtype=torch.float64), 2.0 * j / rot_dim)
+        if scaling:
+            freq = stretched_frequencies(freq, scaling)
         ang = torch.arange(positions, dtype=torch.float64)[:, None] * freq[None, :]
         _TABLES[key] = (torch.cos(ang).to(torch.float32).to(device).contiguous(),
                         torch.sin(ang).to(torch.float32).to(device).contiguous())
@@ -45,7 +67,8 @@ def rotary_table(theta: float, rot_dim: int, positions: int, device):
 
 @register_part("position", "rotary")
 class Rotary(Part):
-    """params: ``theta``, ``rotary_dim``, ``pairing`` ("half" or "interleaved")."""
+    """params: ``theta``, ``rotary_dim``, ``pairing`` ("half" or "interleaved"), ``scaling``
+    (optional: factor, low, high, original)."""
 
     graph_safe = True
 
@@ -61,7 +84,8 @@ class Rotary(Part):
         self._table = None
 
     def prepare(self, max_positions: int) -> None:
-        self._table = rotary_table(self.theta, self.rot_dim, max_positions, self.device)
+        self._table = rotary_table(self.theta, self.rot_dim, max_positions, self.device,
+                                   self.params.get("scaling"))
 
     def rotary_table(self):
         cos, sin = self._table
