@@ -21,7 +21,7 @@ fraction for each); ``prefill_b8`` and ``prefill_b64`` are steps over 8 and 64 p
 ``--dtype float32`` measures the true 32-bit path.
 Every weight plus the cache exceed the L2 cache, so no flush is needed between steps.
 
-    python bench.py --design rigozen|losorax|virorax|mipurax [--design-size s|m] [--layers L]
+    python bench.py --design rigozen|losorax|virorax|mipurax|gibipel [--design-size s|m] [--layers L]
 
 measures another thing and leaves the line above as it is: prefill (1 and 8 prompts of 2,048
 tokens) and decode (batch 1, 8, 64 from a context of 2,048) of Rigozen models whose layers
@@ -38,6 +38,10 @@ layers.  ``--design mipurax`` does it for Mipurax models (all layers chunked att
 slope by distance; all layers latent attention of either kind; dense and routed feed-forwards;
 a mixture in which every fourth layer reads an earlier layer's keys and values) beside Llama
 with a window as long as the chunk, Rigozen's latent attention and Losorax's routed experts.
+``--design gibipel`` does it for Gibipel models (attention with pooled blocks beside a matrix memory
+in every layer, without and with its routed feed-forward) beside Virorax's attention and retention
+layers, whose sizes its two mixers have, and Losorax's routed experts; ``--models NAME,...`` measures
+only the named ones of any of these lists.
 """
 from __future__ import annotations
 
@@ -447,6 +451,37 @@ def mipurax_configs(z, layers):
     }
 
 
+def gibipel_configs(z, layers):
+    """name -> config.json of the models --design gibipel measures: the left mixer has the sizes and
+    the window of Virorax's attention, the right one those of its retention; of the router's outputs
+    an eighth are identities."""
+    left = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"],
+            "scale": z["dim"] ** -0.5, "mask": {"size": z["window"], "pool": 16},
+            "rot": {"base": 500000.0, "dims": z["dim"],
+                    "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 1024}}}
+    right = {"heads": z["d_heads"], "dim": z["d_dim"], "vdim": z["d_vdim"], "gate_cap": 15.0}
+    mixer = {"left": left, "right": right, "left_scale": 0.8, "right_scale": 1.1}
+    ident = z["experts"] // 8
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]},
+           "router": {"experts": z["experts"] - ident, "top": z["top"], "identity": ident,
+                      "groups": {"count": z["experts"] // 4, "keep": z["experts"] // 8}},
+           "shared": {"ff": z["expert_ff"]}}
+
+    def gibipel(mlp):
+        return {"architecture": "Gibipel", "vocab": z["vocab"], "width": z["width"],
+                "norm": {"eps": 1e-6}, "max_positions": CONTEXT, "logit_scale": 0.5,
+                "embedding": {"scale": z["width"] ** 0.5},
+                "layers": [{"type": "parallel", "mixer": mixer, "mlp": mlp}] * layers}
+    vir, los = virorax_configs(z, layers), losorax_configs(z, layers)
+    return {
+        "virorax attention": vir["virorax attention"],
+        "virorax retention": vir["virorax retention"],
+        "losorax attention routed": los["losorax attention routed"],
+        "gibipel mixers alone": gibipel(None),
+        "gibipel routed": gibipel(moe),
+    }
+
+
 def design_configs(z, layers):
     """name -> config.json of the models --design measures."""
     att = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"],
@@ -496,7 +531,15 @@ def design_bench(args) -> int:
     configs = (losorax_configs(z, layers) if args.design == "losorax"
                else virorax_configs(z, layers) if args.design == "virorax"
                else mipurax_configs(z, layers) if args.design == "mipurax"
+               else gibipel_configs(z, layers) if args.design == "gibipel"
                else design_configs(z, layers))
+    if args.models:
+        wanted = [n.strip() for n in args.models.split(",")]
+        unknown = [n for n in wanted if n not in configs]
+        if unknown:
+            print(f"--models: {unknown} are not among {sorted(configs)}")
+            return 2
+        configs = {n: configs[n] for n in wanted}
     with ClockSampler() as clocks:
         for name, cfg in configs.items():
             tmp = tempfile.mkdtemp(prefix="cretif_design_")
@@ -530,23 +573,37 @@ def design_bench(args) -> int:
             mats = 2 if cfg.get("architecture") == "Mipurax" else 3
             expert_params = sum(mats * W * m["expert"]["ff"] * m["router"]["experts"]
                                 for m in routed)
+            # (choices that fall on identities multiply nothing: counted as their share of the
+            # router's outputs)
+            def used(router):
+                return router["experts"] / (router["experts"] + router.get("identity", 0))
             active_params = params - expert_params + sum(
-                mats * W * m["expert"]["ff"] * m["router"]["top"] for m in routed)
+                mats * W * m["expert"]["ff"] * m["router"]["top"] * used(m["router"])
+                for m in routed)
             if params_run is not None:
                 active_params = params_run
 
             def read_params(b):
                 return params - expert_params + sum(
                     mats * W * m["expert"]["ff"] * min(m["router"]["experts"],
-                                                       b * m["router"]["top"])
+                                                       b * m["router"]["top"] * used(m["router"]))
                     for m in routed)
             # the embedding table is read a row at a time; an output matrix of its own is
             # multiplied on the last rows only
-            untied = cfg.get("architecture") == "Losorax"
+            untied = cfg.get("architecture") in ("Losorax", "Gibipel")
             tables = V * W * (2 if untied else 1)
             attn_flops = kept = 0.0
             for i, k in enumerate(kinds):
-                if cfg.get("architecture") == "Mipurax":
+                if k == "parallel":
+                    m, rt = cfg["layers"][i]["mixer"]["left"], cfg["layers"][i]["mixer"]["right"]
+                    w, pool = m["mask"]["size"], m["mask"]["pool"]
+                    keys = sum(min(p + 1, w) + max(0, p - w + 1) // pool for p in range(T))
+                    attn_flops += 4.0 * keys * m["heads"] * m["dim"]
+                    kept += 2 * (2 * m["kv_heads"] * m["dim"]) \
+                        * (min(T, w) + max(0, T - w) // pool)
+                    attn_flops += T * rt["heads"] * 4 * rt["dim"] * rt["vdim"]
+                    kept += 2 * 4 * rt["heads"] * rt["dim"] * rt["vdim"]
+                elif cfg.get("architecture") == "Mipurax":
                     m = cfg["layers"][i]["mixer"]
                     if k == "attention":        # the keys of a query's own chunk; a reader keeps none
                         chunk = m["mask"]["size"]
@@ -694,9 +751,11 @@ def main() -> int:
     ap.add_argument("--unequal", action="store_true",
                     help="prompts of unequal lengths 256..2,048 instead of 2,048 each")
     ap.add_argument("--design", default=None,
-                    choices=["rigozen", "losorax", "virorax", "mipurax"],
+                    choices=["rigozen", "losorax", "virorax", "mipurax", "gibipel"],
                     help="measure this design at real layer sizes beside Llama at the same "
                          "sizes instead of the headline (another JSON line)")
+    ap.add_argument("--models", default=None,
+                    help="with --design: only these models of its list, separated by commas")
     ap.add_argument("--design-size", default="m", choices=sorted(DESIGN_SIZES))
     args = ap.parse_args()
 

@@ -164,7 +164,7 @@ int cretif_moe_gather_rows(const void* x, int ldx, void* xs, int lds, const int*
 // place may be null: the rows are in the pairs' own order; wts may be null: no weights.
 int cretif_moe_combine(const float* rows, int ld, const int* place, int top, const float* wts,
                        float* y, int T, int H, const int* ids, int experts, const float* id_wts,
-                       const void* x, int x_dt, int ldx, void* stream);
+                       const void* x, int x_dt, int ldx, const float* plus, void* stream);
 
 // After a decode step: ids <- sampled (if given), positions and lengths + 1.
 int cretif_advance_decode(int* tok_ids, int* tok_pos, int* seq_start, const int* sampled, int B,

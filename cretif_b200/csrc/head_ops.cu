@@ -162,6 +162,51 @@ __device__ __forceinline__ void write_entry(const T* kc, const T* vc, const int*
   }
 }
 
+// Eight channels a thread (bfloat16, head sizes multiples of eight): grid (entries, 1, B), the threads
+// of a CTA take a token block's heads and channels in turn.
+__global__ void __launch_bounds__(256)
+pool_kv8_kernel(const __nv_bfloat16* kc, const __nv_bfloat16* vc, const int* __restrict__ table,
+                int table_stride, __nv_bfloat16* pk, __nv_bfloat16* pv,
+                const int* __restrict__ pool_table, int pool_stride, int pool,
+                const int* __restrict__ cu_seqlens, const int* __restrict__ seq_start,
+                const int* __restrict__ seq_slot, int nkv, int hd, int vd, int bt,
+                unsigned int* __restrict__ fault) {
+  const int b = blockIdx.z;
+  const int start = seq_start[b], end = start + cu_seqlens[b + 1] - cu_seqlens[b];
+  const int e = start / pool + blockIdx.x;
+  if (e >= end / pool) return;
+  const int slot = seq_slot[b];
+  const int* tab = table + (size_t)slot * table_stride;
+  const int blk = pool_table[(size_t)slot * pool_stride + e / bt];
+  if (blk < 0) {
+    if (threadIdx.x == 0) atomicOr(fault, kFaultBlockTable);
+    return;
+  }
+  const int per = (hd + vd) >> 3;
+  for (int idx = threadIdx.x; idx < nkv * per; idx += 256) {
+    const int kvh = idx / per;
+    int c = (idx - kvh * per) << 3;
+    const bool is_k = c < hd;
+    if (!is_k) c -= hd;
+    const __nv_bfloat16* cache = is_k ? kc : vc;
+    const int n = is_k ? hd : vd;
+    float sum[8];
+#pragma unroll
+    for (int u = 0; u < 8; ++u) sum[u] = 0.f;
+#pragma unroll 8
+    for (int r = 0; r < pool; ++r) {
+      const int p = e * pool + r, from = max(tab[p / bt], 0);
+      float x[8];
+      load8(cache + (((size_t)from * nkv + kvh) * bt + p % bt) * n + c, x);
+#pragma unroll
+      for (int u = 0; u < 8; ++u) sum[u] += x[u];
+    }
+#pragma unroll
+    for (int u = 0; u < 8; ++u) sum[u] /= (float)pool;
+    store8((is_k ? pk : pv) + (((size_t)blk * nkv + kvh) * bt + e % bt) * n + c, sum);
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128)
 pool_kv_kernel(const T* kc, const T* vc, const int* __restrict__ table, int table_stride, T* pk, T* pv,
@@ -179,9 +224,10 @@ pool_kv_kernel(const T* kc, const T* vc, const int* __restrict__ table, int tabl
               (int)threadIdx.x, (int)blockDim.x, fault);
 }
 
-// VEC: four channels a thread (head size, rotated part and addresses allow it).
-template <typename T, bool VEC>
-__global__ void __launch_bounds__(256)
+// VEC: four channels a thread (head size, rotated part and addresses allow it).  NT threads a token:
+// a step of few tokens takes 1024, so that a row is one turn of loads, prompts take 256.
+template <typename T, bool VEC, int NT>
+__global__ void __launch_bounds__(NT)
 projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
                                const float* __restrict__ bias, const float* __restrict__ wq,
                                const float* __restrict__ wk, float eps,
@@ -194,14 +240,33 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
                                const int* __restrict__ pool_table, int pool_stride, int pool,
                                unsigned int* __restrict__ fault) {
   extern __shared__ __align__(16) float row_s[];       // q | k with the bias
-  __shared__ float sums[8][2];
+  __shared__ float sums[NT / 32][2];
   const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int pos = tok_pos[t];
   const float* row = proj + (size_t)t * ldp;
   const int nq = nh * hd, nk = nkv * hd, nqk = nq + nk;
   float ssq = 0.f, ssk = 0.f;
+  int slot = 0, blk = -1;
+  if (write_cache) {                  // (a chain of loads: asked for before the row)
+    slot = seq_slot[tok_seq[t]];
+    blk = table[(size_t)slot * table_stride + pos / bt];
+    if (blk < 0 && tid == 0) atomicOr(fault, kFaultBlockTable);
+  }
+  // the thread's first value column and the weights of its first turn, before the row's sums are known
+  const float v_first = tid < nkv * vd ? row[nqk + tid] + (bias ? bias[nqk + tid] : 0.f) : 0.f;
+  const int half = rot_dim >> 1;
+  const float* c = cos_t + (size_t)pos * half;
+  const float* s = sin_t + (size_t)pos * half;
   if (VEC) {
-    for (int i = 4 * tid; i < nqk; i += 4 * 256) {
+    if (NT > 256 && 4 * tid < nqk) {
+      const int i = 4 * tid % hd;
+      asm volatile("prefetch.global.L1 [%0];" ::"l"(4 * tid < nq ? wq + 4 * tid : wk + 4 * tid - nq));
+      if (i < half) {
+        asm volatile("prefetch.global.L1 [%0];" ::"l"(c + i));
+        asm volatile("prefetch.global.L1 [%0];" ::"l"(s + i));
+      }
+    }
+    for (int i = 4 * tid; i < nqk; i += 4 * NT) {
       float4 v = *reinterpret_cast<const float4*>(row + i);
       if (bias) {
         const float4 b4 = *reinterpret_cast<const float4*>(bias + i);
@@ -212,30 +277,20 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
       if (i < nq) ssq += s4; else ssk += s4;
     }
   } else {
-    for (int i = tid; i < nqk; i += 256) {
+    for (int i = tid; i < nqk; i += NT) {
       const float v = row[i] + (bias ? bias[i] : 0.f);
       row_s[i] = v;
       if (i < nq) ssq += v * v; else ssk += v * v;
     }
   }
-  int slot = 0, blk = -1;
-  if (write_cache) {
-    slot = seq_slot[tok_seq[t]];
-    blk = table[(size_t)slot * table_stride + pos / bt];
-    if (blk < 0 && tid == 0) atomicOr(fault, kFaultBlockTable);
-  }
   ssq = warp_sum(ssq);
   ssk = warp_sum(ssk);
   if (lane == 0) { sums[warp][0] = ssq; sums[warp][1] = ssk; }
   __syncthreads();
-  ssq = ssk = 0.f;
-#pragma unroll
-  for (int w = 0; w < 8; ++w) { ssq += sums[w][0]; ssk += sums[w][1]; }
+  ssq = warp_sum(lane < NT / 32 ? sums[lane][0] : 0.f);
+  ssk = warp_sum(lane < NT / 32 ? sums[lane][1] : 0.f);
   const float fq = 1.0f / sqrtf(ssq / (float)nq + eps);
   const float fk = nk ? 1.0f / sqrtf(ssk / (float)nk + eps) : 0.f;
-  const int half = rot_dim >> 1;
-  const float* c = cos_t + (size_t)pos * half;
-  const float* s = sin_t + (size_t)pos * half;
   const int n_write = write_cache && blk >= 0 ? nqk : nq;
   auto normed = [&](int idx) {
     return idx < nq ? row_s[idx] * fq * wq[idx] : row_s[idx] * fk * wk[idx - nq];
@@ -246,7 +301,7 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
     return kc + (((size_t)blk * nkv + kvh) * bt + pos % bt) * hd + i;
   };
   if (VEC) {
-    for (int idx = 4 * tid; idx < n_write; idx += 4 * 256) {
+    for (int idx = 4 * tid; idx < n_write; idx += 4 * NT) {
       const int i = idx % hd;
       float v[4];
 #pragma unroll
@@ -280,7 +335,7 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
       }
     }
   } else {
-    for (int idx = tid; idx < n_write; idx += 256) {
+    for (int idx = tid; idx < n_write; idx += NT) {
       const int i = idx % hd;
       float v = normed(idx);
       if (i < rot_dim) {
@@ -294,16 +349,16 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
     }
   }
   if (!write_cache || blk < 0) return;
-  for (int idx = tid; idx < nkv * vd; idx += 256) {
+  for (int idx = tid; idx < nkv * vd; idx += NT) {
     const int kvh = idx / vd, i = idx - kvh * vd;
-    const float v = row[nqk + idx] + (bias ? bias[nqk + idx] : 0.f);
+    const float v = idx == tid ? v_first : row[nqk + idx] + (bias ? bias[nqk + idx] : 0.f);
     vc[(((size_t)blk * nkv + kvh) * bt + pos % bt) * vd + i] = from_float<T>(v * v_scale);
   }
   if (pool_table && (pos + 1) % pool == 0) {       // (one token a sequence: this one ends a block)
     __syncthreads();
     write_entry<T>(kc, vc, table + (size_t)slot * table_stride, pk, pv,
                    pool_table + (size_t)slot * pool_stride, pool, pos / pool, nkv, 0, nkv, hd, vd, bt,
-                   tid, 256, fault);
+                   tid, NT, fault);
   }
 }
 
@@ -470,13 +525,18 @@ extern "C" int cretif_projnorm_rope_kv_append(
   cudaStream_t st = (cudaStream_t)stream;
 #define CRETIF_PN(TT, VEC)                                                                        \
   do {                                                                                            \
+    if (T < 64) CRETIF_PN_N(TT, VEC, 1024);                                                       \
+    else CRETIF_PN_N(TT, VEC, 256);                                                               \
+  } while (0)
+#define CRETIF_PN_N(TT, VEC, NT)                                                                  \
+  do {                                                                                            \
     if (smem > 40 * 1024) {                                                                       \
-      cudaError_t err = cudaFuncSetAttribute(projnorm_rope_kv_append_kernel<TT, VEC>,             \
+      cudaError_t err = cudaFuncSetAttribute(projnorm_rope_kv_append_kernel<TT, VEC, NT>,         \
                                              cudaFuncAttributeMaxDynamicSharedMemorySize,         \
                                              (int)smem);                                          \
       if (err != cudaSuccess) return (int)err;                                                    \
     }                                                                                             \
-    projnorm_rope_kv_append_kernel<TT, VEC><<<T, 256, smem, st>>>(                                \
+    projnorm_rope_kv_append_kernel<TT, VEC, NT><<<T, NT, smem, st>>>(                             \
         proj, ldp, bias, wq, wk, eps, cos_t, sin_t, pairing, rot_dim, tok_pos, tok_seq, seq_slot, \
         nh, nkv, hd, vd, v_scale, (TT*)q_out, ldq, table, table_stride, (TT*)kc, (TT*)vc, bt,     \
         write_cache, (TT*)pool_k, (TT*)pool_v, pool_table, pool_stride, pool, fault);             \
@@ -490,6 +550,7 @@ extern "C" int cretif_projnorm_rope_kv_append(
   } else {
     return kBadDType;
   }
+#undef CRETIF_PN_N
 #undef CRETIF_PN
   return launch_status();
 }
@@ -510,6 +571,12 @@ extern "C" int cretif_pool_kv(const void* kc, const void* vc, int dt, const int*
     pool_kv_kernel<float><<<grid, 128, 0, st>>>(
         (const float*)kc, (const float*)vc, table, table_stride, (float*)pool_k, (float*)pool_v,
         pool_table, pool_stride, pool, cu_seqlens, seq_start, seq_slot, nkv, hd, vd, bt, fault);
+  else if (dt == kBF16 && hd % 8 == 0 && vd % 8 == 0 &&
+           (((uintptr_t)kc | (uintptr_t)vc | (uintptr_t)pool_k | (uintptr_t)pool_v) & 15) == 0)
+    pool_kv8_kernel<<<dim3(grid.x, 1, B), 256, 0, st>>>(
+        (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, table, table_stride,
+        (__nv_bfloat16*)pool_k, (__nv_bfloat16*)pool_v, pool_table, pool_stride, pool, cu_seqlens,
+        seq_start, seq_slot, nkv, hd, vd, bt, fault);
   else if (dt == kBF16)
     pool_kv_kernel<__nv_bfloat16><<<grid, 128, 0, st>>>(
         (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc, table, table_stride,

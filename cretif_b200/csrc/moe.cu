@@ -30,6 +30,8 @@
 //   once per pair.
 #include <mma.h>
 
+#include <type_traits>
+
 #include "api.h"
 #include "common.cuh"
 
@@ -55,39 +57,40 @@ struct RouteRule {
 // Warp-wide: the `top` largest choices of E outputs (ties: the lower index) among those of the groups
 // that are kept, their scores as weights, written for token t.  `scratch`: E floats and
 // `groups` ints of shared memory that belong to this warp.
-__device__ __forceinline__ void select_top(const float* logits, int E, const RouteRule rule,
+template <int NPL>
+__device__ __forceinline__ void select_top_n(const float* logits, int E, const RouteRule rule,
                                            int* __restrict__ ids, float* __restrict__ wts, int t,
                                            int lane, float* scratch) {
   const int top = rule.top, renorm = rule.renorm;
-  float z[kMaxExpertsPerLane];
+  float z[NPL];
 #pragma unroll
-  for (int m = 0; m < kMaxExpertsPerLane; ++m) {
+  for (int m = 0; m < NPL; ++m) {
     const int e = lane + 32 * m;
     z[m] = e < E ? logits[e] : -INFINITY;
   }
   // sc: the scores; z from here on: what the choice compares (the logits order like their logistic
   // scores, so without a correction they are compared as they are)
-  float sc[kMaxExpertsPerLane];
+  float sc[NPL];
   if (rule.softmax) {
     float mx = -INFINITY, sum = 0.f;
 #pragma unroll
-    for (int m = 0; m < kMaxExpertsPerLane; ++m) mx = fmaxf(mx, z[m]);
+    for (int m = 0; m < NPL; ++m) mx = fmaxf(mx, z[m]);
     mx = warp_max(mx);
 #pragma unroll
-    for (int m = 0; m < kMaxExpertsPerLane; ++m) {
+    for (int m = 0; m < NPL; ++m) {
       sc[m] = lane + 32 * m < E ? expf(z[m] - mx) : 0.f;
       sum += sc[m];
     }
     sum = warp_sum(sum);
 #pragma unroll
-    for (int m = 0; m < kMaxExpertsPerLane; ++m) sc[m] /= sum;
+    for (int m = 0; m < NPL; ++m) sc[m] /= sum;
   } else {
 #pragma unroll
-    for (int m = 0; m < kMaxExpertsPerLane; ++m) sc[m] = 1.0f / (1.0f + expf(-z[m]));
+    for (int m = 0; m < NPL; ++m) sc[m] = 1.0f / (1.0f + expf(-z[m]));
   }
   if (rule.correction) {
 #pragma unroll
-    for (int m = 0; m < kMaxExpertsPerLane; ++m) {
+    for (int m = 0; m < NPL; ++m) {
       const int e = lane + 32 * m;
       if (e < E) z[m] = sc[m] + rule.correction[e];
     }
@@ -97,16 +100,16 @@ __device__ __forceinline__ void select_top(const float* logits, int E, const Rou
     int* kept = reinterpret_cast<int*>(scratch + E);
     __syncwarp();
 #pragma unroll
-    for (int m = 0; m < kMaxExpertsPerLane; ++m) {
+    for (int m = 0; m < NPL; ++m) {
       const int e = lane + 32 * m;
       if (e < E) scratch[e] = rule.correction ? z[m] : sc[m];
     }
     for (int g = lane; g < rule.groups; g += 32) kept[g] = 0;
     __syncwarp();
     // lane g % 32 scores group g by its largest or its two largest choice scores
-    float gs[kMaxExpertsPerLane];
+    float gs[NPL];
 #pragma unroll
-    for (int m = 0; m < kMaxExpertsPerLane; ++m) {
+    for (int m = 0; m < NPL; ++m) {
       const int g = lane + 32 * m;
       gs[m] = -INFINITY;
       if (g < rule.groups) {
@@ -122,7 +125,7 @@ __device__ __forceinline__ void select_top(const float* logits, int E, const Rou
       float best = -INFINITY;
       int best_g = 0x7fffffff;
 #pragma unroll
-      for (int m = 0; m < kMaxExpertsPerLane; ++m) {
+      for (int m = 0; m < NPL; ++m) {
         const int g = lane + 32 * m;
         if (g < rule.groups && gs[m] > best) { best = gs[m]; best_g = g; }
       }
@@ -135,14 +138,14 @@ __device__ __forceinline__ void select_top(const float* logits, int E, const Rou
       if (best_g == 0x7fffffff) break;
       if ((best_g & 31) == lane) {
 #pragma unroll
-        for (int m = 0; m < kMaxExpertsPerLane; ++m)
+        for (int m = 0; m < NPL; ++m)
           if (m == (best_g >> 5)) gs[m] = -INFINITY;
         kept[best_g] = 1;
       }
     }
     __syncwarp();
 #pragma unroll
-    for (int m = 0; m < kMaxExpertsPerLane; ++m) {
+    for (int m = 0; m < NPL; ++m) {
       const int e = lane + 32 * m;
       if (e < E && !kept[e / per]) z[m] = -INFINITY;
     }
@@ -154,7 +157,7 @@ __device__ __forceinline__ void select_top(const float* logits, int E, const Rou
     float best = -INFINITY;
     int best_e = 0x7fffffff;
 #pragma unroll
-    for (int m = 0; m < kMaxExpertsPerLane; ++m) {
+    for (int m = 0; m < NPL; ++m) {
       const int e = lane + 32 * m;
       if (e < E && z[m] > best) { best = z[m]; best_e = e; }
     }
@@ -168,7 +171,7 @@ __device__ __forceinline__ void select_top(const float* logits, int E, const Rou
     float s = 0.f;
     if ((best_e & 31) == lane) {
 #pragma unroll
-      for (int m = 0; m < kMaxExpertsPerLane; ++m)
+      for (int m = 0; m < NPL; ++m)
         if (m == (best_e >> 5)) {
           z[m] = -INFINITY;
           s = sc[m];
@@ -188,6 +191,15 @@ __device__ __forceinline__ void select_top(const float* logits, int E, const Rou
   }
   if (renorm && top > 32 && lane == 0)
     for (int k = 32; k < top; ++k) wts[(size_t)t * top + k] /= total + rule.sum_eps;
+}
+
+// (a lane holds as many outputs as E asks for)
+__device__ __forceinline__ void select_top(const float* logits, int E, const RouteRule rule,
+                                           int* __restrict__ ids, float* __restrict__ wts, int t,
+                                           int lane, float* scratch) {
+  if (E <= 32) select_top_n<1>(logits, E, rule, ids, wts, t, lane, scratch);
+  else if (E <= 64) select_top_n<2>(logits, E, rule, ids, wts, t, lane, scratch);
+  else select_top_n<kMaxExpertsPerLane>(logits, E, rule, ids, wts, t, lane, scratch);
 }
 
 // A CTA per token: its sixteen warps take the experts in turn (a dot product each, every load of
@@ -568,64 +580,106 @@ moe_gemv_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, void*
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const size_t w_rows = (size_t)(mode == 0 ? 2 * N : N);
   const T* We = W + (size_t)e * w_rows * K;
-  auto dot = [&](const T* wrow) {
-    float acc = 0.f;
+  // The warp's rows together, so that their loads travel together: row n of its two columns and, with
+  // a gate, row N + n of each.  (A column beyond N reads the last one's rows and stores nothing.)
+  const int n0 = blockIdx.x * 16 + warp * 2;
+  const T* w0 = We + (size_t)min(n0, N - 1) * K;
+  const T* w1 = We + (size_t)min(n0 + 1, N - 1) * K;
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  auto rows_of = [&](auto gate) {
+    constexpr int R = decltype(gate)::value ? 4 : 2;
+    const T* w[4] = {w0, w1, w0 + (R == 4 ? (size_t)N * K : 0), w1 + (R == 4 ? (size_t)N * K : 0)};
     if (vec) {
-#pragma unroll 4
+#pragma unroll 2
       for (int i = lane * 8; i < K; i += 256) {
-        float a[8], b[8];
-        load8(wrow + i, a);
+        float a[R][8], b[8];
+#pragma unroll
+        for (int r = 0; r < R; ++r) load8(w[r] + i, a[r]);
         load8(xs + i, b);
 #pragma unroll
-        for (int q = 0; q < 8; ++q) acc = fmaf(a[q], b[q], acc);
+        for (int r = 0; r < R; ++r)
+#pragma unroll
+          for (int q = 0; q < 8; ++q) acc[r] = fmaf(a[r][q], b[q], acc[r]);
       }
     } else {
-      for (int i = lane; i < K; i += 32) acc = fmaf(to_float(wrow[i]), to_float(xs[i]), acc);
+      for (int i = lane; i < K; i += 32)
+#pragma unroll
+        for (int r = 0; r < R; ++r) acc[r] = fmaf(to_float(w[r][i]), to_float(xs[i]), acc[r]);
     }
-    return warp_sum(acc);
+#pragma unroll
+    for (int r = 0; r < R; ++r) acc[r] = warp_sum(acc[r]);
   };
+  if (mode == 0) rows_of(std::true_type{});
+  else rows_of(std::false_type{});
 #pragma unroll
   for (int c = 0; c < 2; ++c) {
-    const int n = blockIdx.x * 16 + warp * 2 + c;
+    const int n = n0 + c;
     if (n >= N) continue;
     if (mode == 0) {
       const float sg = scale_at == 1 ? s : 1.f;
-      const float g = dot(We + (size_t)n * K) * sg, u = dot(We + ((size_t)N + n) * K) * sg;
+      const float g = acc[c] * sg, u = acc[2 + c] * sg;
       if (lane == 0)
         reinterpret_cast<T*>(Cv)[(size_t)p * ldc + n] = from_float<T>(g / (1.0f + expf(-g)) * u);
     } else if (mode >= 2) {
-      const float v = dot(We + (size_t)n * K) * (scale_at == 1 ? s : 1.f);
+      const float v = acc[c] * (scale_at == 1 ? s : 1.f);
       if (lane == 0)
         reinterpret_cast<T*>(Cv)[(size_t)p * ldc + n] = from_float<T>(unary_activation(v, mode - 2));
     } else {
-      const float v = dot(We + (size_t)n * K) * (scale_at == 2 ? s : 1.f);
+      const float v = acc[c] * (scale_at == 2 ? s : 1.f);
       if (lane == 0) reinterpret_cast<float*>(Cv)[(size_t)p * ldc + n] = v;
     }
   }
 }
 
+// V columns a thread (4: rows, y and x allow 16-byte accesses, 8-byte ones for bfloat16).
 // Identity pairs (ids[pair] >= experts): id_wts[pair] times the token's row of x instead of a row of
 // the products.  wts: weights that the products have not applied yet.
-template <typename TX>
+template <typename TX, int V>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ rows, int ld, const int* __restrict__ place, int top,
                    const float* __restrict__ wts, float* __restrict__ y, int T, int H,
                    const int* __restrict__ ids, int experts, const float* __restrict__ id_wts,
-                   const TX* __restrict__ x, int ldx) {
-  const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+                   const TX* __restrict__ x, int ldx, const float* __restrict__ plus) {
+  const long long idx = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
   if (idx >= (long long)T * H) return;
   const int t = (int)(idx / H), c = (int)(idx - (long long)t * H);
-  float acc = 0.f;
+  float acc[V];
+#pragma unroll
+  for (int u = 0; u < V; ++u) acc[u] = 0.f;
+#pragma unroll 4
   for (int k = 0; k < top; ++k) {
     const size_t pair = (size_t)t * top + k;
+    float v[V], w;
     if (ids && ids[pair] >= experts) {
-      acc += id_wts[pair] * to_float(x[(size_t)t * ldx + c]);
-      continue;
+      w = id_wts[pair];
+      if (V == 4) {
+        const float4 a = ld4_as_float(x + (size_t)t * ldx + c);
+        v[0] = a.x; v[V > 1 ? 1 : 0] = a.y; v[V > 2 ? 2 : 0] = a.z; v[V > 3 ? 3 : 0] = a.w;
+      } else {
+        v[0] = to_float(x[(size_t)t * ldx + c]);
+      }
+    } else {
+      w = wts ? wts[pair] : 1.0f;
+      const float* row = rows + (place ? (size_t)place[pair] : pair) * ld + c;
+      if (V == 4) {
+        const float4 a = *reinterpret_cast<const float4*>(row);
+        v[0] = a.x; v[V > 1 ? 1 : 0] = a.y; v[V > 2 ? 2 : 0] = a.z; v[V > 3 ? 3 : 0] = a.w;
+      } else {
+        v[0] = *row;
+      }
     }
-    const float v = rows[(place ? (size_t)place[pair] : pair) * ld + c];
-    acc += wts ? wts[pair] * v : v;
+#pragma unroll
+    for (int u = 0; u < V; ++u) acc[u] += w * v[u];
   }
-  y[idx] = acc;
+  if (plus) {
+#pragma unroll
+    for (int u = 0; u < V; ++u) acc[u] += plus[idx + u];
+  }
+  if (V == 4)
+    *reinterpret_cast<float4*>(y + idx) = make_float4(acc[0], acc[V > 1 ? 1 : 0], acc[V > 2 ? 2 : 0],
+                                                      acc[V > 3 ? 3 : 0]);
+  else
+    y[idx] = acc[0];
 }
 
 }  // namespace
@@ -795,22 +849,30 @@ extern "C" int cretif_moe_gemv(const void* A, int a_dt, int lda, const void* W, 
   return launch_status();
 }
 
-// ids non-null: pairs whose id is `experts` or more are identities (see moe_combine_kernel).
+// ids non-null: pairs whose id is `experts` or more are identities (see moe_combine_kernel).  plus
+// [T, H] (may be null) is added last.
 extern "C" int cretif_moe_combine(const float* rows, int ld, const int* place, int top,
                                   const float* wts, float* y, int T, int H, const int* ids,
                                   int experts, const float* id_wts, const void* x, int x_dt, int ldx,
-                                  void* stream) {
+                                  const float* plus, void* stream) {
   if (T <= 0) return kOk;
   if (H <= 0 || ld < H || top <= 0 || (ids && (!id_wts || !x || ldx < H))) return kBadArgument;
-  const unsigned blocks = (unsigned)(((long long)T * H + 255) / 256);
+  const bool vec = H % 4 == 0 && ld % 4 == 0 && (!ids || ldx % 4 == 0) &&
+                   (((uintptr_t)rows | (uintptr_t)y | (uintptr_t)x) & 15) == 0;
+  const unsigned blocks = (unsigned)(((long long)T * H / (vec ? 4 : 1) + 255) / 256);
   cudaStream_t st = (cudaStream_t)stream;
-  if (x_dt == kF32)
-    moe_combine_kernel<float><<<blocks, 256, 0, st>>>(rows, ld, place, top, wts, y, T, H, ids, experts,
-                                                      id_wts, (const float*)x, ldx);
-  else if (x_dt == kBF16)
-    moe_combine_kernel<__nv_bfloat16><<<blocks, 256, 0, st>>>(
-        rows, ld, place, top, wts, y, T, H, ids, experts, id_wts, (const __nv_bfloat16*)x, ldx);
-  else
-    return kBadDType;
+#define CRETIF_COMBINE(TX)                                                                          \
+  do {                                                                                              \
+    if (vec)                                                                                        \
+      moe_combine_kernel<TX, 4><<<blocks, 256, 0, st>>>(rows, ld, place, top, wts, y, T, H, ids,    \
+                                                        experts, id_wts, (const TX*)x, ldx, plus);  \
+    else                                                                                            \
+      moe_combine_kernel<TX, 1><<<blocks, 256, 0, st>>>(rows, ld, place, top, wts, y, T, H, ids,    \
+                                                        experts, id_wts, (const TX*)x, ldx, plus);  \
+  } while (0)
+  if (x_dt == kF32) CRETIF_COMBINE(float);
+  else if (x_dt == kBF16) CRETIF_COMBINE(__nv_bfloat16);
+  else return kBadDType;
+#undef CRETIF_COMBINE
   return launch_status();
 }

@@ -105,6 +105,56 @@ rmsnorm_add_kernel(float* __restrict__ h, const TY* __restrict__ y, int ldy,
   }
 }
 
+// The same for few rows (a decode step): a CTA per row, four columns a thread and turn, everything a
+// thread reads asked for before the row's sum is known.  Up to 2 x 1024 columns stay in registers.
+template <typename TY>
+__global__ void __launch_bounds__(256)
+rmsnorm_add_row_block_kernel(float* __restrict__ h, const TY* __restrict__ y, int ldy,
+                             const float* __restrict__ weight, int H, float eps,
+                             __nv_bfloat16* __restrict__ x_out) {
+  __shared__ float sums[8];
+  const int r = blockIdx.x, tid = threadIdx.x, n4 = H >> 2;
+  const TY* yrow = y + (size_t)r * ldy;
+  float* hrow = h + (size_t)r * H;
+  __nv_bfloat16* xrow = x_out ? x_out + (size_t)r * H : nullptr;
+  constexpr int kKeep = 2;
+  float4 a[kKeep], w[kKeep], v[kKeep];
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u) {
+    const int i = u * 256 + tid;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    a[u] = i < n4 ? ld4(yrow + 4 * i) : zero;
+    w[u] = i < n4 ? ld4(weight + 4 * i) : zero;
+    v[u] = i < n4 ? ld4(hrow + 4 * i) : zero;
+    ss += a[u].x * a[u].x + a[u].y * a[u].y + a[u].z * a[u].z + a[u].w * a[u].w;
+  }
+  for (int i = kKeep * 256 + tid; i < n4; i += 256) {
+    const float4 b = ld4(yrow + 4 * i);
+    ss += b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w;
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) sums[tid >> 5] = ss;
+  __syncthreads();
+  ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < 8; ++u) ss += sums[u];
+  const float inv = 1.0f / sqrtf(ss / (float)H + eps);
+  auto put = [&](int i, float4 b, float4 g, float4 t) {
+    t.x += b.x * inv * g.x; t.y += b.y * inv * g.y;
+    t.z += b.z * inv * g.z; t.w += b.w * inv * g.w;
+    *reinterpret_cast<float4*>(hrow + 4 * i) = t;
+    if (xrow) st4_bf16(xrow + 4 * i, t);
+  };
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u) {
+    const int i = u * 256 + tid;
+    if (i < n4) put(i, a[u], w[u], v[u]);
+  }
+  for (int i = kKeep * 256 + tid; i < n4; i += 256)
+    put(i, ld4(yrow + 4 * i), ld4(weight + 4 * i), ld4(hrow + 4 * i));
+}
+
 template <typename TO>
 __global__ void convert_rows_kernel(const float* __restrict__ h, TO* __restrict__ out,
                                     size_t total) {
@@ -178,6 +228,16 @@ extern "C" int cretif_rmsnorm_add(float* h, const void* y, int y_dt, int ldy, co
   const bool vec = H % 4 == 0 && ldy % 4 == 0 &&
                    (((uintptr_t)h | (uintptr_t)y | (uintptr_t)weight | (uintptr_t)x_out) & 15) == 0;
   __nv_bfloat16* xo = (__nv_bfloat16*)x_out;
+  if (vec && R < 256 && H >= 512) {
+    if (y_dt == kF32)
+      rmsnorm_add_row_block_kernel<float><<<R, 256, 0, st>>>(h, (const float*)y, ldy, weight, H, eps, xo);
+    else if (y_dt == kBF16)
+      rmsnorm_add_row_block_kernel<__nv_bfloat16><<<R, 256, 0, st>>>(h, (const __nv_bfloat16*)y, ldy,
+                                                                     weight, H, eps, xo);
+    else
+      return kBadDType;
+    return launch_status();
+  }
   if (y_dt == kF32) {
     if (vec) rmsnorm_add_kernel<float, true><<<blocks, 256, 0, st>>>(h, (const float*)y, ldy, weight, R, H, eps, xo);
     else rmsnorm_add_kernel<float, false><<<blocks, 256, 0, st>>>(h, (const float*)y, ldy, weight, R, H, eps, xo);

@@ -1101,11 +1101,12 @@ def gemm_tc_grouped(a, w, c, tile_expert, used) -> None:
         _p(used), _p(fault_word(a.device)), _stream()), "gemm_tc_grouped")
 
 
-def moe_combine(rows, place, top: int, y, wts=None, identity=None) -> None:
+def moe_combine(rows, place, top: int, y, wts=None, identity=None, plus=None) -> None:
     """y[t] = the sum of the token's ``top`` rows of ``rows`` (float32), in their order, each
     times its weight when ``wts`` is given; ``place`` None: the rows are in the pairs' own
     order.  ``identity`` (``(ids, experts, weights, x)``): a pair whose id is ``experts`` or more has
-    no row of its own and adds its weight times the token's row of ``x``."""
+    no row of its own and adds its weight times the token's row of ``x``.  ``plus`` (float32, like
+    ``y``) is added last."""
     _need(rows, "rows", torch.float32, 2); _need(y, "y", torch.float32, 2)
     if place is not None:
         _need(place, "place", torch.int32)
@@ -1113,6 +1114,10 @@ def moe_combine(rows, place, top: int, y, wts=None, identity=None) -> None:
     if (rows.shape[1] != H or (place is not None and place.numel() != T * top)
             or rows.shape[0] < T * top or not y.is_contiguous()):
         raise KernelError("moe_combine: sizes do not fit")
+    if plus is not None:
+        _need(plus, "plus", torch.float32, 2)
+        if plus.shape != y.shape or not plus.is_contiguous():
+            raise KernelError("moe_combine: plus must match y")
     ids = id_wts = x = None
     experts = ldx = x_dt = 0
     if identity is not None:
@@ -1124,7 +1129,7 @@ def moe_combine(rows, place, top: int, y, wts=None, identity=None) -> None:
         ldx, x_dt = _rows(x, "x"), _dt(x)
     _check(lib().cretif_moe_combine(_p(rows), _rows(rows, "rows"), _p(place), top, _p(wts), _p(y),
                                     T, H, _p(ids), int(experts), _p(id_wts), _p(x), x_dt, ldx,
-                                    _stream()), "moe_combine")
+                                    _p(plus), _stream()), "moe_combine")
 
 
 # ------------------------------------------------------------------ attention

@@ -21,7 +21,8 @@ token uses with weight one.
 The step's (token, choice) pairs are sorted by expert on the device and each expert's rows
 are one slice of two grouped products (csrc/moe.cu): gate|up with the activation — and the
 weight, when it scales the input: the products are linear, so it is applied to the 32-bit sums —
-in its epilogue, then down; the choices are summed in their order.  The grid of every launch is
+in its epilogue, then down; the choices are summed in their order.  In a step of few tokens the shared
+expert runs on a stream of its own beside them.  The grid of every launch is
 fixed by the step's size alone, so steps can be captured as CUDA graphs.
 """
 from __future__ import annotations
@@ -32,6 +33,7 @@ from ..csrc import ops
 from ..weights.loader import WeightSpec
 from ..config.spec import PartSpec
 from .base import Part, build_part, register_part
+from .side_stream import Fork, forks
 
 
 # Steps of at most this many (token, choice) pairs take the streaming kernel, which reads an
@@ -164,6 +166,13 @@ class RoutedExperts(Part):
         T, H = x.shape
         dev = x.device
         P = T * self.top
+        # the shared expert: in a step of few tokens beside the routed ones, its output then joins
+        # where the choices are summed; otherwise added to their sum
+        fork = beside = None
+        if self.shared is not None and forks(T):
+            fork = Fork(dev)
+            with fork:
+                beside = self.shared.forward(x, ctx)
         ids = torch.empty((T, self.top), dtype=torch.int32, device=dev)
         wts = torch.empty((T, self.top), dtype=torch.float32, device=dev)
         if self.router_matrix is not None and (T > ROUTE_BY_PRODUCT
@@ -175,10 +184,10 @@ class RoutedExperts(Part):
             ops.moe_route(x, self.router, self.top, ids, wts, **self._rule())
         y = torch.empty((T, H), dtype=torch.float32, device=dev)
         if self.gated:
-            self._gated_experts(x, ids, wts, y)
+            self._gated_experts(x, ids, wts, y, fork, beside)
         else:
-            self._plain_experts(x, ids, wts, y)
-        if self.shared is not None:
+            self._plain_experts(x, ids, wts, y, fork, beside)
+        if self.shared is not None and beside is None:
             self.shared.forward(x, ctx, into=y)
         return y
 
@@ -186,12 +195,15 @@ class RoutedExperts(Part):
         return dict(renorm=self.renorm, groups=self.groups, keep=self.keep, sum_eps=self.sum_eps,
                     softmax=self.softmax, group_best=self.group_best, correction=self.correction)
 
-    def _combine(self, rows, place, y, x, ids, wts, scaled: bool):
-        """The choices summed; ``scaled``: the rows carry their weights already."""
+    def _combine(self, rows, place, y, x, ids, wts, scaled: bool, fork, beside):
+        """The choices (and what ran beside them) summed; ``scaled``: the rows carry their weights
+        already."""
+        if fork is not None:
+            fork.join()
         ops.moe_combine(rows, place, self.top, y, wts=None if scaled else wts,
-                        identity=(ids, self.E, wts, x) if self.identities else None)
+                        identity=(ids, self.E, wts, x) if self.identities else None, plus=beside)
 
-    def _plain_experts(self, x, ids, wts, y):
+    def _plain_experts(self, x, ids, wts, y, fork, beside):
         """Experts without a gate: the activation sits in the first product's epilogue."""
         T, H = x.shape
         dev, P = x.device, T * self.top
@@ -202,7 +214,7 @@ class RoutedExperts(Part):
             rows = torch.empty((P, H), dtype=torch.float32, device=dev)
             ops.moe_gemv(x, self.w_up, act, self.top, mode, 1 if on_input else 0, ids, wts)
             ops.moe_gemv(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, ids, wts)
-            self._combine(rows, None, y, x, ids, wts, True)
+            self._combine(rows, None, y, x, ids, wts, True, fork, beside)
             return
         if self.dtype == torch.bfloat16 and ops.moe_tc_supported(x, self.w_up, self.w_down,
                                                                  gated=False):
@@ -217,7 +229,7 @@ class RoutedExperts(Part):
             ops.gemm_tc_act_grouped(xs, self.w_up, act, tile_expert, used, self.activation)
             rows = torch.empty((rows_pad, H), dtype=torch.float32, device=dev)
             ops.gemm_tc_grouped(act, self.w_down, rows, tile_expert, used)
-            self._combine(rows, place, y, x, ids, wts, on_input)
+            self._combine(rows, place, y, x, ids, wts, on_input, fork, beside)
             return
         tiles = ops.moe_max_tiles(P, self.E)
         idx = torch.empty(self.E + 1 + 2 * P + 2 * tiles, dtype=torch.int32, device=dev)
@@ -232,9 +244,9 @@ class RoutedExperts(Part):
                      tile_expert, tile_row0)
         ops.moe_gemm(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, wts, order,
                      offsets, tile_expert, tile_row0)
-        self._combine(rows, place, y, x, ids, wts, True)
+        self._combine(rows, place, y, x, ids, wts, True, fork, beside)
 
-    def _gated_experts(self, x, ids, wts, y):
+    def _gated_experts(self, x, ids, wts, y, fork, beside):
         T, H = x.shape
         dev, P = x.device, T * self.top
         on_input = self.weight_on == "input"
@@ -244,7 +256,7 @@ class RoutedExperts(Part):
             rows = torch.empty((P, H), dtype=torch.float32, device=dev)
             ops.moe_gemv(x, self.w_gu, act, self.top, 0, 1 if on_input else 0, ids, wts)
             ops.moe_gemv(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, ids, wts)
-            self._combine(rows, None, y, x, ids, wts, True)
+            self._combine(rows, None, y, x, ids, wts, True, fork, beside)
             return
         if self.w_gu_blocks is not None and ops.moe_tc_supported(x, self.w_gu_blocks, self.w_down):
             # many pairs, bfloat16: the tcgen05 product in its grouped mode over rows sorted
@@ -260,7 +272,7 @@ class RoutedExperts(Part):
             ops.gemm_tc_silu_grouped(xs, self.w_gu_blocks, act, tile_expert, used)
             rows = torch.empty((rows_pad, H), dtype=torch.float32, device=dev)
             ops.gemm_tc_grouped(act, self.w_down, rows, tile_expert, used)
-            self._combine(rows, place, y, x, ids, wts, on_input)
+            self._combine(rows, place, y, x, ids, wts, on_input, fork, beside)
             return
         tiles = ops.moe_max_tiles(P, self.E)
         idx = torch.empty(self.E + 1 + 2 * P + 2 * tiles, dtype=torch.int32, device=dev)
@@ -275,7 +287,7 @@ class RoutedExperts(Part):
                      tile_expert, tile_row0)
         ops.moe_gemm(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, wts, order,
                      offsets, tile_expert, tile_row0)
-        self._combine(rows, place, y, x, ids, wts, True)
+        self._combine(rows, place, y, x, ids, wts, True, fork, beside)
 
     def weight_bytes(self):
         # (the blocked copy of gate|up serves the many-pairs path and is not counted twice)

@@ -4,7 +4,8 @@ factor, ``y = sum_s scale_s * mixer_s(x)``.
 Where every side offers ``mix`` (what lies between its input and its output product) the sides share
 both products: one input product whose columns are the sides' one after the other, then each side's
 ``mix`` on its columns, leaving its result in its columns of one matrix, then ONE output product over
-all of them, which sums the sides in its 32-bit accumulator.  The factors cost nothing there: a side
+all of them, which sums the sides in its 32-bit accumulator.  In a step of few tokens the last
+side's kernels run on a stream of their own beside the others'.  The factors cost nothing: a side
 takes its own as ``out_scale`` and applies it where it writes in 32-bit anyway.  Other mixers run one
 after the other and their outputs are scaled and added.
 
@@ -18,6 +19,7 @@ from ..config.spec import PartSpec
 from ..csrc import ops
 from .base import Part, build_part, lookup_part, register_part
 from .linear import linear_few
+from .side_stream import Fork, forks
 
 _apart = False
 
@@ -104,8 +106,18 @@ class ParallelMixers(Part):
         proj = linear_few(x, self.w_in, out_dtype=torch.float32)
         make = torch.zeros if self.padded else torch.empty     # (columns of zeros stay zero)
         o = make((ctx.T, self.o_dim), dtype=self.dtype, device=x.device)
-        for side, c, (r0, r1), (a, b) in zip(self.sides, caches, self.rows, self.cols):
-            side.mix(proj[:, r0:r1], ctx, c, o[:, a:b])
+        run = [lambda s=side, c=c, r=r, k=k: s.mix(proj[:, r[0]:r[1]], ctx, c, o[:, k[0]:k[1]])
+               for side, c, r, k in zip(self.sides, caches, self.rows, self.cols)]
+        if forks(ctx.T):                        # few tokens: the last side beside the others
+            fork = Fork(x.device)
+            with fork:
+                run.pop()()
+            for mix in run:
+                mix()
+            fork.join()
+        else:
+            for mix in run:
+                mix()
         return linear_few(o, self.w_out, out_dtype=torch.float32)
 
     def weight_bytes(self):
