@@ -17,14 +17,13 @@ static size_t dm_smem_bytes(bool cluster, int n_stages) {
   return dm_smem_core<HD16>(cluster, n_stages) + 1024;
 }
 
-template <int HD16, bool CLUSTER>
+template <int HD16, bool CLUSTER, bool POOLED>
 static int launch_dm(const CUtensorMap& mk, const CUtensorMap& mv, const void* q, int ldq,
                      const int* table, int table_stride, const int* tok_pos, const int* tok_seq,
                      const int* seq_slot, int nh, int nkv, float scale_log2, int window,
                      float* part_o, float* part_ml, void* out, int ldo, int* counters,
                      unsigned int* fault, dim3 grid, cudaStream_t st, const float* sink,
-                     DistanceBias bias, const CUtensorMap& mpk, const CUtensorMap& mpv,
-                     const PooledKeys& pooled) {
+                     DistanceBias bias, const PooledTiles<POOLED>& pool) {
   // Few CTAs (at most two per SM) walk many tiles each: a deeper ring keeps more of the cache
   // in flight per CTA, as long as two CTAs still fit an SM.
   static int sm_count = 0;
@@ -42,7 +41,7 @@ static int launch_dm(const CUtensorMap& mk, const CUtensorMap& mv, const void* q
   const size_t smem = dm_smem_bytes<HD16>(CLUSTER, n_stages);
   static size_t configured = 0;
   if (smem > configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_decode_mma_kernel<HD16, CLUSTER>,
+    cudaError_t e = cudaFuncSetAttribute(attn_decode_mma_kernel<HD16, CLUSTER, POOLED>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = smem;
@@ -68,9 +67,9 @@ static int launch_dm(const CUtensorMap& mk, const CUtensorMap& mv, const void* q
   }
   count_variant(CLUSTER ? kVarDecodeCluster : kVarDecodeSplit);
   cudaError_t e = cudaLaunchKernelEx(
-      &cfg, attn_decode_mma_kernel<HD16, CLUSTER>, mk, mv, (const __nv_bfloat16*)q, ldq, table,
+      &cfg, attn_decode_mma_kernel<HD16, CLUSTER, POOLED>, mk, mv, (const __nv_bfloat16*)q, ldq, table,
       table_stride, tok_pos, tok_seq, seq_slot, nh, nkv, scale_log2, window, part_o, part_ml,
-      (__nv_bfloat16*)out, ldo, counters, fault, g_dm_stamps, n_stages, sink, bias, mpk, mpv, pooled);
+      (__nv_bfloat16*)out, ldo, counters, fault, g_dm_stamps, n_stages, sink, bias, pool);
   return e == cudaSuccess ? launch_status() : (int)e;
 }
 
@@ -141,7 +140,6 @@ extern "C" int cretif_attn_decode_mma_pooled(
   if (B <= 0) return kOk;
   if (pool_table && (!pool_k || !pool_v || pool <= 0 || window <= 0 || pool_blocks <= 0))
     return kBadArgument;
-  const PooledKeys pooled{pool_k, pool_v, pool_table, pool_stride, pool > 0 ? pool : 1, pool_blocks};
   if ((bias_near != nullptr) != (bias_far != nullptr) || (bias_near && n_far < 1) ||
       head_groups < 1 || B % head_groups || (bias_near && bias_slope))
     return kBadArgument;
@@ -158,32 +156,34 @@ extern "C" int cretif_attn_decode_mma_pooled(
   CUtensorMap mk, mv;
   if (make_tile_map_bf16(&mk, kc, (int)cache_rows, hd, hd, kDmTile)) return kBadArgument;
   if (make_tile_map_bf16(&mv, vc, (int)cache_rows, hd, hd, kDmTile)) return kBadArgument;
-  CUtensorMap mpk = mk, mpv = mv;               // (not read without entries)
-  if (pool_table && (make_tile_map_bf16(&mpk, pool_k, (int)pool_rows, hd, hd, kDmTile) ||
-                     make_tile_map_bf16(&mpv, pool_v, (int)pool_rows, hd, hd, kDmTile)))
-    return kBadArgument;
+  PooledTiles<true> with;
+  const PooledTiles<false> without;
+  if (pool_table) {
+    if (make_tile_map_bf16(&with.map_k, pool_k, (int)pool_rows, hd, hd, kDmTile) ||
+        make_tile_map_bf16(&with.map_v, pool_v, (int)pool_rows, hd, hd, kDmTile))
+      return kBadArgument;
+    with.keys = PooledKeys{pool_k, pool_v, pool_table, pool_stride, pool, pool_blocks};
+  }
   const float scale_log2 = scale * 1.4426950408889634f;
   dim3 grid(n_splits, nkv, B);
   cudaStream_t st = (cudaStream_t)stream;
   // Without scratch the ranges are merged inside a cluster (at most eight of them).
   const bool cluster = part_o == nullptr;
   if (cluster ? n_splits > kDmClusterMax : (!part_ml || !counters)) return kBadArgument;
-#define CRETIF_DM(N)                                                                          \
-  case N:                                                                                     \
-    return cluster                                                                            \
-               ? launch_dm<N, true>(mk, mv, q, ldq, table, table_stride, tok_pos, tok_seq,    \
-                                    seq_slot, nh, nkv, scale_log2, window, part_o, part_ml,   \
-                                    out, ldo, counters, fault, grid, st, sink, bias, mpk,     \
-                                    mpv, pooled)                                              \
-               : launch_dm<N, false>(mk, mv, q, ldq, table, table_stride, tok_pos, tok_seq,   \
-                                     seq_slot, nh, nkv, scale_log2, window, part_o, part_ml,  \
-                                     out, ldo, counters, fault, grid, st, sink, bias, mpk,    \
-                                     mpv, pooled)
+#define CRETIF_DM_L(N, CL, P, PO)                                                              \
+  launch_dm<N, CL, P>(mk, mv, q, ldq, table, table_stride, tok_pos, tok_seq, seq_slot, nh, nkv, \
+                       scale_log2, window, part_o, part_ml, out, ldo, counters, fault, grid, st, \
+                       sink, bias, PO)
+#define CRETIF_DM(N)                                                                           \
+  case N:                                                                                      \
+    if (pool_table) return cluster ? CRETIF_DM_L(N, true, true, with) : CRETIF_DM_L(N, false, true, with); \
+    return cluster ? CRETIF_DM_L(N, true, false, without) : CRETIF_DM_L(N, false, false, without)
   switch (hd / 16) {
     CRETIF_DM(1); CRETIF_DM(2); CRETIF_DM(3); CRETIF_DM(4);
     CRETIF_DM(5); CRETIF_DM(6); CRETIF_DM(7); CRETIF_DM(8);
   }
 #undef CRETIF_DM
+#undef CRETIF_DM_L
   return kBadArgument;
 }
 

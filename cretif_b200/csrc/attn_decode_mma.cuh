@@ -108,7 +108,16 @@ struct DistanceBias {
   const float* slope_;      // [heads], times log2 e: n times it is taken off instead of a table
 };
 
-template <int HD16, bool CLUSTER = false>
+// What a launch with pooled entries carries beyond the others (which do not pay for its arguments).
+template <bool POOLED>
+struct PooledTiles {
+  CUtensorMap map_k, map_v;
+  PooledKeys keys;
+};
+template <>
+struct PooledTiles<false> {};
+
+template <int HD16, bool CLUSTER = false, bool POOLED = false>
 __device__ __forceinline__ void attn_decode_mma_item(
     unsigned char* smem, const CUtensorMap* map_k, const CUtensorMap* map_v,
     const __nv_bfloat16* __restrict__ q, int ldq, const int* __restrict__ table, int table_stride,
@@ -119,8 +128,7 @@ __device__ __forceinline__ void attn_decode_mma_item(
     int n_splits, int kvh, int b, uint32_t& it_base, unsigned long long* stamps = nullptr,
     int n_stages = kDmStages, const float* sink = nullptr,
     DistanceBias bias = DistanceBias{nullptr, nullptr, 0, 1, nullptr},
-    const CUtensorMap* map_pk = nullptr, const CUtensorMap* map_pv = nullptr,
-    PooledKeys pooled = PooledKeys{nullptr, nullptr, nullptr, 0, 1, 0}) {
+    const PooledTiles<POOLED>* pool = nullptr) {
   if (bias.head_groups > 1) {           // this item's heads start at head0 of the model's
     const int head0 = (b % bias.head_groups) * nh;
     if (sink) sink += head0;
@@ -178,9 +186,16 @@ __device__ __forceinline__ void attn_decode_mma_item(
   const int first_key = first_visible_key(pos, window);
   const int first_tile = first_key / kDmTile;
   // tiles 0 .. pool_tiles - 1 of the item's list hold pooled entries, the rest the window's keys
-  const int n_pooled = pooled.table ? visible_pooled(pos, window, pooled.pool) : 0;
-  const int pool_tiles = (n_pooled + kDmTile - 1) / kDmTile;
-  const int* ptab = pooled.table + (size_t)slot * pooled.table_stride;
+  int n_pooled = 0, pool_tiles = 0;
+  const int* ptab = nullptr;
+  const CUtensorMap *map_pk = map_k, *map_pv = map_v;
+  if constexpr (POOLED) {
+    n_pooled = visible_pooled(pos, window, pool->keys.pool);
+    pool_tiles = (n_pooled + kDmTile - 1) / kDmTile;
+    ptab = pool->keys.table + (size_t)slot * pool->keys.table_stride;
+    map_pk = &pool->map_k;
+    map_pv = &pool->map_v;
+  }
   const int shift = first_tile - pool_tiles;             // list index + shift = the window's tile
   // the tiles are dealt out evenly: the first (tiles % ranges) ranges take one more
   const int span = pos / kDmTile + 1 - shift, per = span / n_splits, extra = span - per * n_splits;
@@ -209,7 +224,7 @@ __device__ __forceinline__ void attn_decode_mma_item(
     int st = (int)(it_base % (uint32_t)n_stages), turn = (int)(it_base / (uint32_t)n_stages);
     for (int i0 = 0; i0 < my_tiles; i0 += 32) {
       const int at = t_begin + i0 + lane;
-      const int mine = i0 + lane < my_tiles ? (at < pool_tiles ? ptab[at] : tab[at + shift]) : 0;
+      const int mine = i0 + lane < my_tiles ? (POOLED && at < pool_tiles ? ptab[at] : tab[at + shift]) : 0;
       const int n = min(32, my_tiles - i0);
       if (stamping && mine >= -1) stamp(threadIdx.x >> 5, 2);
       bool go = true;
@@ -227,7 +242,7 @@ __device__ __forceinline__ void attn_decode_mma_item(
           } else {
             if (blk < 0) atomicOr(fault, kFaultBlockTable);
             const int row = (max(blk, 0) * nkv + kvh) * kDmTile;
-            const bool entries = t_begin + i < pool_tiles;
+            const bool entries = POOLED && t_begin + i < pool_tiles;
             const CUtensorMap* mk = entries ? map_pk : map_k;
             const CUtensorMap* mv = entries ? map_pv : map_v;
             tc::mbar_expect_tx(&full[s], 2u * kTileBytes);
@@ -294,7 +309,7 @@ __device__ __forceinline__ void attn_decode_mma_item(
         }
       }
       // ---- online softmax of row r over this thread's 4 keys (and the quad's 16)
-      const bool entries = t_begin + i < pool_tiles;
+      const bool entries = POOLED && t_begin + i < pool_tiles;
       const int key0 = (t_begin + i + (entries ? 0 : shift)) * kDmTile + warp * 16;
       const int key_lo = entries ? 0 : first_key, key_hi = entries ? n_pooled - 1 : pos;
       float t4[4];
@@ -550,7 +565,7 @@ __device__ __forceinline__ void dm_init(unsigned char* smem, int n_stages = kDmS
   __syncthreads();
 }
 
-template <int HD16, bool CLUSTER>
+template <int HD16, bool CLUSTER, bool POOLED>
 __global__ void __launch_bounds__(kDmThreads)
 attn_decode_mma_kernel(const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v,
@@ -562,8 +577,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap map_k,
                        __nv_bfloat16* __restrict__ out, int ldo, int* __restrict__ counters,
                        unsigned int* __restrict__ fault, unsigned long long* stamps,
                        int n_stages, const float* __restrict__ sink, DistanceBias bias,
-                       const __grid_constant__ CUtensorMap map_pk,
-                       const __grid_constant__ CUtensorMap map_pv, PooledKeys pooled) {
+                       const __grid_constant__ PooledTiles<POOLED> pool) {
   extern __shared__ unsigned char smem_raw[];
   if (kStamps && stamps && blockIdx.x + blockIdx.y + blockIdx.z == 0 && threadIdx.x == 0) {
     unsigned long long t;
@@ -576,11 +590,10 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap map_k,
   dm_init<HD16>(smem, n_stages);
   if (CLUSTER) cluster_arrive();      // "this CTA runs": waited for before anything is sent
   uint32_t it_base = 0;
-  attn_decode_mma_item<HD16, CLUSTER>(smem, &map_k, &map_v, q, ldq, table, table_stride, tok_pos,
-                                      tok_seq, seq_slot, nh, nkv, scale_log2, window, part_o,
-                                      part_ml, out, ldo, counters, fault, blockIdx.x, gridDim.x,
-                                      blockIdx.y, blockIdx.z, it_base, stamps, n_stages, sink,
-                                      bias, &map_pk, &map_pv, pooled);
+  attn_decode_mma_item<HD16, CLUSTER, POOLED>(
+      smem, &map_k, &map_v, q, ldq, table, table_stride, tok_pos, tok_seq, seq_slot, nh, nkv,
+      scale_log2, window, part_o, part_ml, out, ldo, counters, fault, blockIdx.x, gridDim.x,
+      blockIdx.y, blockIdx.z, it_base, stamps, n_stages, sink, bias, &pool);
 }
 
 }  // namespace cretif
