@@ -226,6 +226,16 @@ pool_kv_kernel(const T* kc, const T* vc, const int* __restrict__ table, int tabl
 
 // VEC: four channels a thread (head size, rotated part and addresses allow it).  NT threads a token:
 // a step of few tokens takes 1024, so that a row is one turn of loads, prompts take 256.
+__device__ __forceinline__ float4 hn_ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void hn_st4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void hn_st4(__nv_bfloat16* p, const float4& v) {
+  __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<uint32_t*>(&lo);
+  u.y = *reinterpret_cast<uint32_t*>(&hi);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+
 template <typename T, bool VEC, int NT>
 __global__ void __launch_bounds__(NT)
 projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
@@ -252,12 +262,15 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
     blk = table[(size_t)slot * table_stride + pos / bt];
     if (blk < 0 && tid == 0) atomicOr(fault, kFaultBlockTable);
   }
-  // the thread's first value column and the weights of its first turn, before the row's sums are known
-  const float v_first = tid < nkv * vd ? row[nqk + tid] + (bias ? bias[nqk + tid] : 0.f) : 0.f;
   const int half = rot_dim >> 1;
   const float* c = cos_t + (size_t)pos * half;
   const float* s = sin_t + (size_t)pos * half;
   if (VEC) {
+    // (few tokens: what the thread's first turn reads after the row's sums are known)
+    if (NT > 256 && 4 * tid < nkv * vd) {
+      asm volatile("prefetch.global.L1 [%0];" ::"l"(row + nqk + 4 * tid));
+      if (bias) asm volatile("prefetch.global.L1 [%0];" ::"l"(bias + nqk + 4 * tid));
+    }
     if (NT > 256 && 4 * tid < nqk) {
       const int i = 4 * tid % hd;
       asm volatile("prefetch.global.L1 [%0];" ::"l"(4 * tid < nq ? wq + 4 * tid : wk + 4 * tid - nq));
@@ -301,38 +314,35 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
     return kc + (((size_t)blk * nkv + kvh) * bt + pos % bt) * hd + i;
   };
   if (VEC) {
+    auto normed4 = [&](int idx) {
+      float4 x = hn_ld4(row_s + idx);
+      const bool is_q = idx < nq;
+      const float4 w = hn_ld4(is_q ? wq + idx : wk + idx - nq);
+      const float f = is_q ? fq : fk;
+      x.x *= f * w.x; x.y *= f * w.y; x.z *= f * w.z; x.w *= f * w.w;
+      return x;
+    };
     for (int idx = 4 * tid; idx < n_write; idx += 4 * NT) {
       const int i = idx % hd;
-      float v[4];
-#pragma unroll
-      for (int u = 0; u < 4; ++u) v[u] = normed(idx + u);
+      float4 v = normed4(idx);
       if (i < rot_dim) {
         if (pairing) {
           const int j = i >> 1;
-          const float c0 = c[j], s0 = s[j], c1 = c[j + 1], s1 = s[j + 1];
-          const float a = v[0], b = v[1], d = v[2], e = v[3];
-          v[0] = a * c0 - b * s0; v[1] = b * c0 + a * s0;
-          v[2] = d * c1 - e * s1; v[3] = e * c1 + d * s1;
+          const float2 c2 = *reinterpret_cast<const float2*>(c + j);
+          const float2 s2 = *reinterpret_cast<const float2*>(s + j);
+          v = make_float4(v.x * c2.x - v.y * s2.x, v.y * c2.x + v.x * s2.x,
+                          v.z * c2.y - v.w * s2.y, v.w * c2.y + v.z * s2.y);
         } else {
           const bool first = i < half;
           const int j = first ? i : i - half;
-#pragma unroll
-          for (int u = 0; u < 4; ++u) {
-            const float other = normed(idx + u + (first ? half : -half));
-            v[u] = first ? v[u] * c[j + u] - other * s[j + u] : v[u] * c[j + u] + other * s[j + u];
-          }
+          const float4 c4 = hn_ld4(c + j), o = normed4(idx + (first ? half : -half));
+          float4 s4 = hn_ld4(s + j);
+          if (first) s4 = make_float4(-s4.x, -s4.y, -s4.z, -s4.w);
+          v = make_float4(v.x * c4.x + o.x * s4.x, v.y * c4.y + o.y * s4.y, v.z * c4.z + o.z * s4.z,
+                          v.w * c4.w + o.w * s4.w);
         }
       }
-      T* dst = target(idx, i);
-      if constexpr (sizeof(T) == 2) {
-        __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
-        uint2 u2;
-        u2.x = *reinterpret_cast<uint32_t*>(&lo);
-        u2.y = *reinterpret_cast<uint32_t*>(&hi);
-        *reinterpret_cast<uint2*>(dst) = u2;
-      } else {
-        *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
-      }
+      hn_st4(target(idx, i), v);
     }
   } else {
     for (int idx = tid; idx < n_write; idx += NT) {
@@ -349,9 +359,20 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
     }
   }
   if (!write_cache || blk < 0) return;
-  for (int idx = tid; idx < nkv * vd; idx += NT) {
+  const bool vec_v = VEC && (vd & 3) == 0 && (reinterpret_cast<uintptr_t>(vc) & 15) == 0;
+  for (int idx = 4 * tid; vec_v && idx < nkv * vd; idx += 4 * NT) {
     const int kvh = idx / vd, i = idx - kvh * vd;
-    const float v = idx == tid ? v_first : row[nqk + idx] + (bias ? bias[nqk + idx] : 0.f);
+    float4 v = hn_ld4(row + nqk + idx);
+    if (bias) {
+      const float4 b4 = hn_ld4(bias + nqk + idx);
+      v.x += b4.x; v.y += b4.y; v.z += b4.z; v.w += b4.w;
+    }
+    v.x *= v_scale; v.y *= v_scale; v.z *= v_scale; v.w *= v_scale;
+    hn_st4(vc + (((size_t)blk * nkv + kvh) * bt + pos % bt) * vd + i, v);
+  }
+  for (int idx = tid; !vec_v && idx < nkv * vd; idx += NT) {
+    const int kvh = idx / vd, i = idx - kvh * vd;
+    const float v = row[nqk + idx] + (bias ? bias[nqk + idx] : 0.f);
     vc[(((size_t)blk * nkv + kvh) * bt + pos % bt) * vd + i] = from_float<T>(v * v_scale);
   }
   if (pool_table && (pos + 1) % pool == 0) {       // (one token a sequence: this one ends a block)
@@ -521,7 +542,8 @@ extern "C" int cretif_projnorm_rope_kv_append(
   if (smem > 200 * 1024) return kBadArgument;
   const bool vec = hd % 4 == 0 && ldp % 4 == 0 && ldq % 4 == 0 &&
                    (pairing ? rot_dim % 4 == 0 : rot_dim % 8 == 0) &&
-                   (((uintptr_t)proj | (uintptr_t)bias | (uintptr_t)q_out | (uintptr_t)kc) & 15) == 0;
+                   (((uintptr_t)proj | (uintptr_t)bias | (uintptr_t)q_out | (uintptr_t)kc | (uintptr_t)wq |
+                     (uintptr_t)wk | (uintptr_t)cos_t | (uintptr_t)sin_t) & 15) == 0;
   cudaStream_t st = (cudaStream_t)stream;
 #define CRETIF_PN(TT, VEC)                                                                        \
   do {                                                                                            \

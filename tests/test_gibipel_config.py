@@ -273,3 +273,24 @@ def test_identities_and_weights():
     y = plain.routed(h, W, "p.", mlp)                             # equal scores: identity 2, expert 0
     for t in range(2):
         assert torch.allclose(y[t], 0.5 * h[t] + 0.5 * plain.gated(h[t], W, "p.e0."))
+
+
+def test_the_bench_configurations_build():
+    import importlib.util
+    import os
+    path = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "bench.py")
+    mod_spec = importlib.util.spec_from_file_location("bench_for_gibipel", path)
+    bench = importlib.util.module_from_spec(mod_spec)
+    mod_spec.loader.exec_module(bench)
+    for z in bench.DESIGN_SIZES.values():
+        configs = bench.gibipel_configs(z, 4)
+        assert {"virorax attention", "virorax retention", "losorax attention routed"} < set(configs)
+        for name, cfg in configs.items():
+            if name.startswith("gibipel"):
+                spec = _spec(cfg)
+                spec.validate()
+                assert len(spec.schedule) == 4 and spec.architecture == "Gibipel"
+                left = cfg["layers"][0]["mixer"]["left"]
+                other = configs["virorax attention"]["layers"][0]["mixer"]
+                assert all(left[k] == other[k] for k in ("heads", "kv_heads", "dim", "vdim", "scale"))
+                assert left["mask"]["size"] == other["mask"]["size"]
