@@ -15,8 +15,9 @@ by; ``scores: "softmax"`` takes the softmax over all router outputs instead of t
 function; ``correction`` names a tensor with a number per router output that is added to the scores
 for the choice alone; a group's score is then that of its choice scores, and ``groups`` may say
 ``"score": "best"`` for the largest instead of the sum of two; ``identities`` appends that many router
-outputs that are no experts: their output is the input itself; ``shared`` (``{"intermediate_size", "names"}``) is one more expert of the same form that every
-token uses with weight one.
+outputs that are no experts: their output is the input itself; ``shared``
+(``{"intermediate_size", "names"}``) is one more expert of the same form that every token uses with
+weight one.
 
 The step's (token, choice) pairs are sorted by expert on the device and each expert's rows
 are one slice of two grouped products (csrc/moe.cu): gate|up with the activation — and the

@@ -269,8 +269,8 @@ def test_norms_over_whole_projections_rotation_cache_write_and_entries(dtype, H,
 
 
 def _attention_case(H, G, d, e, window, P, S, seed):
-    """Queries, keys and values in which, for every query, the first and the last thing it sees and
-    the first things it does not see stand out."""
+    """Queries, keys and values with a key in seven that stands out: for some queries it is the last
+    one their window or a visible block still shows, for others the first one that is not seen."""
     g = torch.Generator().manual_seed(seed)
     q = torch.randn(S, H, d, generator=g)
     k = torch.randn(S, G, d, generator=g)
