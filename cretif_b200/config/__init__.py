@@ -8,6 +8,7 @@ from .losorax import LosoraxConfig, build_losorax_spec, losorax_config_from_dict
 from .virorax import ViroraxConfig, build_virorax_spec, virorax_config_from_dict
 from .mipurax import MipuraxConfig, build_mipurax_spec, mipurax_config_from_dict
 from .gibipel import GibipelConfig, build_gibipel_spec, gibipel_config_from_dict
+from .pudorax import PudoraxConfig, build_pudorax_spec, pudorax_config_from_dict
 from .presets import PRESETS, preset
 
 __all__ = [
@@ -20,4 +21,5 @@ __all__ = [
     "ViroraxConfig", "build_virorax_spec", "virorax_config_from_dict",
     "MipuraxConfig", "build_mipurax_spec", "mipurax_config_from_dict",
     "GibipelConfig", "build_gibipel_spec", "gibipel_config_from_dict",
+    "PudoraxConfig", "build_pudorax_spec", "pudorax_config_from_dict",
 ]

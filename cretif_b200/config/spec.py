@@ -86,12 +86,14 @@ class ScheduleEntry:
     the last inputs of a convolution, a shifted row) is always the visit's own.
     ``add_input`` adds the model's input (the embedding part's output, as it was before the
     first layer) to the residual stream once more, right before this visit: a model that runs
-    a span of layers several times over feeds each further pass that way.
+    a span of layers several times over feeds each further pass that way.  ``merge_input`` merges
+    it in instead, by the model's ``merge`` part, right before this visit.
     """
 
     layer: int
     cache: Optional[int] = None
     add_input: bool = False
+    merge_input: bool = False
 
 
 @dataclass
@@ -107,6 +109,7 @@ class ModelSpec:
     max_positions: int
     stop_token_ids: List[int] = field(default_factory=list)
     bos_token_id: Optional[int] = None
+    merge: Optional[PartSpec] = None      # how the input is merged in again (ScheduleEntry.merge_input)
 
     def validate(self) -> None:
         if self.vocab_size <= 0 or self.hidden_size <= 0:
@@ -117,6 +120,9 @@ class ModelSpec:
             if not 0 <= e.layer < len(self.layers):
                 raise ValueError(f"schedule entry {i} names layer {e.layer}, "
                                  f"but the model has {len(self.layers)} layers")
+            if e.merge_input and self.merge is None:
+                raise ValueError(f"schedule entry {i} merges the model's input in, but the model has no "
+                                 "merge part")
             for b in self.layers[e.layer].branches:
                 if b.role not in ("mixer", "feed_forward"):
                     raise ValueError(f"layer {e.layer}: a branch's role is 'mixer' or "

@@ -25,7 +25,15 @@ int cretif_add_rmsnorm(float* h, const void* delta, int delta_dt, const float* w
 
 // act[t, i] = silu(gate) * up; block = 0: gu row = [gate | up]; block = b: groups of b gate
 // columns followed by their b up columns.
-int cretif_silu_mul(const void* gu, void* act, int dt, int T, int I, int block, void* stream);
+// limit > 0: a clamped gate instead (GateRule in common.cuh; slope and offset are its others).
+int cretif_silu_mul(const void* gu, void* act, int dt, int T, int I, int block, float limit,
+                    float slope, float offset, void* stream);
+
+// v = h[src] (+ delta[src]); if write_h, h[src] = v;
+// out[r] = (v - mean(v)) * rsqrt(mean((v - mean(v))^2) + eps) * weight + bias.  As cretif_add_rmsnorm.
+int cretif_add_layernorm(float* h, const void* delta, int delta_dt, const float* weight,
+                         const float* bias, void* out, int out_dt, const int* rows, int R, int H,
+                         float eps, int write_h, void* stream);
 
 // Rotate q and k of every token by its position's angles (pairing 0: (j, j+rot/2),
 // 1: (2j, 2j+1)); q in place.  write_cache bit 0: rotated k and v into the block cache;
@@ -43,6 +51,8 @@ int cretif_rmsnorm_add(float* h, const void* y, int y_dt, int ldy, const float* 
 
 // out = h converted to the element type out_dt (the stream handed to a sublayer without a norm).
 int cretif_convert_rows(const float* h, void* out, int out_dt, long long total, void* stream);
+// ... into columns of a wider matrix: out row r starts at out + r * ldo.
+int cretif_convert_into(const float* h, void* out, int out_dt, int ldo, int R, int H, void* stream);
 
 // rows [T, ld] = [q (q_dim) | k (nkv * hd) | ...].  With wq: q <- rmsnorm over all q_dim columns
 // times wq, in place.  k: rmsnorm over all nkv*hd columns times wk goes to the key cache at each
@@ -143,20 +153,22 @@ int cretif_rmsnorm_rows(float* x, int ld, const float* w, int R, int H, float ep
 // renorm: the chosen scores are divided by (their sum + sum_eps).
 int cretif_moe_route(const void* x, int x_dt, int ldx, const float* router_w, int E, int H,
                      int top, int renorm, int groups, int keep, float sum_eps, int softmax,
-                     int group_best, const float* correction, int* ids, float* wts, int T,
-                     void* stream);
+                     int group_best, const float* correction, const float* bias, int* ids,
+                     float* wts, int T, void* stream);
 int cretif_moe_topk(const float* logits, int ld, int E, int top, int renorm, int groups, int keep,
-                    float sum_eps, int softmax, int group_best, const float* correction, int* ids,
-                    float* wts, int T, void* stream);
+                    float sum_eps, int softmax, int group_best, const float* correction,
+                    const float* bias, int* ids, float* wts, int T, void* stream);
 int cretif_moe_group(const int* ids, int P, int E, int* offsets, int* place, int* order,
                      int* tile_expert, int* tile_row0, int max_tiles, void* stream);
 int cretif_moe_gemm(const void* A, int a_dt, int lda, const void* W, int w_dt, void* C, int ldc,
                     int N, int K, int top, int mode, int scale_at, const float* wts,
                     const int* order, const int* offsets, const int* tile_expert,
-                    const int* tile_row0, int max_tiles, int use_mma, void* stream);
+                    const int* tile_row0, int max_tiles, int use_mma, float limit, float slope,
+                    float offset, void* stream);
 int cretif_moe_gemv(const void* A, int a_dt, int lda, const void* W, int w_dt, void* C, int ldc,
                     int N, int K, int top, int mode, int scale_at, const int* ids,
-                    const float* wts, int P, int experts, void* stream);
+                    const float* wts, int P, int experts, float limit, float slope, float offset,
+                    void* stream);
 int cretif_moe_group_padded(const int* ids, int P, int E, int tile, int* place, int* tile_expert,
                             int max_tiles, int* used, void* stream);
 int cretif_moe_gather_rows(const void* x, int ldx, void* xs, int lds, const int* place,
@@ -164,7 +176,8 @@ int cretif_moe_gather_rows(const void* x, int ldx, void* xs, int lds, const int*
 // place may be null: the rows are in the pairs' own order; wts may be null: no weights.
 int cretif_moe_combine(const float* rows, int ld, const int* place, int top, const float* wts,
                        float* y, int T, int H, const int* ids, int experts, const float* id_wts,
-                       const void* x, int x_dt, int ldx, const float* plus, void* stream);
+                       const void* x, int x_dt, int ldx, const float* plus, int add, void* x_out,
+                       void* stream);
 
 // After a decode step: ids <- sampled (if given), positions and lengths + 1.
 int cretif_advance_decode(int* tok_ids, int* tok_pos, int* seq_start, const int* sampled, int B,
@@ -200,6 +213,7 @@ int cretif_gemm_skinny_max_rows(void);
 // 32-bit sums before they are rounded.  A wait that expires sets bit 2 of *fault.
 int cretif_gemm_tc(const void* A, const void* W, void* C, int c_dt, int M, int N, int K, int lda,
                    int ldw, int ldc, int accumulate, int bn, float alpha, int unary,
+                   const void* mul, int mul_ld, int mul_rows, const int* mul_ids,
                    unsigned int* fault, void* stream);
 
 // (For tests that run both.)  Epilogue warps of the tensor-core product: 4 or 8; 0, the default,
@@ -219,7 +233,8 @@ int cretif_set_tc_pair(int mode);
 // matrix whose rows are interleaved in blocks of 64 (I % 64 == 0), and rotary + cache write for
 // the stacked q|k|v matrix (head_dim 64 or 128, rotary over the whole head).
 int cretif_gemm_tc_silu(const void* A, const void* Wgu, void* act, int M, int I, int K, int lda,
-                        int ldw, unsigned int* fault, void* stream);
+                        int ldw, float limit, float slope, float offset, unsigned int* fault,
+                        void* stream);
 // The same products in groups: A [M, K], M a multiple of 128, whose 128-row tiles each belong to a
 // group (tile_group[M / 128]; *used_m_tiles tiles are in use, the others are left alone), and
 // W [groups, N, K] ([groups, 2 I, K] interleaved as above); C float32 [M, N], act [M, I].
@@ -233,7 +248,8 @@ int cretif_gemm_tc_act_grouped(const void* A, const void* W, void* C, int M, int
                                void* stream);
 int cretif_gemm_tc_silu_grouped(const void* A, const void* Wgu, void* act, int M, int I, int K,
                                 int lda, int ldw, int groups, const int* tile_group,
-                                const int* used_m_tiles, unsigned int* fault, void* stream);
+                                const int* used_m_tiles, float limit, float slope, float offset,
+                                unsigned int* fault, void* stream);
 int cretif_gemm_tc_qkv_rope(const void* A, const void* Wqkv, void* Q, int ldq, const float* cos_t,
                             const float* sin_t, int pairing, int nh, int nkv, int hd,
                             const int* tok_pos, const int* tok_seq, const int* seq_slot,
@@ -330,11 +346,13 @@ int cretif_attn_decode_mma_pooled(
 
 // Fused decode projections (see decode_fused.cu).  H is the float32 residual stream; when it
 // is given, x = bf16(rmsnorm(H[rows])) is computed in the kernel, else X (bfloat16) is read.
-// cretif_fused_linear stores or adds alpha times the product; unary as in cretif_gemm_tc.
+// cretif_fused_linear stores or adds alpha times the product; unary and mul as in cretif_gemm_tc.
+// norm_b (with H): the norm takes the mean off and adds norm_b (a layer norm).
 int cretif_fused_linear(const void* X, int ldx, const float* H, const float* norm_w,
-                        const int* rows, float eps, const void* W, int ldw, void* C, int c_dt,
-                        int ldc, int accumulate, float alpha, int unary, int M, int N, int K,
-                        unsigned int* fault, void* stream);
+                        const float* norm_b, const int* rows, float eps, const void* W, int ldw,
+                        void* C, int c_dt, int ldc, int accumulate, float alpha, int unary,
+                        const void* mul, int mul_ld, int mul_rows, const int* mul_ids, int M, int N,
+                        int K, unsigned int* fault, void* stream);
 int cretif_fused_qkv_rope(const float* H, const float* norm_w, float eps, const void* Wqkv, int ldw,
                           void* Q, int ldq, const float* cos_t, const float* sin_t, int pairing,
                           int nh, int nkv, int hd, const int* tok_pos, const int* tok_seq,
@@ -342,10 +360,12 @@ int cretif_fused_qkv_rope(const float* H, const float* norm_w, float eps, const 
                           void* vc, int bt, int write_cache, int M, int K, unsigned int* fault,
                           void* stream);
 int cretif_fused_gate_up_silu(const float* H, const float* norm_w, float eps, const void* Wgu,
-                              int ldw, void* act, int I, int gu_block, int M, int K,
-                              unsigned int* fault, void* stream);
+                              int ldw, void* act, int I, int gu_block, float limit, float slope,
+                              float offset, int M, int K, unsigned int* fault, void* stream);
 int cretif_fused_gate_up_silu_x(const void* X, int ldx, const void* Wgu, int ldw, void* act, int I,
-                                int gu_block, int M, int K, unsigned int* fault, void* stream);
+                                int gu_block, float limit, float slope, float offset, int M, int K,
+                                unsigned int* fault, void* stream);
+// norm_prologue: 0 none, 1 an RMS norm, 2 a layer norm.
 int cretif_fused_smem_ok(int M, int K, int norm_prologue);
 // The three switches below exist so that tests can run both variants of a kernel on one
 // shape; an ordinary run never touches them.
@@ -419,7 +439,8 @@ int cretif_gate_heads(void* o, int ldo, int dt, const float* g, int ldg, int nh,
 // out = act(in) element by element: kind 0 relu(z)^2, 1 gelu in its tanh form, 2 silu,
 // 3 gelu with the error function.
 int cretif_activation(const void* in, int ldi, int in_dt, void* out, int ldo, int out_dt, int T,
-                      int width, int kind, void* stream);
+                      int width, int kind, const void* mul, int mul_ld, int mul_rows,
+                      const int* mul_ids, void* stream);
 // z <- cap * tanh(z / cap) in place.
 int cretif_softcap(float* z, long long total, float cap, void* stream);
 // z <- factor * z, in place.
@@ -437,7 +458,8 @@ int cretif_projnorm_rope_kv_append(
     const int* tok_seq, const int* seq_slot, int nh, int nkv, int hd, int vd, float v_scale,
     void* q_out, int ldq, int dt, const int* table, int table_stride, void* kc, void* vc, int bt,
     int write_cache, void* pool_k, void* pool_v, const int* pool_table, int pool_stride, int pool,
-    int T, unsigned int* fault, void* stream);
+    const float* conv_w, int taps, float* conv_state, long long conv_stride, const int* seq_start,
+    int save_inputs, int T, unsigned int* fault, void* stream);
 
 // Matrix memory with exponential gates (matrix_memory.cu): proj rows (float32) [q (H d) | k (H d) |
 // v (H e) | gate (H e) | z_i (H) | z_f (H) | ...] -> out [T, H e], the normed and gated read-outs; a
@@ -449,6 +471,20 @@ int cretif_matrix_memory(const float* proj, int ldp, const float* bias_i, const 
                          int d, int e, const float* norm_w, float eps, float* o_raw, float* den,
                          float* ref, double* gates, void* out, int out_dt, int ldo, int write_state,
                          int T, int form, void* stream);
+
+// The Mamba-2 recurrence (state_space.cu): proj rows (float32) [z (H e) | x (H e) | B (G N) | C (G N) |
+// dt (H) | ...] -> out [T, H e], the gated and normed read-outs.  conv_w [taps, C'], conv_b [C'],
+// C' = H e + 2 G N.  A slot's state: S [H, N, e] and, at inputs_at, the last taps - 1 inputs of every
+// convolved channel.  Scratch: y [T, H e]; for chunks xbc [T, ldx >= C'], dts [H, T], sums [H, T]
+// (float64).  parts: equal parts of the H e channels that are normed on their own.  save_inputs: a step
+// of one token a sequence, whose inputs are saved here.  form: 0 chooses, 1 token by token, 2 chunks.
+int cretif_state_space(const float* proj, int ldp, const float* conv_w, const float* conv_b, int taps,
+                       const float* a_log, const float* dt_bias, const float* d_skip, float* state,
+                       long long state_stride, long long inputs_at, const int* cu_seqlens,
+                       const int* seq_slot, const int* tok_seq, int B, int H, int G, int N, int e,
+                       float* y, float* xbc, int ldx, float* dts, double* sums, int parts,
+                       const float* norm_w, float eps, void* out, int out_dt, int ldo,
+                       int write_state, int save_inputs, int T, int form, void* stream);
 
 // Retention (retention.cu).  proj rows (float32): [q (H d) | k (H d) | ...]; prep rows: the
 // rotated q and the rotated k times k_scale.  state points at the first sequence slot's

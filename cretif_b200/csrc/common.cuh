@@ -44,6 +44,33 @@ __device__ __forceinline__ float silu_bf16_path(float g) {
   return __fdividef(g, 1.0f + __expf(-g));
 }
 
+// What a gated feed-forward makes of its gate product g and its up product u.  limit 0:
+// silu(g) u.  Else the gate is clamped from above and the other product on both sides:
+//   g' / (1 + e^(-slope g')) (u' + offset),   g' = min(g, limit),  u' = clamp(u, -limit, limit).
+struct GateRule {
+  float limit, slope, offset;
+};
+__device__ __forceinline__ void gate_clamp(float& g, float& u, const GateRule& r) {
+  g = fminf(g, r.limit);
+  u = fminf(fmaxf(u, -r.limit), r.limit) + r.offset;
+}
+__device__ __forceinline__ float gate_mul(float g, float u, const GateRule& r) {
+  if (r.limit > 0.f) {
+    gate_clamp(g, u, r);
+    return g / (1.0f + expf(-r.slope * g)) * u;
+  }
+  return g / (1.0f + expf(-g)) * u;
+}
+// (the bfloat16 kernels' form, see silu_bf16_path)
+__device__ __forceinline__ float gate_mul_bf16_path(float g, float u, const GateRule& r) {
+  if (r.limit > 0.f) {
+    gate_clamp(g, u, r);
+    return __fdividef(g, 1.0f + __expf(-r.slope * g)) * u;
+  }
+  return silu_bf16_path(g) * u;
+}
+inline bool gate_rule_ok(float limit) { return limit >= 0.f; }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

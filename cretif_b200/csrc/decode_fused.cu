@@ -45,7 +45,7 @@ static int launch_fused(const FusedParams& p, int tiles, cudaStream_t st, int gr
   // give 32 rows one warp each; on a grid that fills the chip, clusters of four find their
   // places more slowly than they save (64 rows: 1.38 against 1.33 ms a step with two).
   int cluster = 1;
-  if (NT > 1 && PRO == kProNorm && g_fused_cluster > 1) {
+  if (NT > 1 && pro_is_norm(PRO) && g_fused_cluster > 1) {
     cluster = group_rows > 16 && 4 * (int)grid.x * groups <= 3 * max_ctas ? 4 : 2;
     if (cluster > g_fused_cluster) cluster = g_fused_cluster;
     if ((int)grid.x < cluster) cluster = 1;
@@ -197,22 +197,31 @@ using namespace cretif;
 
 // out (+)= norm(h[rows]) · W^T  or  x · W^T, plain epilogue.
 extern "C" int cretif_fused_linear(const void* X, int ldx, const float* H, const float* norm_w,
-                                   const int* rows, float eps, const void* W, int ldw, void* C,
-                                   int c_dt, int ldc, int accumulate, float alpha, int unary,
-                                   int M, int N, int K, unsigned int* fault, void* stream) {
+                                   const float* norm_b, const int* rows, float eps, const void* W,
+                                   int ldw, void* C, int c_dt, int ldc, int accumulate, float alpha,
+                                   int unary, const void* mul, int mul_ld, int mul_rows,
+                                   const int* mul_ids, int M, int N, int K, unsigned int* fault,
+                                   void* stream) {
   if (M <= 0 || N <= 0) return kOk;
   if (unary < 0 || unary > kUnaryKinds || (unary && accumulate)) return kBadArgument;
+  if (mul && (accumulate || !mul_ids || mul_ld < N)) return kBadArgument;
   FusedParams p = {};
   p.alpha = alpha; p.scaled = alpha != 1.0f; p.unary = unary;
   p.W = (const __nv_bfloat16*)W; p.M = M; p.N = N; p.K = K; p.ldw = ldw;
   p.X = (const __nv_bfloat16*)X; p.ldx = ldx; p.H = H; p.norm_w = norm_w; p.rows = rows;
   p.eps = eps; p.C = C; p.ldc = ldc; p.c_dt = c_dt; p.accumulate = accumulate; p.fault = fault;
+  p.norm_b = norm_b;
+  p.mul = (const __nv_bfloat16*)mul; p.mul_ids = mul ? mul_ids : nullptr; p.mul_ld = mul_ld;
+  p.mul_rows = mul_rows;
   if (!common_ok(p) || !derive_fields(p) || ldc < N || (c_dt != kF32 && c_dt != kBF16) ||
       (c_dt == kBF16 && accumulate))
     return kBadArgument;
   const int tiles = (N + kFuRows - 1) / kFuRows;
   cudaStream_t st = (cudaStream_t)stream;
-  const bool ex = p.scaled || p.unary;
+  const bool ex = p.scaled || p.unary || p.mul;
+  if (H && norm_b)
+    return ex ? dispatch_nt<kProLayer, kEpiPlainEx>(p, tiles, st)
+              : dispatch_nt<kProLayer, kEpiPlain>(p, tiles, st);
   if (H)
     return ex ? dispatch_nt<kProNorm, kEpiPlainEx>(p, tiles, st)
               : dispatch_nt<kProNorm, kEpiPlain>(p, tiles, st);
@@ -247,11 +256,14 @@ extern "C" int cretif_fused_qkv_rope(const float* H, const float* norm_w, float 
 // act = silu(norm(h) · Wg^T) * (norm(h) · Wu^T), Wgu = [Wg; Wu] stacked.
 extern "C" int cretif_fused_gate_up_silu(const float* H, const float* norm_w, float eps,
                                          const void* Wgu, int ldw, void* act, int I, int gu_block,
-                                         int M, int K, unsigned int* fault, void* stream) {
+                                         float limit, float slope, float offset, int M, int K,
+                                         unsigned int* fault, void* stream) {
   if (M <= 0) return kOk;
+  if (!gate_rule_ok(limit)) return kBadArgument;
   FusedParams p = {};
   p.W = (const __nv_bfloat16*)Wgu; p.M = M; p.N = 2 * I; p.K = K; p.ldw = ldw;
   p.H = H; p.norm_w = norm_w; p.eps = eps; p.act = (__nv_bfloat16*)act; p.I = I; p.gu_block = gu_block; p.fault = fault;
+  p.gate = GateRule{limit, slope, offset};
   if (!common_ok(p) || !derive_fields(p) || !H || I <= 0 || gu_block < 0 ||
       (gu_block && (I % gu_block || gu_block % 8)))
     return kBadArgument;
@@ -261,13 +273,16 @@ extern "C" int cretif_fused_gate_up_silu(const float* H, const float* norm_w, fl
 // The same from rows that are already in bfloat16 (a feed-forward that reads the stream itself,
 // without a norm in front of it).
 extern "C" int cretif_fused_gate_up_silu_x(const void* X, int ldx, const void* Wgu, int ldw,
-                                           void* act, int I, int gu_block, int M, int K,
-                                           unsigned int* fault, void* stream) {
+                                           void* act, int I, int gu_block, float limit, float slope,
+                                           float offset, int M, int K, unsigned int* fault,
+                                           void* stream) {
   if (M <= 0) return kOk;
+  if (!gate_rule_ok(limit)) return kBadArgument;
   FusedParams p = {};
   p.W = (const __nv_bfloat16*)Wgu; p.M = M; p.N = 2 * I; p.K = K; p.ldw = ldw;
   p.X = (const __nv_bfloat16*)X; p.ldx = ldx;
   p.act = (__nv_bfloat16*)act; p.I = I; p.gu_block = gu_block; p.fault = fault;
+  p.gate = GateRule{limit, slope, offset};
   if (!common_ok(p) || !derive_fields(p) || !X || ldx % 8 || ldx < K || (((uintptr_t)X) & 15) ||
       I <= 0 || gu_block < 0 || (gu_block && (I % gu_block || gu_block % 8)))
     return kBadArgument;
@@ -303,5 +318,5 @@ extern "C" int cretif_fused_smem_ok(int M, int K, int norm_prologue) {
   if (M > kFuMaxRows) return 0;
   if (M > kFuMaxGroupRows) M = kFuMaxGroupRows;
   const int nt = M <= 8 ? 1 : (M <= 16 ? 2 : 4);
-  return fused_smem(nt, norm_prologue ? kProNorm : kProPlain, M, K) <= 200 * 1024 ? 1 : 0;
+  return fused_smem(nt, norm_prologue == 2 ? kProLayer : norm_prologue ? kProNorm : kProPlain, M, K) <= 200 * 1024 ? 1 : 0;
 }

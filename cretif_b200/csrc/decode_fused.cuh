@@ -6,6 +6,7 @@
 //                   32-bit residual stream (a few KB for a decode batch) into shared memory,
 //                   optionally from gathered rows (the rows whose logits are wanted); with
 //                   more than 8 rows the CTAs of a thread-block cluster share that work;
+//   prologue LAYER  the same with the mean taken off and a bias added: a layer norm;
 //   epilogue ROPE   the stacked q|k|v product: rotary pairs of q and k are rotated in 32-bit,
 //                   q goes to the query buffer, rotated k and v go straight into the block
 //                   cache at each token's position;
@@ -30,9 +31,10 @@ namespace cretif {
 
 constexpr int kFuWarps = 8;
 constexpr int kFuRows = 16;
-enum Prologue : int { kProPlain = 0, kProNorm = 1 };
-// kEpiPlainEx is kEpiPlain with a factor on the product and an optional activation; it is a
-// kind of its own so that the plain epilogue's code stays what it was.
+enum Prologue : int { kProPlain = 0, kProNorm = 1, kProLayer = 2 };
+__host__ __device__ constexpr bool pro_is_norm(int pro) { return pro != kProPlain; }
+// kEpiPlainEx is kEpiPlain with a factor on the product, an optional activation and an optional
+// factor per token and column from a table; it is a kind of its own so that the plain epilogue's code stays what it was.
 enum Epilogue : int { kEpiPlain = 0, kEpiRope = 1, kEpiSilu = 2, kEpiPlainEx = 3 };
 __host__ __device__ constexpr bool epi_is_plain(int epi) {
   return epi == kEpiPlain || epi == kEpiPlainEx;
@@ -68,6 +70,7 @@ struct FusedParams {
   int ldx;
   const float* H;           // norm: residual stream [*, K]
   const float* norm_w;      // [K]
+  const float* norm_b;      // [K], layer norm
   const int* rows;          // optional gather: x row m comes from H[rows[m]]
   float eps;
   // epilogue plain
@@ -75,6 +78,9 @@ struct FusedParams {
   int ldc, c_dt, accumulate;
   float alpha;              // scaled != 0: the product times alpha is what is stored or added
   int scaled, unary;        // unary: 0 none, else 1 + the kind of unary_activation (stores only)
+  const __nv_bfloat16* mul; // row m is multiplied by row mul_ids[m] of this table (stores only)
+  const int* mul_ids;
+  int mul_ld, mul_rows;     // (an id outside [0, mul_rows) multiplies by zero)
   // epilogue rope
   __nv_bfloat16* Q;         // [M, nh*hd]
   int ldq;
@@ -92,6 +98,7 @@ struct FusedParams {
   unsigned int* fault;
   // epilogue silu
   __nv_bfloat16* act;       // [M, I]
+  GateRule gate;
   int I, gu_block;          // gu_block > 0: gate/up rows interleaved in groups of that size
   // set by the launcher from the above
   FastDiv gu_div, tph_div;  // by gu_block; by tiles per head (hd / 16)
@@ -215,6 +222,11 @@ __device__ __forceinline__ void finish_tile(const FusedParams& p, int tile,
       if (EPI == kEpiPlainEx) {
         if (p.scaled) sum *= p.alpha;
         if (p.unary) sum = unary_activation(sum, p.unary - 1);
+        if (p.mul) {
+          const int id = p.mul_ids[m];
+          sum *= id >= 0 && id < p.mul_rows
+                     ? __bfloat162float(p.mul[(size_t)id * p.mul_ld + n]) : 0.f;
+        }
       }
       if (p.c_dt == kF32) {
         float* out = reinterpret_cast<float*>(p.C) + (size_t)m * p.ldc + n;
@@ -240,7 +252,7 @@ __device__ __forceinline__ void finish_tile(const FusedParams& p, int tile,
         // the unfused path stores gate and up as bfloat16 before the activation
         const float g = __bfloat162float(__float2bfloat16_rn(s0));
         const float u = __bfloat162float(__float2bfloat16_rn(s1));
-        p.act[(size_t)m * p.I + col] = __float2bfloat16_rn(silu_bf16_path(g) * u);
+        p.act[(size_t)m * p.I + col] = __float2bfloat16_rn(gate_mul_bf16_path(g, u, p.gate));
       } else {
         const int tiles_per_head = p.hd >> 4;
         const int head = fast_div(p.tph_div, tile), t = tile - head * tiles_per_head;
@@ -284,8 +296,8 @@ __device__ __forceinline__ void finish_tile(const FusedParams& p, int tile,
   }
 }
 
-// The norm prologue: x[m] = bf16(h[row m] * w * rsqrt(mean(h^2) + eps)) into shared memory, a
-// warp per token.  A row of up to 128 * REGS columns makes one trip from memory: the lane
+// The norm prologue: x[m] = bf16(h[row m] * w * rsqrt(mean(h^2) + eps)), or with LAYER
+// bf16((h - mean) * w * rsqrt(mean((h - mean)^2) + eps) + b), into shared memory, a warp per token.  A row of up to 128 * REGS columns makes one trip from memory: the lane
 // keeps its REGS float4 in registers between the sum of squares and the scaling.
 //
 // The norm's weight depends on nothing that runs before the kernel.  For K <= 1024 N the
@@ -299,9 +311,10 @@ struct NormStash {
 };
 
 template <int N>
-__device__ __forceinline__ void norm_weight_fetch(const FusedParams& p, NormStash<N>& st) {
+__device__ __forceinline__ void norm_weight_fetch(const FusedParams& p, const float* weight,
+                                                  NormStash<N>& st) {
   const int n4 = p.K >> 2;
-  const float4* w4 = reinterpret_cast<const float4*>(p.norm_w);
+  const float4* w4 = reinterpret_cast<const float4*>(weight);
 #pragma unroll
   for (int u = 0; u < N; ++u) {
     const int i = threadIdx.x + u * kFuWarps * 32;
@@ -310,15 +323,54 @@ __device__ __forceinline__ void norm_weight_fetch(const FusedParams& p, NormStas
   }
 }
 
+// Four columns of a normed row, and the sums a warp makes of its row.
+__device__ __forceinline__ float4 norm_apply(const float4& t, const float4& w, float inv) {
+  return make_float4(t.x * w.x * inv, t.y * w.y * inv, t.z * w.z * inv, t.w * w.w * inv);
+}
+__device__ __forceinline__ float4 layer_apply(const float4& t, const float4& w, const float4& b,
+                                              float mean, float inv) {
+  return make_float4((t.x - mean) * inv * w.x + b.x, (t.y - mean) * inv * w.y + b.y,
+                     (t.z - mean) * inv * w.z + b.z, (t.w - mean) * inv * w.w + b.w);
+}
+__device__ __forceinline__ uint2 pack4_bf16(const float4& y) {
+  __nv_bfloat162 lo = __floats2bfloat162_rn(y.x, y.y);
+  __nv_bfloat162 hi = __floats2bfloat162_rn(y.z, y.w);
+  uint2 pk;
+  pk.x = *reinterpret_cast<uint32_t*>(&lo);
+  pk.y = *reinterpret_cast<uint32_t*>(&hi);
+  return pk;
+}
+__device__ __forceinline__ float sum4(const float4& v) { return (v.x + v.y) + (v.z + v.w); }
+__device__ __forceinline__ float sq4(const float4& v, float mean) {
+  const float a = v.x - mean, b = v.y - mean, c = v.z - mean, d = v.w - mean;
+  return a * a + b * b + c * c + d * d;
+}
+// The mean of a row (layer norm): its lanes' float4 in v (fits), else read again.
+template <int REGS>
+__device__ __forceinline__ float row_mean(const float4 (&v)[REGS], const float4* h4, int n4, int lane,
+                                          bool fits, int K) {
+  float s = 0.f;
+  if (fits) {
+#pragma unroll
+    for (int u = 0; u < REGS; ++u) s += sum4(v[u]);        // (columns beyond the row are zero)
+  } else {
+#pragma unroll 8
+    for (int i = lane; i < n4; i += 32) s += sum4(__ldcg(h4 + i));
+  }
+  return warp_sum(s) / (float)K;
+}
+
 // Called by the kFuWarps * 32 threads that also called norm_weight_fetch; `sync` is the
 // barrier among exactly those threads, run once by each after its first loads are issued.
-template <int REGS, int N, typename Sync>
+template <int REGS, bool LAYER, int N, typename Sync>
 __device__ __forceinline__ void norm_rows_to_smem(const FusedParams& p, unsigned char* xs,
                                                   int xs_stride, int warp, int lane, float4* nws,
-                                                  const NormStash<N>& st, Sync sync) {
+                                                  const NormStash<N>& st,
+                                                  const NormStash<N>& st_b, Sync sync) {
   const int n4 = p.K >> 2;
   const bool stash = p.K <= NormStash<N>::kMaxK;
   const float4* w4 = reinterpret_cast<const float4*>(p.norm_w);
+  const float4* b4 = reinterpret_cast<const float4*>(p.norm_b);
   bool first = true;
   for (int m = warp; m < p.M || first; m += kFuWarps) {
     const bool row = m < p.M;
@@ -341,26 +393,27 @@ __device__ __forceinline__ void norm_rows_to_smem(const FusedParams& p, unsigned
         for (int u = 0; u < N; ++u) {
           const int i = warp * 32 + lane + u * kFuWarps * 32;
           if (i < n4) nws[i] = st.w[u];
+          if (LAYER && i < n4) nws[n4 + i] = st_b.w[u];
         }
       }
       sync();                 // always, and by every warp: the caller may count on it
     }
     if (!row) break;
     auto weight = [&](int i) { return stash ? nws[i] : __ldg(w4 + i); };
+    const float mean = LAYER ? row_mean(v, h4, n4, lane, fits, p.K) : 0.f;
     auto put = [&](int i, const float4& t, float inv) {
       const float4 w = weight(i);
-      __nv_bfloat162 lo = __floats2bfloat162_rn(t.x * w.x * inv, t.y * w.y * inv);
-      __nv_bfloat162 hi = __floats2bfloat162_rn(t.z * w.z * inv, t.w * w.w * inv);
-      uint2 pk;
-      pk.x = *reinterpret_cast<uint32_t*>(&lo);
-      pk.y = *reinterpret_cast<uint32_t*>(&hi);
-      *reinterpret_cast<uint2*>(xr + 4 * i) = pk;
+      *reinterpret_cast<uint2*>(xr + 4 * i) =
+          pack4_bf16(LAYER ? layer_apply(t, w, stash ? nws[n4 + i] : __ldg(b4 + i), mean, inv)
+                           : norm_apply(t, w, inv));
     };
     float ss = 0.f;
     if (fits) {
 #pragma unroll
-      for (int u = 0; u < REGS; ++u)
-        ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+      for (int u = 0; u < REGS; ++u) {
+        if (LAYER) ss += u * 32 + lane < n4 ? sq4(v[u], mean) : 0.f;
+        else ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+      }
       ss = warp_sum(ss);
       const float inv = rsqrtf(ss / (float)p.K + p.eps);
 #pragma unroll
@@ -372,7 +425,7 @@ __device__ __forceinline__ void norm_rows_to_smem(const FusedParams& p, unsigned
 #pragma unroll 8
       for (int i = lane; i < n4; i += 32) {
         const float4 t = __ldcg(h4 + i);
-        ss += t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
+        ss += LAYER ? sq4(t, mean) : t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
       }
       ss = warp_sum(ss);
       const float inv = rsqrtf(ss / (float)p.K + p.eps);
@@ -389,16 +442,17 @@ __device__ __forceinline__ void norm_rows_to_smem(const FusedParams& p, unsigned
 // the shared memory of every CTA of the cluster; a cluster barrier ends the prologue.
 constexpr int kFuClusterMax = 4;
 
-template <int REGS, int N>
+template <int REGS, bool LAYER, int N>
 __device__ __forceinline__ void norm_rows_to_cluster(const FusedParams& p, unsigned char* xs,
                                                      int xs_stride, int warp, int lane,
                                                      float4* nws, const NormStash<N>& st,
-                                                     uint32_t csize) {
+                                                     const NormStash<N>& st_b, uint32_t csize) {
   uint32_t rank;
   asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(rank));
   const int n4 = p.K >> 2;
   const bool stash = p.K <= NormStash<N>::kMaxK;
   const float4* w4 = reinterpret_cast<const float4*>(p.norm_w);
+  const float4* b4 = reinterpret_cast<const float4*>(p.norm_b);
   const bool fits = n4 <= 32 * REGS;
   const uint32_t local = (uint32_t)__cvta_generic_to_shared(xs);
   uint32_t base[kFuClusterMax];
@@ -428,6 +482,7 @@ __device__ __forceinline__ void norm_rows_to_cluster(const FusedParams& p, unsig
         for (int u = 0; u < N; ++u) {
           const int i = warp * 32 + lane + u * kFuWarps * 32;
           if (i < n4) nws[i] = st.w[u];
+          if (LAYER && i < n4) nws[n4 + i] = st_b.w[u];
         }
       }
       __syncthreads();
@@ -437,11 +492,13 @@ __device__ __forceinline__ void norm_rows_to_cluster(const FusedParams& p, unsig
     }
     if (!row) break;
     const uint32_t row_off = (uint32_t)m * (uint32_t)xs_stride;
+    const float mean = LAYER ? row_mean(v, h4, n4, lane, fits, p.K) : 0.f;
     auto put = [&](int i, const float4& t, float inv) {
       const float4 w = stash ? nws[i] : __ldg(w4 + i);
-      __nv_bfloat162 lo = __floats2bfloat162_rn(t.x * w.x * inv, t.y * w.y * inv);
-      __nv_bfloat162 hi = __floats2bfloat162_rn(t.z * w.z * inv, t.w * w.w * inv);
-      const uint32_t a = *reinterpret_cast<uint32_t*>(&lo), b = *reinterpret_cast<uint32_t*>(&hi);
+      const uint2 pk =
+          pack4_bf16(LAYER ? layer_apply(t, w, stash ? nws[n4 + i] : __ldg(b4 + i), mean, inv)
+                           : norm_apply(t, w, inv));
+      const uint32_t a = pk.x, b = pk.y;
       const uint32_t off = row_off + 8u * (uint32_t)i;
 #pragma unroll
       for (uint32_t t2 = 0; t2 < (uint32_t)kFuClusterMax; ++t2)
@@ -453,8 +510,10 @@ __device__ __forceinline__ void norm_rows_to_cluster(const FusedParams& p, unsig
     float ss = 0.f;
     if (fits) {
 #pragma unroll
-      for (int u = 0; u < REGS; ++u)
-        ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+      for (int u = 0; u < REGS; ++u) {
+        if (LAYER) ss += u * 32 + lane < n4 ? sq4(v[u], mean) : 0.f;
+        else ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+      }
       ss = warp_sum(ss);
       const float inv = rsqrtf(ss / (float)p.K + p.eps);
 #pragma unroll
@@ -466,7 +525,7 @@ __device__ __forceinline__ void norm_rows_to_cluster(const FusedParams& p, unsig
 #pragma unroll 8
       for (int i = lane; i < n4; i += 32) {
         const float4 t = __ldcg(h4 + i);
-        ss += t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
+        ss += LAYER ? sq4(t, mean) : t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
       }
       ss = warp_sum(ss);
       const float inv = rsqrtf(ss / (float)p.K + p.eps);
@@ -520,7 +579,7 @@ __device__ __forceinline__ void skinny_fused_tiles(const FusedParams& p, int n_t
   // A cluster shares the norm prologue by storing into its CTAs' shared memory, which may
   // only be touched once every CTA of the cluster runs: each says so here, at no cost, and
   // waits for the others just before its first remote store (norm_rows_to_cluster).
-  if (NT > 1 && PRO == kProNorm) {
+  if (NT > 1 && pro_is_norm(PRO)) {
     uint32_t csize = 1;
     asm volatile("mov.u32 %0, %%cluster_nctarank;" : "=r"(csize));
     if (csize > 1) asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
@@ -533,8 +592,10 @@ __device__ __forceinline__ void skinny_fused_tiles(const FusedParams& p, int n_t
   // Programmatic dependent launch: the kernel behind this one may start its own weight
   // fetch now, and this one goes on to read activations only when the kernel before it has
   // finished (a no-op when the launch was an ordinary one).
-  NormStash<1> stash;
-  if (PRO == kProNorm) norm_weight_fetch(p, stash);
+  constexpr bool kLayer = PRO == kProLayer;
+  NormStash<1> stash, stash_b;
+  if (pro_is_norm(PRO)) norm_weight_fetch(p, p.norm_w, stash);
+  if (kLayer) norm_weight_fetch(p, p.norm_b, stash_b);
   // Positions, the block table and the rotation table are not the work of the kernel before
   // this one either: the first tile's epilogue operands are on their way before the wait
   // (a chain of four dependent loads that the short product would not hide).
@@ -549,14 +610,15 @@ __device__ __forceinline__ void skinny_fused_tiles(const FusedParams& p, int n_t
     asm volatile("griddepcontrol.wait;" ::: "memory");
   }
 
-  if (PRO == kProNorm) {
+  if (pro_is_norm(PRO)) {
     float4* nws = reinterpret_cast<float4*>(xs + (size_t)p.M * xs_stride);
     uint32_t csize = 1;        // (launched without clusters: 1)
     if (NT > 1) asm volatile("mov.u32 %0, %%cluster_nctarank;" : "=r"(csize));
     if (NT > 1 && csize > 1) {
-      norm_rows_to_cluster<8>(p, xs, xs_stride, warp, lane, nws, stash, csize);
+      norm_rows_to_cluster<8, kLayer>(p, xs, xs_stride, warp, lane, nws, stash, stash_b, csize);
     } else {
-      norm_rows_to_smem<8>(p, xs, xs_stride, warp, lane, nws, stash, [] { __syncthreads(); });
+      norm_rows_to_smem<8, kLayer>(p, xs, xs_stride, warp, lane, nws, stash, stash_b,
+                                   [] { __syncthreads(); });
       __syncthreads();
     }
   }
@@ -580,7 +642,7 @@ __device__ __forceinline__ void skinny_fused_tiles(const FusedParams& p, int n_t
         const int m = t * 8 + r;
         uint4 ux = zero;
         if (in && m < p.M) {
-          if (PRO == kProNorm)
+          if (pro_is_norm(PRO))
             ux = *reinterpret_cast<const uint4*>(xs + (size_t)m * xs_stride + (size_t)k * 2);
           else
             ux = __ldcg(reinterpret_cast<const uint4*>(p.X + (size_t)m * p.ldx + k));
@@ -637,6 +699,7 @@ __host__ __device__ inline FusedParams rows_of(const FusedParams& p, int m0, int
   if (p.Q) q.Q = p.Q + (size_t)m0 * p.ldq;
   if (p.tok_pos) q.tok_pos = p.tok_pos + m0;
   if (p.tok_seq) q.tok_seq = p.tok_seq + m0;
+  if (p.mul_ids) q.mul_ids = p.mul_ids + m0;
   if (p.act) q.act = p.act + (size_t)m0 * p.I;
   return q;
 }
@@ -658,8 +721,9 @@ skinny_fused_kernel(const FusedParams p, int n_tiles, int group_rows) {
 
 inline size_t fused_smem(int nt, int pro, int M, int K) {
   size_t bytes = sizeof(float) * kFuWarps * kFuRows * (8 * nt + 1) + 16;
-  if (pro == kProNorm)     // normed x, and the norm's weight when it is kept (kNormStashK)
-    bytes += (size_t)M * (((K * 2 + 127) / 128) * 128 + 64) + (K <= NormStash<1>::kMaxK ? (size_t)K * 4 : 0);
+  if (pro_is_norm(pro))    // normed x, and the norm's weight (and bias) when they are kept
+    bytes += (size_t)M * (((K * 2 + 127) / 128) * 128 + 64) +
+             (K <= NormStash<1>::kMaxK ? (size_t)K * 4 * (pro == kProLayer ? 2 : 1) : 0);
   return bytes;
 }
 

@@ -34,7 +34,9 @@ __host__ __device__ inline size_t stream_smem(int nt, int pro, int M, int K, int
   size_t bytes = sizeof(float) * kFuWarps * kFuRows * (8 * nt + 1) + 16;        // reduction
   bytes = (bytes + 127) & ~size_t(127);
   bytes += (size_t)stages * kStW;                                                 // W stages
-  if (pro == kProNorm) bytes += (size_t)M * (((K * 2 + 127) / 128) * 128 + 64) + (size_t)K * 4;
+  if (pro_is_norm(pro))
+    bytes += (size_t)M * (((K * 2 + 127) / 128) * 128 + 64) +
+             (size_t)K * 4 * (pro == kProLayer ? 2 : 1);
   else bytes += (size_t)stages * kStBoxes * nt * kStGroup;                        // x stages
   return bytes + (2 * kStMaxStages + 1) * 8 + 256;
 }
@@ -77,9 +79,9 @@ skinny_stream_kernel(const FusedParams whole, const __grid_constant__ CUtensorMa
   const int xs_stride = ((p.K * 2 + 127) / 128) * 128 + 64;
   constexpr int kXStage = kStBoxes * NT * kStGroup;       // plain: [stages][box][8 NT][512 B]
   unsigned char* xs = stsmem + off;                       // norm: [M][xs_stride]
-  off += PRO == kProNorm ? (size_t)p.M * xs_stride : (size_t)n_stages * kXStage;
+  off += pro_is_norm(PRO) ? (size_t)p.M * xs_stride : (size_t)n_stages * kXStage;
   float4* nws = reinterpret_cast<float4*>(stsmem + off);  // norm: the norm's weight, float[K]
-  if (PRO == kProNorm) off += (size_t)p.K * 4;
+  if (pro_is_norm(PRO)) off += (size_t)p.K * 4 * (PRO == kProLayer ? 2 : 1);   // (and its bias)
   uint64_t* full = reinterpret_cast<uint64_t*>(stsmem + ((off + 7) & ~size_t(7)));
   uint64_t* empty = full + kStMaxStages;
   volatile int* abort = reinterpret_cast<volatile int*>(empty + kStMaxStages);
@@ -151,7 +153,7 @@ skinny_stream_kernel(const FusedParams whole, const __grid_constant__ CUtensorMa
     }
     __syncwarp();
     asm volatile("griddepcontrol.wait;" ::: "memory");               // x comes from the kernel before
-    if (PRO == kProNorm) asm volatile("bar.sync 2, %0;" ::"n"(kStThreads) : "memory");
+    if (pro_is_norm(PRO)) asm volatile("bar.sync 2, %0;" ::"n"(kStThreads) : "memory");
     if (lane == 0) {
       cur = first;
       for (int it = 0; it < ahead; ++it, advance(cur)) fill(cur, it >= early, true);
@@ -171,13 +173,18 @@ skinny_stream_kernel(const FusedParams whole, const __grid_constant__ CUtensorMa
       epi_prefetch<NT, EPI>(p, blockIdx.x, ahead);
       have_ahead = true;
     }
-    if (PRO == kProNorm) {
+    if (pro_is_norm(PRO)) {
+      constexpr bool LAYER = PRO == kProLayer;
       // The norm's weight depends on nothing: it is in shared memory before the wait ends.
       // After it a warp asks for its token's whole residual row at once and tells the
       // producer, whose remaining weight copies then queue behind these loads.
       const int n4 = p.K >> 2;
       const float4* w4 = reinterpret_cast<const float4*>(p.norm_w);
       for (int i = threadIdx.x; i < n4; i += kFuWarps * 32) nws[i] = __ldg(w4 + i);
+      if (LAYER) {
+        const float4* b4 = reinterpret_cast<const float4*>(p.norm_b);
+        for (int i = threadIdx.x; i < n4; i += kFuWarps * 32) nws[n4 + i] = __ldg(b4 + i);
+      }
       asm volatile("bar.sync 1, 256;" ::: "memory");
       asm volatile("griddepcontrol.wait;" ::: "memory");
       constexpr int REGS = 16;
@@ -202,27 +209,26 @@ skinny_stream_kernel(const FusedParams whole, const __grid_constant__ CUtensorMa
           told = true;
         }
         if (!row) break;
+        const float mean = LAYER ? row_mean(v, h4, n4, lane, fits, p.K) : 0.f;
         if (fits) {
 #pragma unroll
-          for (int u = 0; u < REGS; ++u)
-            ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+          for (int u = 0; u < REGS; ++u) {
+            if (LAYER) ss += u * 32 + lane < n4 ? sq4(v[u], mean) : 0.f;
+            else ss += v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+          }
         } else {
 #pragma unroll 8
           for (int i = lane; i < n4; i += 32) {
             const float4 t = __ldcg(h4 + i);
-            ss += t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
+            ss += LAYER ? sq4(t, mean) : t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
           }
         }
         ss = warp_sum(ss);
         const float inv = rsqrtf(ss / (float)p.K + p.eps);
         auto put = [&](int i, const float4& t) {
           const float4 w = nws[i];
-          __nv_bfloat162 lo = __floats2bfloat162_rn(t.x * w.x * inv, t.y * w.y * inv);
-          __nv_bfloat162 hi = __floats2bfloat162_rn(t.z * w.z * inv, t.w * w.w * inv);
-          uint2 pk;
-          pk.x = *reinterpret_cast<uint32_t*>(&lo);
-          pk.y = *reinterpret_cast<uint32_t*>(&hi);
-          *reinterpret_cast<uint2*>(xr + 4 * i) = pk;
+          *reinterpret_cast<uint2*>(xr + 4 * i) = pack4_bf16(
+              LAYER ? layer_apply(t, w, nws[n4 + i], mean, inv) : norm_apply(t, w, inv));
         };
         if (fits) {
 #pragma unroll
@@ -273,7 +279,7 @@ skinny_stream_kernel(const FusedParams whole, const __grid_constant__ CUtensorMa
             const int m = t * 8 + r;
             uint4 ux = zero;
             if (in) {
-              if (PRO == kProNorm) {
+              if (pro_is_norm(PRO)) {
                 if (m < p.M) ux = *reinterpret_cast<const uint4*>(xs + (size_t)m * xs_stride + (size_t)k * 2);
               } else {                 // rows beyond M arrived as zeros
                 ux = *reinterpret_cast<const uint4*>(xs + (size_t)s * kXStage +

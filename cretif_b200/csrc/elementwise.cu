@@ -209,7 +209,7 @@ add_rmsnorm_rows_kernel(float* __restrict__ h, const TD* __restrict__ delta,
 // columns (b gate columns, then the b up columns that belong to them).
 template <typename T>
 __global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ act, int I, int block,
-                                size_t total) {
+                                GateRule gate, size_t total) {
   const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= total) return;
   const size_t t = idx / I;
@@ -220,8 +220,7 @@ __global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ act, i
   const float u = to_float(gu[t * 2 * (size_t)I + ucol]);
   // float32: the reference's x / (1 + expf(-x)) (src/kernels/elementwise.cu:93-99);
   // bfloat16: the same on the special-function unit, as in the fused epilogues
-  const float s = sizeof(T) == 4 ? g / (1.0f + expf(-g)) : silu_bf16_path(g);
-  act[idx] = from_float<T>(s * u);
+  act[idx] = from_float<T>(sizeof(T) == 4 ? gate_mul(g, u, gate) : gate_mul_bf16_path(g, u, gate));
 }
 
 // ---------------------------------------------------------------- rotary + cache write
@@ -414,17 +413,19 @@ extern "C" int cretif_add_rmsnorm(float* h, const void* delta, int delta_dt, con
 }
 
 extern "C" int cretif_silu_mul(const void* gu, void* act, int dt, int T, int I, int block,
-                               void* stream) {
+                               float limit, float slope, float offset, void* stream) {
   if (T <= 0) return kOk;
-  if (I <= 0 || block < 0 || (block > 0 && I % block)) return kBadArgument;
+  const GateRule gate{limit, slope, offset};
+  if (!gate_rule_ok(limit) || I <= 0 || block < 0 || (block > 0 && I % block)) return kBadArgument;
   cudaStream_t st = (cudaStream_t)stream;
   const size_t total = (size_t)T * I;
   const unsigned blocks = (unsigned)((total + 255) / 256);
   if (dt == kF32)
-    silu_mul_kernel<float><<<blocks, 256, 0, st>>>((const float*)gu, (float*)act, I, block, total);
+    silu_mul_kernel<float><<<blocks, 256, 0, st>>>((const float*)gu, (float*)act, I, block, gate,
+                                                  total);
   else if (dt == kBF16)
     silu_mul_kernel<__nv_bfloat16><<<blocks, 256, 0, st>>>((const __nv_bfloat16*)gu,
-                                                          (__nv_bfloat16*)act, I, block, total);
+                                                          (__nv_bfloat16*)act, I, block, gate, total);
   else
     return kBadDType;
   return launch_status();

@@ -73,7 +73,8 @@ struct TcSmem {
 //   kTcStore  store as bfloat16 / float32, or add into a float32 matrix;
 //   kTcSilu   the stacked gate|up product whose weight rows are interleaved in blocks of 64
 //             (64 gate rows, then the 64 up rows that belong to them): a 128-wide tile holds
-//             matching gate and up columns, and act = silu(gate) * up is stored (BN = 128);
+//             matching gate and up columns, and act = silu(gate) * up, or what another GateRule
+//             makes of the two, is stored (BN = 128);
 //   kTcRope   the stacked q|k|v product with one head per tile (BN = head_dim): rotary on q and
 //             k, q to the query buffer, k and v into the block cache at the token's position.
 enum TcEpilogue : int { kTcStore = 0, kTcSilu = 1, kTcRope = 2, kTcStoreEx = 3 };
@@ -103,6 +104,10 @@ struct TcEpi {
   // added, and passes an activation (unary: 0 none, else 1 + the kind of unary_activation)
   // before it is stored
   float alpha; int scaled; int unary;
+  // kTcStoreEx: what is stored of row m is multiplied by row mul_ids[m] of a bfloat16 table (null:
+  // none; an id outside [0, mul_rows) multiplies by zero)
+  const __nv_bfloat16* mul; int mul_ld, mul_rows; const int* mul_ids;
+  GateRule gate;                                           // silu
 };
 
 __device__ __forceinline__ float round_bf16(float x) {
@@ -388,6 +393,18 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 for (int e = 0; e < 8; ++e) v[e] = unary_activation(v[e], ep.unary - 1);
               }
               const int n = n0 + c0 + j;
+              if (EPI == kTcStoreEx && ep.mul && n < N) {          // (N is a multiple of 8 then)
+                const int id = ep.mul_ids[m];
+                float f[8];
+                if (id >= 0 && id < ep.mul_rows) {
+                  load8(ep.mul + (size_t)id * ep.mul_ld + n, f);
+                } else {
+#pragma unroll
+                  for (int e = 0; e < 8; ++e) f[e] = 0.f;
+                }
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[e] *= f[e];
+              }
               if (n + 8 <= N) {
                 if (pre) {
                   const float4 a = cur[j >> 2], b = cur[(j >> 2) + 1];
@@ -437,8 +454,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
               const float g1 = round_bf16(__uint_as_float(g[j + e + 1]));
               const float u0 = round_bf16(__uint_as_float(u[j + e]));
               const float u1 = round_bf16(__uint_as_float(u[j + e + 1]));
-              __nv_bfloat162 h2 = __floats2bfloat162_rn(silu_bf16_path(g0) * u0,
-                                                        silu_bf16_path(g1) * u1);
+              __nv_bfloat162 h2 = __floats2bfloat162_rn(gate_mul_bf16_path(g0, u0, ep.gate),
+                                                        gate_mul_bf16_path(g1, u1, ep.gate));
               w4[e >> 1] = *reinterpret_cast<uint32_t*>(&h2);
             }
             const int piece = chalf * 4 + (j >> 3);
@@ -474,7 +491,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                   // gate and up pass through bfloat16 as they do when stored separately
                   const float gg = round_bf16(__uint_as_float(g[j + e]));
                   const float uu = round_bf16(__uint_as_float(u[j + e]));
-                  v[e] = silu_bf16_path(gg) * uu;
+                  v[e] = gate_mul_bf16_path(gg, uu, ep.gate);
                 }
                 if (col0 + c0 + j + 8 <= ep.I) store8(out + j, v);
               }
@@ -792,8 +809,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
               const float g1 = round_bf16(__uint_as_float(g[j + e + 1]));
               const float u0 = round_bf16(__uint_as_float(u[j + e]));
               const float u1 = round_bf16(__uint_as_float(u[j + e + 1]));
-              __nv_bfloat162 h2 = __floats2bfloat162_rn(silu_bf16_path(g0) * u0,
-                                                        silu_bf16_path(g1) * u1);
+              __nv_bfloat162 h2 = __floats2bfloat162_rn(gate_mul_bf16_path(g0, u0, ep.gate),
+                                                        gate_mul_bf16_path(g1, u1, ep.gate));
               w4[e >> 1] = *reinterpret_cast<uint32_t*>(&h2);
             }
             const int piece = chalf * 4 + (j >> 3);
@@ -1132,9 +1149,12 @@ extern "C" void cretif_gemm_tc_stamps(unsigned long long* device_buffer) {
 
 extern "C" int cretif_gemm_tc(const void* A, const void* W, void* C, int c_dt, int M, int N, int K,
                               int lda, int ldw, int ldc, int accumulate, int bn, float alpha,
-                              int unary, unsigned int* fault, void* stream) {
+                              int unary, const void* mul, int mul_ld, int mul_rows,
+                              const int* mul_ids, unsigned int* fault, void* stream) {
   if (M <= 0 || N <= 0) return kOk;
   if (unary < 0 || unary > kUnaryKinds || (unary && accumulate)) return kBadArgument;
+  if (mul && (accumulate || !mul_ids || N % 8 || mul_ld % 8 || mul_ld < N || ((uintptr_t)mul & 15)))
+    return kBadArgument;
   if (K <= 0 || K % 8 || lda % 8 || ldw % 8 || lda < K || ldw < K || ldc < N) return kBadArgument;
   if ((M + kTcBM - 1) / kTcBM > 65535) return kBadArgument;
   if (((uintptr_t)A | (uintptr_t)W | (uintptr_t)C) & 15) return kMisaligned;
@@ -1151,6 +1171,7 @@ extern "C" int cretif_gemm_tc(const void* A, const void* W, void* C, int c_dt, i
   TcEpi ep = {};
   ep.C = C; ep.ldc = ldc; ep.accumulate = accumulate;
   ep.alpha = alpha; ep.scaled = alpha != 1.0f; ep.unary = unary;
+  ep.mul = (const __nv_bfloat16*)mul; ep.mul_ld = mul_ld; ep.mul_rows = mul_rows; ep.mul_ids = mul_ids;
   // The float32 add of a large product: two CTAs a tile (see gemm_tc_pair_kernel), as wide as
   // the single-CTA tile would be.
   if (c_dt == kF32 && accumulate && g_tc_pair != 0 && g_tc_bulk_add && (bn == 256 || bn == 192) &&
@@ -1166,7 +1187,7 @@ extern "C" int cretif_gemm_tc(const void* A, const void* W, void* C, int c_dt, i
   (c_dt == kBF16 ? launch_tc<BN, EPI, __nv_bfloat16>(A, W, ep, M, N, K, lda, ldw, fault, st)   \
                  : launch_tc<BN, EPI, float>(A, W, ep, M, N, K, lda, ldw, fault, st))
 #define CRETIF_TC(BN) \
-  ((ep.scaled || ep.unary) ? CRETIF_TC_AS(BN, kTcStoreEx) : CRETIF_TC_AS(BN, kTcStore))
+  ((ep.scaled || ep.unary || ep.mul) ? CRETIF_TC_AS(BN, kTcStoreEx) : CRETIF_TC_AS(BN, kTcStore))
   if (c_dt != kBF16 && c_dt != kF32) return kBadDType;
   if (c_dt == kBF16 && accumulate) return kBadArgument;
   switch (bn) {
@@ -1182,12 +1203,14 @@ extern "C" int cretif_gemm_tc(const void* A, const void* W, void* C, int c_dt, i
 
 // act[M, I] = silu(A·Wg^T) * (A·Wu^T); Wgu holds gate and up rows interleaved in blocks of 64.
 extern "C" int cretif_gemm_tc_silu(const void* A, const void* Wgu, void* act, int M, int I, int K,
-                                   int lda, int ldw, unsigned int* fault, void* stream) {
+                                   int lda, int ldw, float limit, float slope, float offset,
+                                   unsigned int* fault, void* stream) {
   if (M <= 0 || I <= 0) return kOk;
-  if (!tc_operands_ok(A, Wgu, M, K, lda, ldw) || I % 64) return kBadArgument;
+  if (!tc_operands_ok(A, Wgu, M, K, lda, ldw) || I % 64 || !gate_rule_ok(limit)) return kBadArgument;
   if (((uintptr_t)act) & 15) return kMisaligned;
   TcEpi ep = {};
   ep.act = (__nv_bfloat16*)act; ep.I = I;
+  ep.gate = GateRule{limit, slope, offset};
   // wide tiles (two gate|up pairs, one CTA per SM) once there are four waves of them for the
   // whole chip; with fewer, the last wave's empty seats cost more than the wide tile saves
   const long long wide_tiles = (long long)((2 * I + 255) / 256) * ((M + kTcBM - 1) / kTcBM);
@@ -1256,14 +1279,17 @@ extern "C" int cretif_gemm_tc_act_grouped(const void* A, const void* W, void* C,
 extern "C" int cretif_gemm_tc_silu_grouped(const void* A, const void* Wgu, void* act, int M, int I,
                                            int K, int lda, int ldw, int groups,
                                            const int* tile_group, const int* used_m_tiles,
+                                           float limit, float slope, float offset,
                                            unsigned int* fault, void* stream) {
   if (M <= 0 || I <= 0 || groups <= 0) return kOk;
+  if (!gate_rule_ok(limit)) return kBadArgument;
   if (!tc_operands_ok(A, Wgu, M, K, lda, ldw) || I % 64 || M % kTcBM || !tile_group ||
       (long long)groups * 2 * I > 0x7fffffffLL)
     return kBadArgument;
   if (((uintptr_t)act) & 15) return kMisaligned;
   TcEpi ep = {};
   ep.act = (__nv_bfloat16*)act; ep.I = I;
+  ep.gate = GateRule{limit, slope, offset};
   ep.tile_group = tile_group; ep.group_rows = 2 * I; ep.used_m_tiles = used_m_tiles;
   const long long wide_tiles = (long long)((2 * I + 255) / 256) * (M / kTcBM);
   if (wide_tiles >= 4 * 148)

@@ -14,7 +14,13 @@
 //
 // projnorm_rope_kv_append: the same with the norms over the WHOLE query and the whole key projection
 // (a weight per channel), from float32 rows, a CTA per token; v is multiplied by v_scale before it is
-// stored, so that a factor on the attention's output costs nothing.
+// stored, so that a factor on the attention's output costs nothing.  Instead of a bias the projected
+// rows may pass a short causal convolution over time, channel by channel, before norms and rotation:
+//   x_t[c] = sum_j conv_w[j, c] u_(t - taps + 1 + j)[c]
+// with u from this step's rows or, where the window reaches back before the step, from the sequence's
+// saved last taps - 1 inputs (conv_state, [C, taps - 1] per slot, zeros at a sequence's start).  A
+// step of one token a sequence also brings the saved inputs up to date (save_inputs): each channel is
+// read and replaced by one thread.  After any other step delta_conv_state (delta_rule.cu) does.
 //
 // Pooled entries (PooledKeys in common.cuh): pool_kv writes the means of the blocks of tokens that
 // the step completes; a step of one token a sequence does it at the end of
@@ -236,7 +242,18 @@ __device__ __forceinline__ void hn_st4(__nv_bfloat16* p, const float4& v) {
   *reinterpret_cast<uint2*>(p) = u;
 }
 
-template <typename T, bool VEC, int NT>
+// The convolution in front of the norms.  w [taps, C]: a tap's weights lie side by side.
+struct ProjConv {
+  const float* w;
+  float* state;
+  size_t stride;
+  const int* seq_start;
+  int taps, C, save;
+};
+
+// TAPS: 0 no convolution; 2, 3, 4: that many taps, four channels at a time; -1: any number, a channel
+// at a time.
+template <typename T, bool VEC, int NT, int TAPS>
 __global__ void __launch_bounds__(NT)
 projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
                                const float* __restrict__ bias, const float* __restrict__ wq,
@@ -248,7 +265,7 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
                                T* __restrict__ q_out, int ldq, const int* __restrict__ table,
                                int table_stride, T* kc, T* vc, int bt, int write_cache, T* pk, T* pv,
                                const int* __restrict__ pool_table, int pool_stride, int pool,
-                               unsigned int* __restrict__ fault) {
+                               const ProjConv conv, unsigned int* __restrict__ fault) {
   extern __shared__ __align__(16) float row_s[];       // q | k with the bias
   __shared__ float sums[NT / 32][2];
   const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -265,6 +282,76 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
   const int half = rot_dim >> 1;
   const float* c = cos_t + (size_t)pos * half;
   const float* s = sin_t + (size_t)pos * half;
+  int lt = 0, keep = 0;               // tokens of the sequence before t in the step; saved inputs
+  float* st = nullptr;
+  if (TAPS != 0) {
+    const int b = tok_seq[t];
+    lt = pos - conv.seq_start[b];
+    keep = conv.taps - 1;
+    if (keep) st = conv.state + (size_t)seq_slot[b] * conv.stride;
+  }
+  auto conv1 = [&](int ch) {
+    float acc = 0.f;
+    for (int j = 0; j <= keep; ++j) {
+      const int back = keep - j;
+      const float u = back <= lt ? row[ch - (ptrdiff_t)back * ldp]
+                                 : st[(size_t)ch * keep + keep - (back - lt)];
+      acc = fmaf(conv.w[(size_t)j * conv.C + ch], u, acc);
+    }
+    if (conv.save && keep) {
+      float* mine = st + (size_t)ch * keep;
+      for (int j = 0; j + 1 < keep; ++j) mine[j] = mine[j + 1];
+      mine[keep - 1] = row[ch];
+    }
+    return acc;
+  };
+  auto conv4 = [&](int ch) {
+    constexpr int K = TAPS > 1 ? TAPS - 1 : 1;
+    float4 u[K + 1];
+    float4 w[K + 1];
+    u[K] = hn_ld4(row + ch);
+#pragma unroll
+    for (int j = 0; j <= K; ++j) w[j] = hn_ld4(conv.w + (size_t)j * conv.C + ch);
+    float4 saved[K];                   // four channels' saved inputs: channel u's are 4 / K apart
+    float* f = reinterpret_cast<float*>(saved);
+    float* mine = st + (size_t)ch * K;
+    if (lt < K) {
+#pragma unroll
+      for (int j = 0; j < K; ++j) saved[j] = hn_ld4(mine + 4 * j);
+    }
+#pragma unroll
+    for (int j = 0; j < K; ++j) {
+      const int back = K - j;
+      if (back <= lt) {
+        u[j] = hn_ld4(row + ch - (ptrdiff_t)back * ldp);
+      } else {                         // entry K - (back - lt) = j + lt of every channel
+        u[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < K; ++i)
+          if (i == j + lt) u[j] = make_float4(f[i], f[K + i], f[2 * K + i], f[3 * K + i]);
+      }
+    }
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j <= K; ++j) {
+      acc.x = fmaf(w[j].x, u[j].x, acc.x);
+      acc.y = fmaf(w[j].y, u[j].y, acc.y);
+      acc.z = fmaf(w[j].z, u[j].z, acc.z);
+      acc.w = fmaf(w[j].w, u[j].w, acc.w);
+    }
+    if (conv.save) {                   // (lt is zero)
+      float g[4 * K];
+#pragma unroll
+      for (int i = 0; i < K; ++i) {
+        const float4& v = u[i + 1];
+        g[i] = v.x; g[K + i] = v.y; g[2 * K + i] = v.z; g[3 * K + i] = v.w;
+      }
+#pragma unroll
+      for (int j = 0; j < K; ++j)
+        hn_st4(mine + 4 * j, make_float4(g[4 * j], g[4 * j + 1], g[4 * j + 2], g[4 * j + 3]));
+    }
+    return acc;
+  };
   if (VEC) {
     // (few tokens: what the thread's first turn reads after the row's sums are known)
     if (NT > 256 && 4 * tid < nkv * vd) {
@@ -280,8 +367,8 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
       }
     }
     for (int i = 4 * tid; i < nqk; i += 4 * NT) {
-      float4 v = *reinterpret_cast<const float4*>(row + i);
-      if (bias) {
+      float4 v = TAPS != 0 ? conv4(i) : hn_ld4(row + i);
+      if (TAPS == 0 && bias) {
         const float4 b4 = *reinterpret_cast<const float4*>(bias + i);
         v.x += b4.x; v.y += b4.y; v.z += b4.z; v.w += b4.w;
       }
@@ -291,7 +378,7 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
     }
   } else {
     for (int i = tid; i < nqk; i += NT) {
-      const float v = row[i] + (bias ? bias[i] : 0.f);
+      const float v = TAPS != 0 ? conv1(i) : row[i] + (bias ? bias[i] : 0.f);
       row_s[i] = v;
       if (i < nq) ssq += v * v; else ssk += v * v;
     }
@@ -362,8 +449,8 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
   const bool vec_v = VEC && (vd & 3) == 0 && (reinterpret_cast<uintptr_t>(vc) & 15) == 0;
   for (int idx = 4 * tid; vec_v && idx < nkv * vd; idx += 4 * NT) {
     const int kvh = idx / vd, i = idx - kvh * vd;
-    float4 v = hn_ld4(row + nqk + idx);
-    if (bias) {
+    float4 v = TAPS != 0 ? conv4(nqk + idx) : hn_ld4(row + nqk + idx);
+    if (TAPS == 0 && bias) {
       const float4 b4 = hn_ld4(bias + nqk + idx);
       v.x += b4.x; v.y += b4.y; v.z += b4.z; v.w += b4.w;
     }
@@ -372,7 +459,7 @@ projnorm_rope_kv_append_kernel(const float* __restrict__ proj, int ldp,
   }
   for (int idx = tid; !vec_v && idx < nkv * vd; idx += NT) {
     const int kvh = idx / vd, i = idx - kvh * vd;
-    const float v = row[nqk + idx] + (bias ? bias[nqk + idx] : 0.f);
+    const float v = TAPS != 0 ? conv1(nqk + idx) : row[nqk + idx] + (bias ? bias[nqk + idx] : 0.f);
     vc[(((size_t)blk * nkv + kvh) * bt + pos % bt) * vd + i] = from_float<T>(v * v_scale);
   }
   if (pool_table && (pos + 1) % pool == 0) {       // (one token a sequence: this one ends a block)
@@ -446,12 +533,18 @@ __global__ void gate_channels8_kernel(__nv_bfloat16* __restrict__ o, int ldo,
 
 template <typename TI, typename TO>
 __global__ void activation_kernel(const TI* __restrict__ in, int ldi, TO* __restrict__ out, int ldo,
-                                  int width, long long total, int kind) {
+                                  int width, long long total, int kind, const TO* __restrict__ mul,
+                                  int mul_ld, int mul_rows, const int* __restrict__ mul_ids) {
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= total) return;
   const long long t = idx / width;
   const int col = (int)(idx - t * width);
-  out[(size_t)t * ldo + col] = from_float<TO>(unary_activation(to_float(in[(size_t)t * ldi + col]), kind));
+  float v = unary_activation(to_float(in[(size_t)t * ldi + col]), kind);
+  if (mul) {                          // times the token's row of a table
+    const int id = mul_ids[t];
+    v *= id >= 0 && id < mul_rows ? to_float(mul[(size_t)id * mul_ld + col]) : 0.f;
+  }
+  out[(size_t)t * ldo + col] = from_float<TO>(v);
 }
 
 // z <- cap * tanh(z / cap), in place, 32-bit.
@@ -529,8 +622,15 @@ extern "C" int cretif_projnorm_rope_kv_append(
     const int* tok_seq, const int* seq_slot, int nh, int nkv, int hd, int vd, float v_scale,
     void* q_out, int ldq, int dt, const int* table, int table_stride, void* kc, void* vc, int bt,
     int write_cache, void* pool_k, void* pool_v, const int* pool_table, int pool_stride, int pool,
-    int T, unsigned int* fault, void* stream) {
+    const float* conv_w, int taps, float* conv_state, long long conv_stride, const int* seq_start,
+    int save_inputs, int T, unsigned int* fault, void* stream) {
   if (T <= 0) return kOk;
+  if (conv_w && (taps < 1 || bias || !write_cache || !seq_start ||
+                 (taps > 1 && (!conv_state ||
+                               conv_stride < (long long)((nh + nkv) * hd + nkv * vd) * (taps - 1)))))
+    return kBadArgument;
+  const ProjConv conv{conv_w, conv_state, (size_t)conv_stride, seq_start, taps,
+                      (nh + nkv) * hd + nkv * vd, save_inputs};
   if (nh <= 0 || nkv < 0 || hd <= 0 || vd <= 0 || ldq < nh * hd || rot_dim < 0 || rot_dim > hd ||
       (rot_dim & 1) || !wq || (nkv && !wk) || ldp < (nh + nkv) * hd + nkv * vd)
     return kBadArgument;
@@ -543,36 +643,47 @@ extern "C" int cretif_projnorm_rope_kv_append(
   const bool vec = hd % 4 == 0 && ldp % 4 == 0 && ldq % 4 == 0 &&
                    (pairing ? rot_dim % 4 == 0 : rot_dim % 8 == 0) &&
                    (((uintptr_t)proj | (uintptr_t)bias | (uintptr_t)q_out | (uintptr_t)kc | (uintptr_t)wq |
-                     (uintptr_t)wk | (uintptr_t)cos_t | (uintptr_t)sin_t) & 15) == 0;
+                     (uintptr_t)wk | (uintptr_t)cos_t | (uintptr_t)sin_t) & 15) == 0 &&
+                   (!conv_w || (taps >= 2 && taps <= 4 && conv.C % 4 == 0 && vd % 4 == 0 &&
+                                conv_stride % 4 == 0 &&
+                                (((uintptr_t)conv_w | (uintptr_t)conv_state | (uintptr_t)vc) & 15) == 0));
   cudaStream_t st = (cudaStream_t)stream;
-#define CRETIF_PN(TT, VEC)                                                                        \
+#define CRETIF_PN(TT, VEC, TAPS)                                                                  \
   do {                                                                                            \
-    if (T < 64) CRETIF_PN_N(TT, VEC, 1024);                                                       \
-    else CRETIF_PN_N(TT, VEC, 256);                                                               \
+    if (T < 64) CRETIF_PN_N(TT, VEC, 1024, TAPS);                                                 \
+    else CRETIF_PN_N(TT, VEC, 256, TAPS);                                                         \
   } while (0)
-#define CRETIF_PN_N(TT, VEC, NT)                                                                  \
+#define CRETIF_PN_T(TT)                                                                           \
+  do {                                                                                            \
+    if (vec && !conv_w) CRETIF_PN(TT, true, 0);                                                   \
+    else if (vec && taps == 2) CRETIF_PN(TT, true, 2);                                            \
+    else if (vec && taps == 3) CRETIF_PN(TT, true, 3);                                            \
+    else if (vec) CRETIF_PN(TT, true, 4);                                                         \
+    else if (!conv_w) CRETIF_PN(TT, false, 0);                                                    \
+    else CRETIF_PN(TT, false, -1);                                                                \
+  } while (0)
+#define CRETIF_PN_N(TT, VEC, NT, TAPS)                                                            \
   do {                                                                                            \
     if (smem > 40 * 1024) {                                                                       \
-      cudaError_t err = cudaFuncSetAttribute(projnorm_rope_kv_append_kernel<TT, VEC, NT>,         \
+      cudaError_t err = cudaFuncSetAttribute(projnorm_rope_kv_append_kernel<TT, VEC, NT, TAPS>,   \
                                              cudaFuncAttributeMaxDynamicSharedMemorySize,         \
                                              (int)smem);                                          \
       if (err != cudaSuccess) return (int)err;                                                    \
     }                                                                                             \
-    projnorm_rope_kv_append_kernel<TT, VEC, NT><<<T, NT, smem, st>>>(                             \
+    projnorm_rope_kv_append_kernel<TT, VEC, NT, TAPS><<<T, NT, smem, st>>>(                       \
         proj, ldp, bias, wq, wk, eps, cos_t, sin_t, pairing, rot_dim, tok_pos, tok_seq, seq_slot, \
         nh, nkv, hd, vd, v_scale, (TT*)q_out, ldq, table, table_stride, (TT*)kc, (TT*)vc, bt,     \
-        write_cache, (TT*)pool_k, (TT*)pool_v, pool_table, pool_stride, pool, fault);             \
+        write_cache, (TT*)pool_k, (TT*)pool_v, pool_table, pool_stride, pool, conv, fault);       \
   } while (0)
   if (dt == kF32) {
-    if (vec) CRETIF_PN(float, true);
-    else CRETIF_PN(float, false);
+    CRETIF_PN_T(float);
   } else if (dt == kBF16) {
-    if (vec) CRETIF_PN(__nv_bfloat16, true);
-    else CRETIF_PN(__nv_bfloat16, false);
+    CRETIF_PN_T(__nv_bfloat16);
   } else {
     return kBadDType;
   }
 #undef CRETIF_PN_N
+#undef CRETIF_PN_T
 #undef CRETIF_PN
   return launch_status();
 }
@@ -639,21 +750,26 @@ extern "C" int cretif_gate_heads(void* o, int ldo, int dt, const float* g, int l
 }
 
 extern "C" int cretif_activation(const void* in, int ldi, int in_dt, void* out, int ldo, int out_dt,
-                                 int T, int width, int kind, void* stream) {
+                                 int T, int width, int kind, const void* mul, int mul_ld,
+                                 int mul_rows, const int* mul_ids, void* stream) {
   if (T <= 0 || width <= 0) return kOk;
   if (ldi < width || ldo < width || kind < 0 || kind >= kUnaryKinds) return kBadArgument;
+  if (mul && (!mul_ids || mul_ld < width)) return kBadArgument;
   const long long total = (long long)T * width;
   const unsigned blocks = (unsigned)((total + 255) / 256);
   cudaStream_t st = (cudaStream_t)stream;
   if (in_dt == kF32 && out_dt == kF32)
     activation_kernel<float, float><<<blocks, 256, 0, st>>>((const float*)in, ldi, (float*)out,
-                                                            ldo, width, total, kind);
+                                                            ldo, width, total, kind,
+                                                            (const float*)mul, mul_ld, mul_rows, mul_ids);
   else if (in_dt == kF32 && out_dt == kBF16)
     activation_kernel<float, __nv_bfloat16><<<blocks, 256, 0, st>>>(
-        (const float*)in, ldi, (__nv_bfloat16*)out, ldo, width, total, kind);
+        (const float*)in, ldi, (__nv_bfloat16*)out, ldo, width, total, kind,
+        (const __nv_bfloat16*)mul, mul_ld, mul_rows, mul_ids);
   else if (in_dt == kBF16 && out_dt == kBF16)
     activation_kernel<__nv_bfloat16, __nv_bfloat16><<<blocks, 256, 0, st>>>(
-        (const __nv_bfloat16*)in, ldi, (__nv_bfloat16*)out, ldo, width, total, kind);
+        (const __nv_bfloat16*)in, ldi, (__nv_bfloat16*)out, ldo, width, total, kind,
+        (const __nv_bfloat16*)mul, mul_ld, mul_rows, mul_ids);
   else
     return kBadDType;
   return launch_status();

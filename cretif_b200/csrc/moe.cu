@@ -42,8 +42,9 @@ namespace {
 constexpr int kTile = 64;
 constexpr int kMaxExpertsPerLane = 8;            // E <= 256
 
-// How a token's experts are chosen.  softmax: the scores are the softmax of the logits, else their
-// logistic function.  correction [E] (may be null): added to the scores for the choice only.
+// How a token's experts are chosen.  bias [E] (may be null): added to the logits.  softmax 1: the
+// scores are the softmax of the logits; 2: their exponentials relative to the largest, which with
+// renorm is the softmax over the chosen ones alone; 0: their logistic function.  correction [E] (may be null): added to the scores for the choice only.
 // groups > 1: the experts form that many equal groups of neighbours, a group's score is the sum of
 // its two largest choice scores (group_best: the largest alone), and only experts of the `keep` best
 // groups can be chosen.  renorm: the chosen scores are divided by their sum plus sum_eps.
@@ -52,6 +53,7 @@ struct RouteRule {
   float sum_eps;
   int softmax, group_best;
   const float* correction;
+  const float* bias;
 };
 
 // Warp-wide: the `top` largest choices of E outputs (ties: the lower index) among those of the groups
@@ -66,7 +68,7 @@ __device__ __forceinline__ void select_top_n(const float* logits, int E, const R
 #pragma unroll
   for (int m = 0; m < NPL; ++m) {
     const int e = lane + 32 * m;
-    z[m] = e < E ? logits[e] : -INFINITY;
+    z[m] = e < E ? logits[e] + (rule.bias ? rule.bias[e] : 0.f) : -INFINITY;
   }
   // sc: the scores; z from here on: what the choice compares (the logits order like their logistic
   // scores, so without a correction they are compared as they are)
@@ -81,9 +83,11 @@ __device__ __forceinline__ void select_top_n(const float* logits, int E, const R
       sc[m] = lane + 32 * m < E ? expf(z[m] - mx) : 0.f;
       sum += sc[m];
     }
-    sum = warp_sum(sum);
+    if (rule.softmax == 1) {
+      sum = warp_sum(sum);
 #pragma unroll
-    for (int m = 0; m < NPL; ++m) sc[m] /= sum;
+      for (int m = 0; m < NPL; ++m) sc[m] /= sum;
+    }
   } else {
 #pragma unroll
     for (int m = 0; m < NPL; ++m) sc[m] = 1.0f / (1.0f + expf(-z[m]));
@@ -343,7 +347,7 @@ __device__ __forceinline__ TileRows tile_rows(const int* tile_expert, const int*
   return tr;
 }
 
-// mode 0: gate|up with the activation; mode 1: plain product into float32 rows; mode 2 + k: an
+// mode 0: gate|up with the activation (a GateRule: SiLU or a clamped gate); mode 1: plain product into float32 rows; mode 2 + k: an
 // expert without a gate, C = act_k(A W^T) with kind k of unary_activation, rows as in mode 0.
 // scale_at: 0 none, 1 the router weight scales the sums of mode 0 (the expert's input),
 // 2 it scales the rows of mode 1 (the expert's output).
@@ -353,7 +357,7 @@ moe_gemm_simt_kernel(const TA* __restrict__ A, int lda, const TW* __restrict__ W
                      int ldc, int N, int K, int top, int mode, int scale_at,
                      const float* __restrict__ wts, const int* __restrict__ order,
                      const int* __restrict__ offsets, const int* __restrict__ tile_expert,
-                     const int* __restrict__ tile_row0) {
+                     const int* __restrict__ tile_row0, const GateRule gate) {
   constexpr int BK = 16, TM = 4, TN = 4;
   const TileRows tr = tile_rows(tile_expert, tile_row0, offsets, blockIdx.y);
   if (tr.rows <= 0) return;
@@ -419,7 +423,7 @@ moe_gemm_simt_kernel(const TA* __restrict__ A, int lda, const TW* __restrict__ W
       if (mode == 0) {
         const float sg = scale_at == 1 ? s : 1.f;
         const float g = acc[0][i][j] * sg, u = acc[1][i][j] * sg;
-        reinterpret_cast<TA*>(Cv)[(size_t)r * ldc + n] = from_float<TA>(g / (1.0f + expf(-g)) * u);
+        reinterpret_cast<TA*>(Cv)[(size_t)r * ldc + n] = from_float<TA>(gate_mul(g, u, gate));
       } else if (mode >= 2) {
         reinterpret_cast<TA*>(Cv)[(size_t)r * ldc + n] = from_float<TA>(
             unary_activation(acc[0][i][j] * (scale_at == 1 ? s : 1.f), mode - 2));
@@ -441,7 +445,7 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda,
                     int mode, int scale_at, const float* __restrict__ wts,
                     const int* __restrict__ order, const int* __restrict__ offsets,
                     const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
-                    int a_vec, int w_vec) {
+                    int a_vec, int w_vec, const GateRule gate) {
   using namespace nvcuda;
   const TileRows tr = tile_rows(tile_expert, tile_row0, offsets, blockIdx.y);
   if (tr.rows <= 0) return;
@@ -539,7 +543,7 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda,
       const float sg = scale_at == 1 ? s : 1.f;
       const float g = Cs[0][warp][lane][c] * sg, u = Cs[1][warp][lane][c] * sg;
       reinterpret_cast<__nv_bfloat16*>(Cv)[(size_t)r * ldc + n] =
-          __float2bfloat16_rn(silu_bf16_path(g) * u);
+          __float2bfloat16_rn(gate_mul_bf16_path(g, u, gate));
     } else if (mode >= 2) {
       reinterpret_cast<__nv_bfloat16*>(Cv)[(size_t)r * ldc + n] = __float2bfloat16_rn(
           unary_activation(Cs[0][warp][lane][c] * (scale_at == 1 ? s : 1.f), mode - 2));
@@ -560,7 +564,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 moe_gemv_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, void* Cv, int ldc, int N,
                 int K, int top, int mode, int scale_at, const int* __restrict__ ids,
-                const float* __restrict__ wts, int vec, int experts) {
+                const float* __restrict__ wts, int vec, int experts, const GateRule gate) {
   extern __shared__ __align__(16) unsigned char gemv_smem[];
   T* xs = reinterpret_cast<T*>(gemv_smem);
   const int p = blockIdx.y;
@@ -619,7 +623,7 @@ moe_gemv_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, void*
       const float sg = scale_at == 1 ? s : 1.f;
       const float g = acc[c] * sg, u = acc[2 + c] * sg;
       if (lane == 0)
-        reinterpret_cast<T*>(Cv)[(size_t)p * ldc + n] = from_float<T>(g / (1.0f + expf(-g)) * u);
+        reinterpret_cast<T*>(Cv)[(size_t)p * ldc + n] = from_float<T>(gate_mul(g, u, gate));
     } else if (mode >= 2) {
       const float v = acc[c] * (scale_at == 1 ? s : 1.f);
       if (lane == 0)
@@ -633,13 +637,15 @@ moe_gemv_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, void*
 
 // V columns a thread (4: rows, y and x allow 16-byte accesses, 8-byte ones for bfloat16).
 // Identity pairs (ids[pair] >= experts): id_wts[pair] times the token's row of x instead of a row of
-// the products.  wts: weights that the products have not applied yet.
+// the products.  wts: weights that the products have not applied yet.  add: the sum is added to y (the residual stream) instead of
+// stored, and x_out (may be null) receives the new rows in bfloat16.
 template <typename TX, int V>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ rows, int ld, const int* __restrict__ place, int top,
                    const float* __restrict__ wts, float* __restrict__ y, int T, int H,
                    const int* __restrict__ ids, int experts, const float* __restrict__ id_wts,
-                   const TX* __restrict__ x, int ldx, const float* __restrict__ plus) {
+                   const TX* __restrict__ x, int ldx, const float* __restrict__ plus, int add,
+                   __nv_bfloat16* __restrict__ x_out) {
   const long long idx = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
   if (idx >= (long long)T * H) return;
   const int t = (int)(idx / H), c = (int)(idx - (long long)t * H);
@@ -675,6 +681,14 @@ moe_combine_kernel(const float* __restrict__ rows, int ld, const int* __restrict
 #pragma unroll
     for (int u = 0; u < V; ++u) acc[u] += plus[idx + u];
   }
+  if (add) {
+#pragma unroll
+    for (int u = 0; u < V; ++u) acc[u] += y[idx + u];
+  }
+  if (x_out) {
+#pragma unroll
+    for (int u = 0; u < V; ++u) x_out[idx + u] = __float2bfloat16_rn(acc[u]);
+  }
   if (V == 4)
     *reinterpret_cast<float4*>(y + idx) = make_float4(acc[0], acc[V > 1 ? 1 : 0], acc[V > 2 ? 2 : 0],
                                                       acc[V > 3 ? 3 : 0]);
@@ -696,13 +710,13 @@ static bool route_rule_ok(int E, int top, int groups, int keep) {
 
 extern "C" int cretif_moe_route(const void* x, int x_dt, int ldx, const float* router_w, int E,
                                 int H, int top, int renorm, int groups, int keep, float sum_eps,
-                                int softmax, int group_best, const float* correction, int* ids,
-                                float* wts, int T, void* stream) {
+                                int softmax, int group_best, const float* correction, const float* bias,
+                                int* ids, float* wts, int T, void* stream) {
   if (T <= 0) return kOk;
   if (E <= 0 || E > 32 * kMaxExpertsPerLane || H <= 0 || top <= 0 || top > E || ldx < H)
     return kBadArgument;
   if (!route_rule_ok(E, top, groups, keep)) return kBadArgument;
-  const RouteRule rule{top, renorm, groups, keep, sum_eps, softmax, group_best, correction};
+  const RouteRule rule{top, renorm, groups, keep, sum_eps, softmax, group_best, correction, bias};
   cudaStream_t st = (cudaStream_t)stream;
   const int vec = H % 4 == 0 && ldx % 4 == 0 && (((uintptr_t)x | (uintptr_t)router_w) & 15) == 0;
   if (x_dt == kF32)
@@ -719,11 +733,12 @@ extern "C" int cretif_moe_route(const void* x, int x_dt, int ldx, const float* r
 // ids/wts from logits [T, ld >= E] that a matrix product computed.
 extern "C" int cretif_moe_topk(const float* logits, int ld, int E, int top, int renorm, int groups,
                                int keep, float sum_eps, int softmax, int group_best,
-                               const float* correction, int* ids, float* wts, int T, void* stream) {
+                               const float* correction, const float* bias, int* ids, float* wts,
+                               int T, void* stream) {
   if (T <= 0) return kOk;
   if (E <= 0 || E > kMaxExperts || top <= 0 || top > E || ld < E) return kBadArgument;
   if (!route_rule_ok(E, top, groups, keep)) return kBadArgument;
-  const RouteRule rule{top, renorm, groups, keep, sum_eps, softmax, group_best, correction};
+  const RouteRule rule{top, renorm, groups, keep, sum_eps, softmax, group_best, correction, bias};
   moe_topk_kernel<<<(unsigned)((T + 7) / 8), 256, 0, (cudaStream_t)stream>>>(logits, ld, E, rule,
                                                                              ids, wts, T);
   return launch_status();
@@ -770,7 +785,10 @@ extern "C" int cretif_moe_gemm(const void* A, int a_dt, int lda, const void* W, 
                                int ldc, int N, int K, int top, int mode, int scale_at,
                                const float* wts, const int* order, const int* offsets,
                                const int* tile_expert, const int* tile_row0, int max_tiles,
-                               int use_mma, void* stream) {
+                               int use_mma, float limit, float slope, float offset,
+                               void* stream) {
+  const GateRule gate{limit, slope, offset};
+  if (!gate_rule_ok(limit)) return kBadArgument;
   if (max_tiles <= 0) return kOk;
   if (N <= 0 || K <= 0 || lda < K || ldc < N || top <= 0 || mode < 0 || mode >= 2 + kUnaryKinds ||
       scale_at < 0 || scale_at > 2 || max_tiles > 65535 || a_dt != w_dt)
@@ -795,17 +813,17 @@ extern "C" int cretif_moe_gemm(const void* A, int a_dt, int lda, const void* W, 
     }
     moe_gemm_mma_kernel<<<grid, 128, smem, st>>>((const bf16*)A, lda, (const bf16*)W, C, ldc, N, K,
                                                  top, mode, scale_at, wts, order, offsets,
-                                                 tile_expert, tile_row0, a_vec, w_vec);
+                                                 tile_expert, tile_row0, a_vec, w_vec, gate);
     return launch_status();
   }
   if (a_dt == kF32)
     moe_gemm_simt_kernel<float, float><<<grid, 256, 0, st>>>(
         (const float*)A, lda, (const float*)W, C, ldc, N, K, top, mode, scale_at, wts, order,
-        offsets, tile_expert, tile_row0);
+        offsets, tile_expert, tile_row0, gate);
   else if (a_dt == kBF16)
     moe_gemm_simt_kernel<bf16, bf16><<<grid, 256, 0, st>>>(
         (const bf16*)A, lda, (const bf16*)W, C, ldc, N, K, top, mode, scale_at, wts, order,
-        offsets, tile_expert, tile_row0);
+        offsets, tile_expert, tile_row0, gate);
   else
     return kBadDType;
   return launch_status();
@@ -815,7 +833,10 @@ extern "C" int cretif_moe_gemm(const void* A, int a_dt, int lda, const void* W, 
 // with C's rows indexed by the pair.
 extern "C" int cretif_moe_gemv(const void* A, int a_dt, int lda, const void* W, int w_dt, void* C,
                                int ldc, int N, int K, int top, int mode, int scale_at,
-                               const int* ids, const float* wts, int P, int experts, void* stream) {
+                               const int* ids, const float* wts, int P, int experts, float limit,
+                               float slope, float offset, void* stream) {
+  const GateRule gate{limit, slope, offset};
+  if (!gate_rule_ok(limit)) return kBadArgument;
   if (P <= 0) return kOk;
   if (N <= 0 || K <= 0 || lda < K || ldc < N || top <= 0 || mode < 0 || mode >= 2 + kUnaryKinds ||
       scale_at < 0 || scale_at > 2 || P > 65535 || a_dt != w_dt)
@@ -834,7 +855,8 @@ extern "C" int cretif_moe_gemv(const void* A, int a_dt, int lda, const void* W, 
       if (err != cudaSuccess) return (int)err;
     }
     moe_gemv_kernel<float><<<grid, 256, smem, st>>>((const float*)A, lda, (const float*)W, C, ldc,
-                                                    N, K, top, mode, scale_at, ids, wts, vec, experts);
+                                                    N, K, top, mode, scale_at, ids, wts, vec, experts,
+                                                    gate);
   } else if (a_dt == kBF16) {
     if (smem > 48 * 1024) {
       cudaError_t err = cudaFuncSetAttribute(moe_gemv_kernel<bf16>,
@@ -842,7 +864,7 @@ extern "C" int cretif_moe_gemv(const void* A, int a_dt, int lda, const void* W, 
       if (err != cudaSuccess) return (int)err;
     }
     moe_gemv_kernel<bf16><<<grid, 256, smem, st>>>((const bf16*)A, lda, (const bf16*)W, C, ldc, N,
-                                                   K, top, mode, scale_at, ids, wts, vec, experts);
+                                                   K, top, mode, scale_at, ids, wts, vec, experts, gate);
   } else {
     return kBadDType;
   }
@@ -854,7 +876,7 @@ extern "C" int cretif_moe_gemv(const void* A, int a_dt, int lda, const void* W, 
 extern "C" int cretif_moe_combine(const float* rows, int ld, const int* place, int top,
                                   const float* wts, float* y, int T, int H, const int* ids,
                                   int experts, const float* id_wts, const void* x, int x_dt, int ldx,
-                                  const float* plus, void* stream) {
+                                  const float* plus, int add, void* x_out, void* stream) {
   if (T <= 0) return kOk;
   if (H <= 0 || ld < H || top <= 0 || (ids && (!id_wts || !x || ldx < H))) return kBadArgument;
   const bool vec = H % 4 == 0 && ld % 4 == 0 && (!ids || ldx % 4 == 0) &&
@@ -865,10 +887,12 @@ extern "C" int cretif_moe_combine(const float* rows, int ld, const int* place, i
   do {                                                                                              \
     if (vec)                                                                                        \
       moe_combine_kernel<TX, 4><<<blocks, 256, 0, st>>>(rows, ld, place, top, wts, y, T, H, ids,    \
-                                                        experts, id_wts, (const TX*)x, ldx, plus);  \
+                                                        experts, id_wts, (const TX*)x, ldx, plus,     \
+                                                        add, (__nv_bfloat16*)x_out);  \
     else                                                                                            \
       moe_combine_kernel<TX, 1><<<blocks, 256, 0, st>>>(rows, ld, place, top, wts, y, T, H, ids,    \
-                                                        experts, id_wts, (const TX*)x, ldx, plus);  \
+                                                        experts, id_wts, (const TX*)x, ldx, plus,     \
+                                                        add, (__nv_bfloat16*)x_out);  \
   } while (0)
   if (x_dt == kF32) CRETIF_COMBINE(float);
   else if (x_dt == kBF16) CRETIF_COMBINE(__nv_bfloat16);

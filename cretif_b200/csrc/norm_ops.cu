@@ -3,6 +3,8 @@
 // * rmsnorm_add: a norm on a sublayer's OUTPUT, fused with the residual addition:
 //   h[t] += y[t] * w * rsqrt(mean(y[t]^2) + eps).  Sum, scaling and addition are 32-bit.  The
 //   kernel can also leave the new rows in bfloat16 for the sublayer that reads them next.
+// * add_layernorm: the norm with the mean taken off and a bias, in front of a sublayer, fused with the
+//   residual addition that precedes it (the RMS norm's counterpart is in elementwise.cu).
 // * convert_rows: the residual stream handed to a sublayer that reads it without a norm
 //   (float32 -> the compute type).
 // * proj_norm_kv_append: RMS norms over whole query / key projections (all heads of a token
@@ -155,11 +157,149 @@ rmsnorm_add_row_block_kernel(float* __restrict__ h, const TY* __restrict__ y, in
     put(i, ld4(yrow + 4 * i), ld4(weight + 4 * i), ld4(hrow + 4 * i));
 }
 
+// Layer norm: v = h[src] (+ delta[src]); h[src] = v when write_h;
+// out[r] = (v - mean) / sqrt(mean((v - mean)^2) + eps) * w + b.  NT threads a row: 32 (many rows) or
+// 256 (few rows, a CTA each).  A row of up to 2048 columns stays in the threads' registers between
+// the sums (VEC); beyond that, and without VEC, it is read again.
+template <int NT, bool VEC, typename TD, typename TO>
+__global__ void __launch_bounds__(256)
+add_layernorm_kernel(float* h, const TD* __restrict__ delta, const float* __restrict__ weight,
+                     const float* __restrict__ bias, TO* __restrict__ out,
+                     const int* __restrict__ rows, int R, int H, float eps, int write_h) {
+  __shared__ float scratch[33];
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  const int r = blockIdx.x * (256 / NT) + threadIdx.x / NT, tid = threadIdx.x % NT;
+  constexpr int kKeep = 512 / NT;
+  const int n4 = VEC ? H >> 2 : 0;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 w[NT == 256 ? kKeep : 1], b[NT == 256 ? kKeep : 1];
+  if (VEC && NT == 256) {             // (they do not wait for the kernel before)
+#pragma unroll
+    for (int u = 0; u < kKeep; ++u) {
+      const int i = u * NT + tid;
+      w[NT == 256 ? u : 0] = i < n4 ? ld4(weight + 4 * i) : zero;
+      b[NT == 256 ? u : 0] = i < n4 ? ld4(bias + 4 * i) : zero;
+    }
+  }
+  asm volatile("griddepcontrol.wait;" ::: "memory");
+  if (r >= R) return;                 // (whole warps; with a CTA a row there is none beyond R)
+  auto total = [&](float v) { return NT == 32 ? warp_sum(v) : block_sum(v, scratch); };
+  const int src = rows ? rows[r] : r;
+  float* hrow = h + (size_t)src * H;
+  const TD* drow = delta ? delta + (size_t)src * H : nullptr;
+  TO* orow = out + (size_t)r * H;
+  if (!VEC) {
+    auto value = [&](int i) { return hrow[i] + (drow ? to_float(drow[i]) : 0.f); };
+    float s = 0.f, ss = 0.f;
+    for (int i = tid; i < H; i += NT) s += value(i);
+    const float mean = total(s) / (float)H;
+    for (int i = tid; i < H; i += NT) { const float d = value(i) - mean; ss += d * d; }
+    const float inv = rsqrtf(total(ss) / (float)H + eps);
+    for (int i = tid; i < H; i += NT) {
+      const float v = value(i);       // (read before the same thread replaces it)
+      if (write_h) hrow[i] = v;
+      orow[i] = from_float<TO>((v - mean) * inv * weight[i] + bias[i]);
+    }
+    return;
+  }
+  auto value = [&](int i) {
+    float4 v = ld4(hrow + 4 * i);
+    if (drow) {
+      const float4 d = ld4(drow + 4 * i);
+      v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
+    }
+    return v;
+  };
+  auto squares = [](const float4& v, float m) {
+    const float a = v.x - m, c = v.y - m, d = v.z - m, e = v.w - m;
+    return a * a + c * c + d * d + e * e;
+  };
+  float4 keep[kKeep];
+  float s = 0.f, ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u) {
+    const int i = u * NT + tid;
+    keep[u] = i < n4 ? value(i) : zero;
+    s += (keep[u].x + keep[u].y) + (keep[u].z + keep[u].w);
+  }
+  for (int i = kKeep * NT + tid; i < n4; i += NT) {
+    const float4 v = value(i);
+    s += (v.x + v.y) + (v.z + v.w);
+  }
+  const float mean = total(s) / (float)H;
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u)
+    if (u * NT + tid < n4) ss += squares(keep[u], mean);
+  for (int i = kKeep * NT + tid; i < n4; i += NT) ss += squares(value(i), mean);
+  const float inv = rsqrtf(total(ss) / (float)H + eps);
+  auto put = [&](int i, const float4& v, const float4& g, const float4& c) {
+    if (write_h) *reinterpret_cast<float4*>(hrow + 4 * i) = v;
+    const float4 y = make_float4((v.x - mean) * inv * g.x + c.x, (v.y - mean) * inv * g.y + c.y,
+                                 (v.z - mean) * inv * g.z + c.z, (v.w - mean) * inv * g.w + c.w);
+    if constexpr (sizeof(TO) == 4) *reinterpret_cast<float4*>(orow + 4 * i) = y;
+    else st4_bf16(orow + 4 * i, y);
+  };
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u) {
+    const int i = u * NT + tid;
+    if (i < n4)
+      put(i, keep[u], NT == 256 ? w[NT == 256 ? u : 0] : ld4(weight + 4 * i),
+          NT == 256 ? b[NT == 256 ? u : 0] : ld4(bias + 4 * i));
+  }
+  for (int i = kKeep * NT + tid; i < n4; i += NT)
+    put(i, value(i), ld4(weight + 4 * i), ld4(bias + 4 * i));
+}
+
+template <typename TD, typename TO>
+static int launch_layernorm(float* h, const TD* delta, const float* w, const float* b, TO* out,
+                            const int* rows, int R, int H, float eps, int write_h, cudaStream_t st) {
+  const bool vec = H % 4 == 0 && (((uintptr_t)h | (uintptr_t)delta | (uintptr_t)w | (uintptr_t)b |
+                                   (uintptr_t)out) & 15) == 0;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(R < 256 ? R : (R + 7) / 8);
+  cfg.blockDim = dim3(256);
+  cfg.stream = st;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = dependent_launch_enabled();
+  cfg.attrs = attr;
+  cfg.numAttrs = 1;
+  cudaError_t e;
+  if (R < 256)
+    e = vec ? cudaLaunchKernelEx(&cfg, add_layernorm_kernel<256, true, TD, TO>, h, delta, w, b, out,
+                                 rows, R, H, eps, write_h)
+            : cudaLaunchKernelEx(&cfg, add_layernorm_kernel<256, false, TD, TO>, h, delta, w, b, out,
+                                 rows, R, H, eps, write_h);
+  else
+    e = vec ? cudaLaunchKernelEx(&cfg, add_layernorm_kernel<32, true, TD, TO>, h, delta, w, b, out,
+                                 rows, R, H, eps, write_h)
+            : cudaLaunchKernelEx(&cfg, add_layernorm_kernel<32, false, TD, TO>, h, delta, w, b, out,
+                                 rows, R, H, eps, write_h);
+  return e == cudaSuccess ? launch_status() : (int)e;
+}
+
 template <typename TO>
 __global__ void convert_rows_kernel(const float* __restrict__ h, TO* __restrict__ out,
                                     size_t total) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i < total) out[i] = from_float<TO>(h[i]);
+}
+
+// The same into some columns of a wider matrix, V columns a thread.
+template <typename TO, int V>
+__global__ void __launch_bounds__(256)
+convert_into_kernel(const float* __restrict__ h, TO* __restrict__ out, int ldo, int H, long long total) {
+  const long long idx = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (idx >= total) return;
+  const long long r = idx / H;
+  TO* to = out + (size_t)r * ldo + (size_t)(idx - r * H);
+  if constexpr (V == 4) {
+    const float4 v = ld4(h + idx);
+    if constexpr (sizeof(TO) == 4) *reinterpret_cast<float4*>(to) = v;
+    else st4_bf16(to, v);
+  } else {
+    *to = from_float<TO>(h[idx]);
+  }
 }
 
 template <typename T>
@@ -251,6 +391,27 @@ extern "C" int cretif_rmsnorm_add(float* h, const void* y, int y_dt, int ldy, co
   return launch_status();
 }
 
+extern "C" int cretif_add_layernorm(float* h, const void* delta, int delta_dt, const float* weight,
+                                    const float* bias, void* out, int out_dt, const int* rows, int R,
+                                    int H, float eps, int write_h, void* stream) {
+  if (R <= 0) return kOk;
+  if (H <= 0 || !weight || !bias || (rows && write_h)) return kBadArgument;
+  if ((delta && delta_dt != kF32 && delta_dt != kBF16) || (out_dt != kF32 && out_dt != kBF16))
+    return kBadDType;
+  cudaStream_t st = (cudaStream_t)stream;
+  typedef __nv_bfloat16 bf16;
+  const bool dbf = delta && delta_dt == kBF16;
+  if (out_dt == kF32)
+    return dbf ? launch_layernorm(h, (const bf16*)delta, weight, bias, (float*)out, rows, R, H, eps,
+                                  write_h, st)
+               : launch_layernorm(h, (const float*)delta, weight, bias, (float*)out, rows, R, H, eps,
+                                  write_h, st);
+  return dbf ? launch_layernorm(h, (const bf16*)delta, weight, bias, (bf16*)out, rows, R, H, eps,
+                                write_h, st)
+             : launch_layernorm(h, (const float*)delta, weight, bias, (bf16*)out, rows, R, H, eps,
+                                write_h, st);
+}
+
 extern "C" int cretif_convert_rows(const float* h, void* out, int out_dt, long long total,
                                    void* stream) {
   if (total <= 0) return kOk;
@@ -263,6 +424,26 @@ extern "C" int cretif_convert_rows(const float* h, void* out, int out_dt, long l
                                                               (size_t)total);
   else
     return kBadDType;
+  return launch_status();
+}
+
+extern "C" int cretif_convert_into(const float* h, void* out, int out_dt, int ldo, int R, int H,
+                                   void* stream) {
+  if (R <= 0) return kOk;
+  if (H <= 0 || ldo < H) return kBadArgument;
+  if (out_dt != kF32 && out_dt != kBF16) return kBadDType;
+  cudaStream_t st = (cudaStream_t)stream;
+  const long long total = (long long)R * H;
+  const bool vec = H % 4 == 0 && ldo % 4 == 0 && (((uintptr_t)h | (uintptr_t)out) & 15) == 0;
+  const unsigned blocks = (unsigned)(((vec ? total / 4 : total) + 255) / 256);
+  if (out_dt == kF32) {
+    if (vec) convert_into_kernel<float, 4><<<blocks, 256, 0, st>>>(h, (float*)out, ldo, H, total);
+    else convert_into_kernel<float, 1><<<blocks, 256, 0, st>>>(h, (float*)out, ldo, H, total);
+  } else {
+    typedef __nv_bfloat16 bf16;
+    if (vec) convert_into_kernel<bf16, 4><<<blocks, 256, 0, st>>>(h, (bf16*)out, ldo, H, total);
+    else convert_into_kernel<bf16, 1><<<blocks, 256, 0, st>>>(h, (bf16*)out, ldo, H, total);
+  }
   return launch_status();
 }
 

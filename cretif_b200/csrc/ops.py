@@ -114,6 +114,25 @@ def _rows(t: torch.Tensor, name: str) -> int:
     return t.stride(0)
 
 
+def _gate_args(gate):
+    """(limit, slope, offset) of a gate rule as the kernels take them; None: silu(g) · u."""
+    limit, slope, offset = gate if gate is not None else (0.0, 1.0, 0.0)
+    if limit < 0 or (gate is not None and not limit > 0):
+        raise KernelError("a clamped gate needs a limit above zero")
+    return ctypes.c_float(limit), ctypes.c_float(slope), ctypes.c_float(offset)
+
+
+def _mul_args(mul, T: int, width: int, dtype):
+    """(table, its row stride, its rows, a row per token) of a factor by token, or of none."""
+    if mul is None:
+        return None, 0, 0, None
+    table, ids = mul
+    _need(table, "table", dtype, 2); _need(ids, "ids", torch.int32, 1)
+    if table.shape[1] < width or ids.numel() < T:
+        raise KernelError("a factor by token: a table as wide as the rows and an id per row")
+    return _p(table), _rows(table, "table"), table.shape[0], _p(ids)
+
+
 # ------------------------------------------------------------------ elementwise
 def embed_rows(table, ids, out, fault, positions=None, tok_pos=None, scale: float = 1.0) -> None:
     """A token's row times ``scale``; ``positions`` [P, H] (same type as ``table``) with
@@ -160,14 +179,42 @@ def add_rmsnorm(h, delta, weight, out, eps: float, rows=None, write_h: bool = Tr
                                     ctypes.c_float(eps), int(write_h), _stream()), "add_rmsnorm")
 
 
-def silu_mul(gu, act, block: int = 0) -> None:
-    """act = silu(gate) * up.  ``block`` = 0: gu rows are [gate | up]; ``block`` = b: groups of b
+def add_layernorm(h, delta, weight, bias, out, eps: float, rows=None, write_h: bool = True) -> None:
+    """``v = h (+ delta)``, optionally written back, and ``out = (v - mean) / sqrt(var + eps) * weight
+    + bias`` row by row (``rows``: the source row of every output row)."""
+    _need(h, "h", torch.float32, 2); _need(out, "out", dim=2)
+    H = h.shape[1]
+    for name, t in (("weight", weight), ("bias", bias)):
+        _need(t, name, torch.float32, 1)
+        if t.numel() != H or not t.is_contiguous():
+            raise KernelError(f"add_layernorm: {name} must have {H} elements")
+    if not h.is_contiguous() or not out.is_contiguous():
+        raise KernelError("add_layernorm: h and out must be contiguous")
+    if delta is not None:
+        _need(delta, "delta", dim=2)
+        if delta.shape != h.shape or not delta.is_contiguous():
+            raise KernelError("add_layernorm: delta must match h")
+    R = h.shape[0] if rows is None else rows.numel()
+    if tuple(out.shape) != (R, H):
+        raise KernelError(f"add_layernorm: out must be [{R}, {H}]")
+    if rows is not None:
+        _need(rows, "rows", torch.int32, 1)
+    _check(lib().cretif_add_layernorm(
+        _p(h), _p(delta), 0 if delta is None else _dt(delta), _p(weight), _p(bias), _p(out), _dt(out),
+        _p(rows), R, H, ctypes.c_float(eps), int(write_h and rows is None and delta is not None),
+        _stream()), "add_layernorm")
+
+
+def silu_mul(gu, act, block: int = 0, gate=None) -> None:
+    """act = silu(gate) * up, or what ``gate`` (limit, slope, offset) makes of the two: with the gate
+    at most ``limit`` and up within ±``limit``, gate · sigmoid(slope · gate) · (up + offset).  ``block`` = 0: gu rows are [gate | up]; ``block`` = b: groups of b
     gate columns each followed by their b up columns."""
     _need(gu, "gu", dim=2); _need(act, "act", gu.dtype, 2)
     T, I = act.shape
     if tuple(gu.shape) != (T, 2 * I) or not gu.is_contiguous() or not act.is_contiguous():
         raise KernelError(f"silu_mul: gu must be contiguous [{T}, {2 * I}]")
-    _check(lib().cretif_silu_mul(_p(gu), _p(act), _dt(gu), T, I, block, _stream()), "silu_mul")
+    _check(lib().cretif_silu_mul(_p(gu), _p(act), _dt(gu), T, I, block, *_gate_args(gate),
+                                 _stream()), "silu_mul")
 
 
 def rope_kv_append(qkv, cos, sin, pairing: int, rot_dim: int, nh: int, nkv: int, hd: int,
@@ -279,6 +326,15 @@ def convert_rows(h, out) -> None:
         raise KernelError("convert_rows: out must match h, both contiguous")
     _check(lib().cretif_convert_rows(_p(h), _p(out), _dt(out), ctypes.c_longlong(h.numel()),
                                      _stream()), "convert_rows")
+
+
+def convert_into(h, out) -> None:
+    """out = h in out's element type; ``out`` may be some columns of a wider matrix."""
+    _need(h, "h", torch.float32, 2); _need(out, "out", dim=2)
+    if h.shape != out.shape or not h.is_contiguous():
+        raise KernelError("convert_into: out must match h, h contiguous")
+    _check(lib().cretif_convert_into(_p(h), _p(out), _dt(out), _rows(out, "out"), h.shape[0],
+                                     h.shape[1], _stream()), "convert_into")
 
 
 def proj_norm_kv_append(rows, q_dim: int, wq, nkv: int, hd: int, wk, eps: float, tok_pos, tok_seq,
@@ -412,11 +468,14 @@ def projnorm_rope_kv_append(proj, bias, wq, wk, eps: float, cos, sin, pairing: i
                             tok_pos, tok_seq, seq_slot, nh: int, nkv: int, hd: int, vd: int, q_out,
                             table=None, kc=None, vc=None, block_tokens: int = 64,
                             write_cache: bool = True, fault=None, v_scale: float = 1.0,
-                            pool=None) -> None:
+                            pool=None, conv=None) -> None:
     """``headnorm_rope_kv_append`` with the norms over the whole query and the whole key projection
     (``wq`` [nh hd], ``wk`` [nkv hd] float32), float32 ``proj``, and v times ``v_scale``.  ``pool``
     (a PoolView; steps of one token a sequence): the entry of a block of tokens that a token
-    completes is written too."""
+    completes is written too.  ``conv`` (``(w, state, seq_start, save)``): before the norms every
+    channel passes a causal convolution over time with weights ``w`` [taps, C] float32; ``state``
+    [slots, >= C (taps - 1)] are the slots' saved inputs (None with one tap), which a step of one
+    token a sequence brings up to date with ``save``."""
     _need(proj, "proj", torch.float32, 2); _need(q_out, "q_out", dim=2)
     _need(wq, "wq", torch.float32, 1)
     T = proj.shape[0]
@@ -450,6 +509,20 @@ def projnorm_rope_kv_append(proj, bias, wq, wk, eps: float, cos, sin, pairing: i
             raise KernelError("projnorm_rope_kv_append: caches must be contiguous [blocks, "
                               f"{nkv}, {block_tokens}, {hd}] and [..., {vd}]")
         _need_pool(pool, kc, vc)
+    conv_w = state = seq_start = None
+    taps = stride = save = 0
+    if conv is not None:
+        conv_w, state, seq_start, save = conv
+        _need(conv_w, "conv weights", torch.float32, 2); _need(seq_start, "seq_start", torch.int32, 1)
+        taps = conv_w.shape[0]
+        if conv_w.shape[1] != n_in or not conv_w.is_contiguous() or bias is not None or not write_cache:
+            raise KernelError("projnorm_rope_kv_append: the convolution has a weight per tap and column, "
+                              "and comes without bias and with the cache write")
+        if taps > 1:
+            _need(state, "saved inputs", torch.float32, 2)
+            if state.stride(1) != 1 or state.shape[1] < n_in * (taps - 1):
+                raise KernelError("projnorm_rope_kv_append: saved inputs are [slots, >= C (taps - 1)]")
+            stride = state.stride(0)
     if fault is None:
         fault = fault_word(proj.device)
     _check(lib().cretif_projnorm_rope_kv_append(
@@ -457,8 +530,9 @@ def projnorm_rope_kv_append(proj, bias, wq, wk, eps: float, cos, sin, pairing: i
         _p(sin), pairing, rot_dim, _p(tok_pos), _p(tok_seq), _p(seq_slot), nh, nkv, hd, vd,
         ctypes.c_float(v_scale), _p(q_out), _rows(q_out, "q_out"), _dt(q_out), _p(table),
         table.stride(0) if table is not None else 0, _p(kc), _p(vc), block_tokens,
-        int(write_cache), *_pool_args(pool if write_cache else None), T, _p(fault), _stream()),
-        "projnorm_rope_kv_append")
+        int(write_cache), *_pool_args(pool if write_cache else None), _p(conv_w), taps,
+        _p(state if taps > 1 else None), ctypes.c_longlong(stride), _p(seq_start), int(bool(save)), T,
+        _p(fault), _stream()), "projnorm_rope_kv_append")
 
 
 def _need_pool(pool, kc, vc) -> None:
@@ -592,8 +666,8 @@ def gate_heads(o, g, nh: int, vd: int) -> None:
 ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "gelu": 3}
 
 
-def activation(x, out, kind: str) -> None:
-    """``out = act(x)`` element by element: ``relu2`` (the square of relu), ``gelu_tanh``,
+def activation(x, out, kind: str, mul=None) -> None:
+    """``out = act(x)`` (times row ids[t] of ``table`` with ``mul`` = (table of out's type, ids)) element by element: ``relu2`` (the square of relu), ``gelu_tanh``,
     ``silu``, ``gelu`` (the exact form, with the error function); ``x`` float32 or of ``out``'s type."""
     _need(x, "x", dim=2); _need(out, "out", dim=2)
     if kind not in ACTIVATIONS:
@@ -602,7 +676,8 @@ def activation(x, out, kind: str) -> None:
         raise KernelError("activation: out has x's shape, x is float32 or of out's type")
     _check(lib().cretif_activation(_p(x), _rows(x, "x"), _dt(x), _p(out), _rows(out, "out"),
                                    _dt(out), x.shape[0], x.shape[1], ACTIVATIONS[kind],
-                                   _stream()), "activation")
+                                   *_mul_args(mul, x.shape[0], x.shape[1], out.dtype), _stream()),
+           "activation")
 
 
 def scale_in_place(z, factor: float) -> None:
@@ -709,6 +784,53 @@ def matrix_memory(proj, bias_i, bias_f, cap: float, q_scale: float, state, cu_se
         _p(scratch[n_o:]), _p(scratch[n_o + T * H:]), _p(gates), _p(out), _dt(out),
         _rows(out, "out"), int(write_state), T, {"auto": 0, "token": 1, "chunk": 2}[form],
         _stream()), "matrix_memory", kernels=3 if chunks else 2)
+
+
+def state_space(proj, conv_w, conv_b, a_log, dt_bias, d_skip, state, inputs_at: int, cu_seqlens,
+                seq_slot, tok_seq, B: int, H: int, G: int, N: int, e: int, parts: int, norm_w,
+                eps: float, out, write_state: bool = True, save_inputs: bool = False,
+                form: str = "auto") -> None:
+    """The Mamba-2 recurrence over the step's tokens of every (sequence, head), from and to ``state``
+    (view [slots, >= inputs_at + C (taps - 1)] float32: S, then the convolution's saved inputs), then
+    ``y silu(z)`` normed in ``parts`` equal parts times ``norm_w`` [H·e] -> ``out`` [T, H·e].  ``proj``
+    rows (float32): [z | x | B | C | dt]; ``conv_w`` [taps, C] and ``conv_b`` [C] with
+    C = H·e + 2·G·N.  ``save_inputs``: the step brings one token a sequence and the saved inputs are
+    brought up to date (else ``delta_conv_state`` does).  ``form``: ``"token"`` walks the tokens one by
+    one, ``"chunk"`` takes 64 at a time as matrix products (refused where sizes or addresses rule out
+    16-byte accesses), ``"auto"`` takes chunks where the step brings 16 tokens a sequence or more and
+    they are allowed."""
+    _need(proj, "proj", torch.float32, 2); _need(state, "state", torch.float32, 2)
+    _need(out, "out", dim=2); _need(conv_w, "conv_w", torch.float32, 2)
+    inner, C = H * e, H * e + 2 * G * N
+    taps = conv_w.shape[0]
+    for name, t, n in (("conv_b", conv_b, C), ("a_log", a_log, H), ("dt_bias", dt_bias, H),
+                       ("d_skip", d_skip, H), ("norm_w", norm_w, inner)):
+        _need(t, name, torch.float32, 1)
+        if t.numel() != n or not t.is_contiguous():
+            raise KernelError(f"state_space: {name} has {n} numbers")
+    for name, t in (("cu_seqlens", cu_seqlens), ("seq_slot", seq_slot), ("tok_seq", tok_seq)):
+        _need(t, name, torch.int32, 1)
+    T = proj.shape[0]
+    if (conv_w.shape[1] != C or not conv_w.is_contiguous() or state.stride(1) != 1
+            or state.shape[1] < inputs_at + C * (taps - 1) or inputs_at < H * N * e
+            or out.shape[0] != T or out.shape[1] < inner or proj.shape[1] < inner + C + H
+            or tok_seq.numel() < T or H % G or inner % parts):
+        raise KernelError("state_space: the sizes do not fit")
+    chunks = form == "chunk" or (form == "auto" and T >= 16 * B)
+    ldx = -(-C // 4) * 4
+    y = torch.empty((T, inner), dtype=torch.float32, device=proj.device)
+    xbc = dts = sums = None
+    if chunks:
+        xbc = torch.empty((T, ldx), dtype=torch.float32, device=proj.device)
+        dts = torch.empty(H * T, dtype=torch.float32, device=proj.device)
+        sums = torch.empty(H * T, dtype=torch.float64, device=proj.device)
+    _check(lib().cretif_state_space(
+        _p(proj), _rows(proj, "proj"), _p(conv_w), _p(conv_b), taps, _p(a_log), _p(dt_bias),
+        _p(d_skip), _p(state), ctypes.c_longlong(state.stride(0)), ctypes.c_longlong(inputs_at),
+        _p(cu_seqlens), _p(seq_slot), _p(tok_seq), B, H, G, N, e, _p(y), _p(xbc), ldx, _p(dts),
+        _p(sums), parts, _p(norm_w), ctypes.c_float(eps), _p(out), _dt(out), _rows(out, "out"),
+        int(write_state), int(save_inputs), T, {"auto": 0, "token": 1, "chunk": 2}[form], _stream()),
+        "state_space", kernels=4 if chunks else 2)
 
 
 def heads_out_norm(o_raw, gate, norm_w, eps: float, out, H: int, e: int,
@@ -900,18 +1022,26 @@ def _route_rule(E: int, top: int, groups: int, keep: int) -> None:
                           f"{keep} hold {top} experts")
 
 
-def _correction(correction, E: int) -> None:
+def _correction(correction, E: int, name: str = "correction") -> None:
     if correction is not None:
-        _need(correction, "correction", torch.float32, 1)
+        _need(correction, name, torch.float32, 1)
         if correction.numel() != E or not correction.is_contiguous():
-            raise KernelError("routing: the correction has a number per router output")
+            raise KernelError(f"routing: the {name} has a number per router output")
+
+
+def _scores(softmax) -> int:
+    """False: logistic scores; True: the softmax over all outputs; "chosen": exponentials relative to
+    the largest logit, which divided by their sum are the softmax over the chosen outputs alone."""
+    return 2 if softmax == "chosen" else int(bool(softmax))
 
 
 def moe_route(x, router_w, top: int, ids, wts, renorm: bool = False, groups: int = 0,
-              keep: int = 0, sum_eps: float = 0.0, softmax: bool = False, group_best: bool = False,
-              correction=None) -> None:
+              keep: int = 0, sum_eps: float = 0.0, softmax=False, group_best: bool = False,
+              correction=None, bias=None) -> None:
     """ids/wts [T, top]: the ``top`` experts with the largest scores per token, a score being
-    sigmoid(router_w · x) or (``softmax``) its share of the softmax over all outputs.
+    sigmoid(router_w · x) or (``softmax``) its share of the softmax over all outputs; ``softmax``
+    "chosen" with ``renorm``: of the softmax over the chosen ones.  ``bias`` (float32 [E]) is added to
+    the logits.
     ``correction`` (float32 [E]) is added to the scores for the choice, not for the weights.
     ``groups`` > 1: the experts form that many equal groups of neighbours, a group's score is
     the sum of its two largest choice scores (``group_best``: the largest), and only experts of the
@@ -928,15 +1058,16 @@ def moe_route(x, router_w, top: int, ids, wts, renorm: bool = False, groups: int
         raise KernelError(f"moe_route: {top} of {E} experts (at most 256) cannot be chosen")
     _route_rule(E, top, groups, keep)
     _correction(correction, E)
+    _correction(bias, E, "bias")
     _check(lib().cretif_moe_route(_p(x), _dt(x), _rows(x, "x"), _p(router_w), E, H, top,
                                   int(renorm), int(groups), int(keep), ctypes.c_float(sum_eps),
-                                  int(softmax), int(group_best), _p(correction),
+                                  _scores(softmax), int(group_best), _p(correction), _p(bias),
                                   _p(ids), _p(wts), T, _stream()), "moe_route")
 
 
 def moe_topk(logits, top: int, ids, wts, renorm: bool = False, groups: int = 0, keep: int = 0,
-             sum_eps: float = 0.0, softmax: bool = False, group_best: bool = False,
-             correction=None) -> None:
+             sum_eps: float = 0.0, softmax=False, group_best: bool = False,
+             correction=None, bias=None) -> None:
     """``moe_route``'s choice from router logits [T, E] (float32) that a matrix product left."""
     _need(logits, "logits", torch.float32, 2); _need(ids, "ids", torch.int32, 2)
     _need(wts, "wts", torch.float32, 2)
@@ -946,9 +1077,11 @@ def moe_topk(logits, top: int, ids, wts, renorm: bool = False, groups: int = 0, 
         raise KernelError("moe_topk: sizes do not fit")
     _route_rule(E, top, groups, keep)
     _correction(correction, E)
+    _correction(bias, E, "bias")
     _check(lib().cretif_moe_topk(_p(logits), _rows(logits, "logits"), E, top, int(renorm),
-                                 int(groups), int(keep), ctypes.c_float(sum_eps), int(softmax),
-                                 int(group_best), _p(correction), _p(ids), _p(wts), T, _stream()),
+                                 int(groups), int(keep), ctypes.c_float(sum_eps),
+                                 _scores(softmax), int(group_best), _p(correction), _p(bias), _p(ids),
+                                 _p(wts), T, _stream()),
            "moe_topk")
 
 
@@ -978,9 +1111,10 @@ def moe_act_mode(kind: str) -> int:
 
 
 def moe_gemm(a, w, c, top: int, mode: int, scale_at: int, wts, order, offsets, tile_expert,
-             tile_row0) -> None:
+             tile_row0, gate=None) -> None:
     """Grouped product over the sorted rows.  mode 0: ``a`` [tokens, K], ``w`` [E, 2N, K]
-    (gate rows then up rows), ``c`` [P, N] = silu(s g)(s u) (scale_at 1) or silu(g) u; mode 1:
+    (gate rows then up rows), ``c`` [P, N] = silu(s g)(s u) (scale_at 1) or silu(g) u (``gate``: a
+    clamped gate instead, as in ``silu_mul``); mode 1:
     ``a`` [P, K] sorted rows, ``w`` [E, N, K], ``c`` [P, N] float32 (scale_at 2: times s);
     mode ``moe_act_mode(kind)``: experts without a gate, ``a`` as in mode 0, ``w`` [E, N, K],
     ``c`` = act(s · product)."""
@@ -994,10 +1128,10 @@ def moe_gemm(a, w, c, top: int, mode: int, scale_at: int, wts, order, offsets, t
     _check(lib().cretif_moe_gemm(
         _p(a), _dt(a), _rows(a, "a"), _p(w), _dt(w), _p(c), _rows(c, "c"), N, K, top, mode,
         scale_at, _p(wts), _p(order), _p(offsets), _p(tile_expert), _p(tile_row0),
-        tile_expert.numel(), use_mma, _stream()), "moe_gemm")
+        tile_expert.numel(), use_mma, *_gate_args(gate), _stream()), "moe_gemm")
 
 
-def moe_gemv(a, w, c, top: int, mode: int, scale_at: int, ids, wts) -> None:
+def moe_gemv(a, w, c, top: int, mode: int, scale_at: int, ids, wts, gate=None) -> None:
     """``moe_gemm`` for a handful of pairs, in the pairs' own order (nothing is sorted): a CTA
     per pair and 16 output columns streams the expert's rows once.  Pairs whose id is no expert's
     (identities) are left out."""
@@ -1010,7 +1144,7 @@ def moe_gemv(a, w, c, top: int, mode: int, scale_at: int, ids, wts) -> None:
         raise KernelError("moe_gemv: sizes or element types do not fit")
     _check(lib().cretif_moe_gemv(
         _p(a), _dt(a), _rows(a, "a"), _p(w), _dt(w), _p(c), _rows(c, "c"), N, K, top, mode,
-        scale_at, _p(ids), _p(wts), P, w.shape[0], _stream()), "moe_gemv")
+        scale_at, _p(ids), _p(wts), P, w.shape[0], *_gate_args(gate), _stream()), "moe_gemv")
 
 
 MOE_TC_TILE = 128
@@ -1056,8 +1190,8 @@ def moe_tc_supported(x, w_gu, w_down, gated: bool = True) -> bool:
             and F % (64 if gated else 8) == 0 and not _moe_simt_only)
 
 
-def gemm_tc_silu_grouped(xs, w_gu, act, tile_expert, used) -> None:
-    """act = silu(xs Wg[e]ᵀ) ⊙ (xs Wu[e]ᵀ) tile by tile; ``w_gu`` [E, 2F, K] with gate and up
+def gemm_tc_silu_grouped(xs, w_gu, act, tile_expert, used, gate=None) -> None:
+    """act = silu(xs Wg[e]ᵀ) ⊙ (xs Wu[e]ᵀ) tile by tile (``gate``: as in ``silu_mul``); ``w_gu`` [E, 2F, K] with gate and up
     rows interleaved in blocks of 64 inside each expert."""
     _need(xs, "xs", torch.bfloat16, 2); _need(w_gu, "w_gu", torch.bfloat16, 3)
     _need(act, "act", torch.bfloat16, 2)
@@ -1069,7 +1203,7 @@ def gemm_tc_silu_grouped(xs, w_gu, act, tile_expert, used) -> None:
         raise KernelError("gemm_tc_silu_grouped: sizes do not fit")
     _check(lib().cretif_gemm_tc_silu_grouped(
         _p(xs), _p(w_gu), _p(act), M, F, K, _rows(xs, "xs"), K, E, _p(tile_expert), _p(used),
-        _p(fault_word(xs.device)), _stream()), "gemm_tc_silu_grouped")
+        *_gate_args(gate), _p(fault_word(xs.device)), _stream()), "gemm_tc_silu_grouped")
 
 
 def gemm_tc_act_grouped(a, w, c, tile_expert, used, kind: str) -> None:
@@ -1101,12 +1235,14 @@ def gemm_tc_grouped(a, w, c, tile_expert, used) -> None:
         _p(used), _p(fault_word(a.device)), _stream()), "gemm_tc_grouped")
 
 
-def moe_combine(rows, place, top: int, y, wts=None, identity=None, plus=None) -> None:
+def moe_combine(rows, place, top: int, y, wts=None, identity=None, plus=None, add: bool = False,
+                x_out=None) -> None:
     """y[t] = the sum of the token's ``top`` rows of ``rows`` (float32), in their order, each
     times its weight when ``wts`` is given; ``place`` None: the rows are in the pairs' own
     order.  ``identity`` (``(ids, experts, weights, x)``): a pair whose id is ``experts`` or more has
     no row of its own and adds its weight times the token's row of ``x``.  ``plus`` (float32, like
-    ``y``) is added last."""
+    ``y``) is added last.  ``add``: the sum is added to ``y`` (the residual stream), and ``x_out``
+    (bfloat16, optional) receives its new rows."""
     _need(rows, "rows", torch.float32, 2); _need(y, "y", torch.float32, 2)
     if place is not None:
         _need(place, "place", torch.int32)
@@ -1118,6 +1254,10 @@ def moe_combine(rows, place, top: int, y, wts=None, identity=None, plus=None) ->
         _need(plus, "plus", torch.float32, 2)
         if plus.shape != y.shape or not plus.is_contiguous():
             raise KernelError("moe_combine: plus must match y")
+    if x_out is not None:
+        _need(x_out, "x_out", torch.bfloat16, 2)
+        if x_out.shape != y.shape or not x_out.is_contiguous():
+            raise KernelError("moe_combine: x_out must match y")
     ids = id_wts = x = None
     experts = ldx = x_dt = 0
     if identity is not None:
@@ -1129,7 +1269,7 @@ def moe_combine(rows, place, top: int, y, wts=None, identity=None, plus=None) ->
         ldx, x_dt = _rows(x, "x"), _dt(x)
     _check(lib().cretif_moe_combine(_p(rows), _rows(rows, "rows"), _p(place), top, _p(wts), _p(y),
                                     T, H, _p(ids), int(experts), _p(id_wts), _p(x), x_dt, ldx,
-                                    _p(plus), _stream()), "moe_combine")
+                                    _p(plus), int(add), _p(x_out), _stream()), "moe_combine")
 
 
 # ------------------------------------------------------------------ attention
@@ -1283,9 +1423,10 @@ def set_tc_epilogue_warps(n: int) -> int:
 
 
 def gemm_tc(x, w, out, accumulate: bool = False, bn: int = 0, alpha: float = 1.0,
-            unary: Optional[str] = None) -> None:
+            unary: Optional[str] = None, mul=None) -> None:
     """out[M,N] (+)= alpha · x[M,K] · w[N,K]ᵀ with TMA, tcgen05.mma and a TMEM accumulator;
-    ``unary`` (a key of ACTIVATIONS; stores only) is applied to the 32-bit sums."""
+    ``unary`` (a key of ACTIVATIONS; stores only) is applied to the 32-bit sums, and what is stored
+    of row m is multiplied by row ids[m] of ``table`` with ``mul`` = (table, ids)."""
     _need(x, "x", torch.bfloat16, 2); _need(w, "w", torch.bfloat16, 2); _need(out, "out", dim=2)
     M, K = x.shape
     N = w.shape[0]
@@ -1295,6 +1436,7 @@ def gemm_tc(x, w, out, accumulate: bool = False, bn: int = 0, alpha: float = 1.0
                                 _rows(w, "w"), _rows(out, "out"), int(accumulate), bn,
                                 ctypes.c_float(alpha),
                                 0 if unary is None else 1 + ACTIVATIONS[unary],
+                                *_mul_args(mul, M, N, torch.bfloat16),
                                 _p(fault_word(x.device)), _stream()), "gemm_tc")
 
 
@@ -1458,9 +1600,9 @@ FUSED_MAX_ROWS = 128     # the kernels' limit; the parts choose how far they use
 FUSED_GROUPS_MAX_BYTES = 16 << 20
 
 
-def fused_supported(M: int, K: int, w, norm: bool = True) -> bool:
+def fused_supported(M: int, K: int, w, norm=True) -> bool:
     """Whether the fused kernel takes M rows of width K against w (``norm``: with the norm
-    prologue, which keeps the normed rows in shared memory)."""
+    prologue, which keeps the normed rows in shared memory; 2: a layer norm)."""
     if M > 32 and w.numel() * w.element_size() > FUSED_GROUPS_MAX_BYTES:
         return False
     return (w.dtype == torch.bfloat16 and 0 < M <= FUSED_MAX_ROWS and K % 8 == 0
@@ -1494,9 +1636,10 @@ def set_dependent_launch(on: bool) -> bool:
 
 
 def fused_norm_linear(h, norm_w, eps: float, w, out, rows=None, accumulate: bool = False,
-                      unary: Optional[str] = None, alpha: float = 1.0) -> None:
+                      unary: Optional[str] = None, alpha: float = 1.0, norm_b=None) -> None:
     """out (+)= alpha · bf16(rmsnorm(h[rows])) · wᵀ in one kernel (decode-sized row counts); ``unary``
-    (a key of ACTIVATIONS; stores only) is applied to the 32-bit sums."""
+    (a key of ACTIVATIONS; stores only) is applied to the 32-bit sums.  ``norm_b`` [K]: the norm takes
+    the mean off and adds it (a layer norm)."""
     _need(h, "h", torch.float32, 2); _need(norm_w, "norm weight", torch.float32, 1)
     _need(w, "w", torch.bfloat16, 2); _need(out, "out", dim=2)
     K = h.shape[1]
@@ -1504,10 +1647,16 @@ def fused_norm_linear(h, norm_w, eps: float, w, out, rows=None, accumulate: bool
     N = w.shape[0]
     if w.shape[1] != K or tuple(out.shape) != (M, N) or not h.is_contiguous():
         raise KernelError("fused_norm_linear: shapes do not fit")
-    _check(lib().cretif_fused_linear(None, 0, _p(h), _p(norm_w), _p(rows), ctypes.c_float(eps),
+    if norm_b is not None:
+        _need(norm_b, "norm bias", torch.float32, 1)
+        if norm_b.numel() != K or not norm_b.is_contiguous():
+            raise KernelError("fused_norm_linear: the norm's bias has a number per column")
+    _check(lib().cretif_fused_linear(None, 0, _p(h), _p(norm_w), _p(norm_b), _p(rows),
+                                     ctypes.c_float(eps),
                                      _p(w), _rows(w, "w"), _p(out), _dt(out), _rows(out, "out"),
                                      int(accumulate), ctypes.c_float(alpha),
-                                     0 if unary is None else 1 + ACTIVATIONS[unary], M, N, K,
+                                     0 if unary is None else 1 + ACTIVATIONS[unary],
+                                     *_mul_args(None, M, N, None), M, N, K,
                                      _p(fault_word(h.device)), _stream()), "fused_norm_linear")
 
 
@@ -1519,31 +1668,35 @@ def fused_linear_add(x, w, h) -> None:
     N = w.shape[0]
     if w.shape[1] != K or tuple(h.shape) != (M, N):
         raise KernelError("fused_linear_add: shapes do not fit")
-    _check(lib().cretif_fused_linear(_p(x), _rows(x, "x"), None, None, None, ctypes.c_float(0.0),
+    _check(lib().cretif_fused_linear(_p(x), _rows(x, "x"), None, None, None, None,
+                                     ctypes.c_float(0.0),
                                      _p(w), _rows(w, "w"), _p(h), F32, _rows(h, "h"), 1,
-                                     ctypes.c_float(1.0), 0, M, N, K,
+                                     ctypes.c_float(1.0), 0, *_mul_args(None, M, N, None), M, N, K,
                                      _p(fault_word(h.device)), _stream()), "fused_linear_add")
 
 
 def fused_linear_x(x, w, out, accumulate: bool = False, alpha: float = 1.0,
-                   unary: Optional[str] = None) -> None:
+                   unary: Optional[str] = None, mul=None) -> None:
     """out (+)= alpha · x · wᵀ with the few-token kernels (x bfloat16; out bfloat16, or float32
     which may be added to); ``unary`` (a key of ACTIVATIONS; stores only) is applied to the
-    32-bit sums."""
+    32-bit sums, ``mul`` as in ``gemm_tc``."""
     _need(x, "x", torch.bfloat16, 2); _need(w, "w", torch.bfloat16, 2); _need(out, "out", dim=2)
     M, K = x.shape
     N = w.shape[0]
     if w.shape[1] != K or tuple(out.shape) != (M, N):
         raise KernelError("fused_linear_x: shapes do not fit")
-    _check(lib().cretif_fused_linear(_p(x), _rows(x, "x"), None, None, None, ctypes.c_float(0.0),
+    _check(lib().cretif_fused_linear(_p(x), _rows(x, "x"), None, None, None, None,
+                                     ctypes.c_float(0.0),
                                      _p(w), _rows(w, "w"), _p(out), _dt(out), _rows(out, "out"),
                                      int(accumulate), ctypes.c_float(alpha),
-                                     0 if unary is None else 1 + ACTIVATIONS[unary], M, N, K,
+                                     0 if unary is None else 1 + ACTIVATIONS[unary],
+                                     *_mul_args(mul, M, N, torch.bfloat16), M, N, K,
                                      _p(fault_word(x.device)), _stream()), "fused_linear_x")
 
 
-def fused_gate_up_silu_x(x, w_gu, act, block: int = 0) -> None:
-    """act = silu(x·Wgᵀ) ⊙ (x·Wuᵀ) from bfloat16 rows, one few-token kernel."""
+def fused_gate_up_silu_x(x, w_gu, act, block: int = 0, gate=None) -> None:
+    """act = silu(x·Wgᵀ) ⊙ (x·Wuᵀ) from bfloat16 rows, one few-token kernel (``gate``: as in
+    ``silu_mul``)."""
     _need(x, "x", torch.bfloat16, 2); _need(w_gu, "w_gu", torch.bfloat16, 2)
     _need(act, "act", torch.bfloat16, 2)
     M, K = x.shape
@@ -1551,8 +1704,9 @@ def fused_gate_up_silu_x(x, w_gu, act, block: int = 0) -> None:
     if tuple(w_gu.shape) != (2 * I, K) or act.shape[0] != M or not act.is_contiguous():
         raise KernelError("fused_gate_up_silu_x: shapes do not fit")
     _check(lib().cretif_fused_gate_up_silu_x(_p(x), _rows(x, "x"), _p(w_gu), _rows(w_gu, "w_gu"),
-                                             _p(act), I, block, M, K, _p(fault_word(x.device)),
-                                             _stream()), "fused_gate_up_silu_x")
+                                             _p(act), I, block, *_gate_args(gate), M, K,
+                                             _p(fault_word(x.device)), _stream()),
+           "fused_gate_up_silu_x")
 
 
 def fused_qkv_rope(h, norm_w, eps: float, w_qkv, q_out, cos, sin, pairing: int, nh: int,
@@ -1573,9 +1727,9 @@ def fused_qkv_rope(h, norm_w, eps: float, w_qkv, q_out, cos, sin, pairing: int, 
         int(write_cache), M, K, _p(fault), _stream()), "fused_qkv_rope")
 
 
-def fused_gate_up_silu(h, norm_w, eps: float, w_gu, act, block: int = 0) -> None:
+def fused_gate_up_silu(h, norm_w, eps: float, w_gu, act, block: int = 0, gate=None) -> None:
     """act = silu(norm(h)·Wgᵀ) ⊙ (norm(h)·Wuᵀ), one kernel; w_gu = [Wg; Wu] stacked
-    (``block`` = 0) or with rows interleaved in groups of ``block``."""
+    (``block`` = 0) or with rows interleaved in groups of ``block``; ``gate``: as in ``silu_mul``."""
     _need(h, "h", torch.float32, 2); _need(w_gu, "w_gu", torch.bfloat16, 2)
     _need(act, "act", torch.bfloat16, 2)
     M, K = h.shape
@@ -1583,13 +1737,15 @@ def fused_gate_up_silu(h, norm_w, eps: float, w_gu, act, block: int = 0) -> None
     if tuple(w_gu.shape) != (2 * I, K) or act.shape[0] != M or not act.is_contiguous():
         raise KernelError("fused_gate_up_silu: shapes do not fit")
     _check(lib().cretif_fused_gate_up_silu(_p(h), _p(norm_w), ctypes.c_float(eps), _p(w_gu),
-                                           _rows(w_gu, "w_gu"), _p(act), I, block, M, K,
+                                           _rows(w_gu, "w_gu"), _p(act), I, block,
+                                           *_gate_args(gate), M, K,
                                            _p(fault_word(h.device)), _stream()),
            "fused_gate_up_silu")
 
 
-def gemm_tc_silu(x, w_gu, act) -> None:
-    """act = silu(x·Wgᵀ) ⊙ (x·Wuᵀ) on the tensor cores; w_gu rows interleaved in groups of 64."""
+def gemm_tc_silu(x, w_gu, act, gate=None) -> None:
+    """act = silu(x·Wgᵀ) ⊙ (x·Wuᵀ) on the tensor cores (``gate``: as in ``silu_mul``); w_gu rows
+    interleaved in groups of 64."""
     _need(x, "x", torch.bfloat16, 2); _need(w_gu, "w_gu", torch.bfloat16, 2)
     _need(act, "act", torch.bfloat16, 2)
     M, K = x.shape
@@ -1597,8 +1753,8 @@ def gemm_tc_silu(x, w_gu, act) -> None:
     if tuple(w_gu.shape) != (2 * I, K) or act.shape[0] != M or not act.is_contiguous():
         raise KernelError("gemm_tc_silu: shapes do not fit")
     _check(lib().cretif_gemm_tc_silu(_p(x), _p(w_gu), _p(act), M, I, K, _rows(x, "x"),
-                                     _rows(w_gu, "w_gu"), _p(fault_word(x.device)), _stream()),
-           "gemm_tc_silu")
+                                     _rows(w_gu, "w_gu"), *_gate_args(gate),
+                                     _p(fault_word(x.device)), _stream()), "gemm_tc_silu")
 
 
 def gemm_tc_qkv_rope(x, w_qkv, q_out, cos, sin, pairing: int, nh: int, nkv: int, hd: int,

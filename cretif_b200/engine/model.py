@@ -57,9 +57,16 @@ def _branch_specs(bs: BranchSpec):
         yield "norm", bs.post_norm
 
 
+def _full_name(prefix: str, name: str) -> str:
+    """A tensor's full name: behind the layer's prefix, or without it when the name begins with "/"."""
+    return name[1:] if name.startswith("/") else prefix + name
+
+
 def _part_specs(spec: ModelSpec):
     """Every (category, PartSpec, name prefix) of the model, in a fixed order."""
     yield "embedding", _with(spec.embedding, vocab_size=spec.vocab_size), ""
+    if spec.merge is not None:
+        yield "merge", spec.merge, ""
     for layer in spec.layers:
         for bs in layer.branches:
             for category, pspec in _branch_specs(bs):
@@ -74,7 +81,7 @@ def manifest(spec: ModelSpec) -> Tuple[Dict[str, WeightSpec], Set[str]]:
     for category, pspec, prefix in _part_specs(spec):
         cls = lookup_part(category, pspec.kind)
         for _, (name, wspec) in cls.weight_specs(pspec.params, spec.hidden_size).items():
-            full = prefix + name
+            full = _full_name(prefix, name)
             if full in out and out[full] != wspec:
                 raise ValueError(f"tensor {full!r} is declared twice with different shapes")
             out[full] = wspec
@@ -97,6 +104,7 @@ class Model:
         self._parts: List[Part] = built
         it = iter(built)
         self.embedding = next(it)
+        self.merge = next(it) if spec.merge is not None else None
         self.layers: List[Layer] = []
         for ls in spec.layers:
             branches = []
@@ -112,7 +120,7 @@ class Model:
         self.head = next(it)
 
     def parts(self) -> List[Part]:
-        """Every part of the model: embedding, each layer's branches in order, final norm, head."""
+        """Every part of the model: embedding, merge (if any), each layer's branches in order, final norm, head."""
         return list(self._parts)
 
     @property
@@ -126,7 +134,7 @@ class Model:
         for part, (category, pspec, prefix) in zip(self._parts, _part_specs(self.spec)):
             specs = lookup_part(category, pspec.kind).weight_specs(pspec.params,
                                                                    self.spec.hidden_size)
-            part.load({key: tensors[prefix + name] for key, (name, _) in specs.items()})
+            part.load({key: tensors[_full_name(prefix, name)] for key, (name, _) in specs.items()})
         if self.spec.head.params.get("tied"):
             self.head.tie(self.embedding)
 
@@ -198,6 +206,16 @@ class Model:
                 views.append(view(shift=shift))
         return views
 
+    def _reads_stream(self, i: int) -> bool:
+        """Whether schedule entry ``i`` begins with a branch that reads the stream itself (no norm in
+        front of it), so that a copy in the compute type is worth leaving."""
+        if i >= len(self.spec.schedule):
+            return False
+        entry = self.spec.schedule[i]
+        first = self.layers[entry.layer].branches[0]
+        return first.norm is None and first.shift is None and not (entry.add_input
+                                                                   or entry.merge_input)
+
     # -- one step ------------------------------------------------------------------
     def forward(self, ctx: StepContext, cache, want_rows: Optional[torch.Tensor]) -> torch.Tensor:
         """Run the scheduled layers on the step's tokens; logits [rows, vocab] float32
@@ -207,16 +225,22 @@ class Model:
         # a schedule entry may ask for the model's input to be added again (a further pass
         # over a span of layers): the embedding's output is kept for it
         h_in = h.clone() if any(e.add_input for e in self.spec.schedule) else None
+        merging = any(e.merge_input for e in self.spec.schedule)
+        merge_rows = self.merge.begin(h) if merging else None
         streams = ctx.extras.get("streams")      # a list: the stream after every layer run
         pending = None
         for i, entry in enumerate(self.spec.schedule):
             layer = self.layers[entry.layer]
-            if entry.add_input:
+            if entry.add_input or entry.merge_input:
                 if pending is not None:
                     ops.axpy_rows(h, pending.contiguous(), 1.0)
                     pending = None
                 ctx.extras.pop("stream_copy", None)
-                ops.axpy_rows(h, h_in, 1.0)
+                if entry.add_input:
+                    ops.axpy_rows(h, h_in, 1.0)
+                if entry.merge_input:
+                    self.merge.forward(h, merge_rows)
+            ctx.extras["copy_wanted"] = self._reads_stream(i + 1)
             pending = layer.run(layer, h, pending, ctx, self.layer_caches(i, cache))
             if streams is not None:
                 streams.append(h.clone() if pending is None else h + pending.to(h.dtype))

@@ -26,6 +26,11 @@ size than the keys) and ``own_kv: False`` (no key and value tensors: the layer r
 and values that another schedule entry stores, with queries, bias and everything else of its
 own).  One kernel does convolution, head norm, gain and the cache write.
 
+``conv`` together with ``qk_norm`` is another member of the family below: the convolved projections are
+normed as a whole, rotated and stored by one kernel, and the saved inputs are the same.  ``out_gate``
+names a matrix with a row per channel of the concatenated heads: the heads are multiplied by the
+logistic function of its product with the layer's input, before the output product.
+
 ``chunk`` (an integer) replaces the sliding window by chunks: a query sees the earlier keys of
 its own run of ``chunk`` positions, runs counted from position 0 of the sequence.
 ``distance_slope`` (``{"exponent": x}``) takes ``slope_h * (i - j)`` off the scaled score of key j
@@ -36,7 +41,7 @@ its own (``own_kv: False``).
 ``pool`` (P tokens; with a sliding ``window``) keeps, beside the window, one key and value for every
 block of P tokens: the means of the block's rows as the cache holds them.  A query sees the blocks
 that lie wholly before its window, in the same softmax as the window's tokens; tokens that have left
-the window and whose block has not left it yet are not seen.  ``qk_norm`` together with biases, a
+the window and whose block has not left it yet are not seen.  ``qk_norm`` together with biases, a convolution, a
 position encoding, values of another size or ``pool`` is one kernel between the input product and
 the attention as well, and there ``out_scale`` (a factor on the layer's output) is applied to the
 values as they are stored.
@@ -228,6 +233,7 @@ class Attention(Part):
         self.bias = self.bias_edges = self.bias_dense = None
         self.bias_names = params.get("bias")
         self.head_gate = params.get("head_gate")
+        self.out_gate = params.get("out_gate")
         # the family that norms head by head without a convolution
         self.slope_spec = params.get("distance_slope")
         self.slope = self.slope_log2e = None
@@ -240,8 +246,8 @@ class Attention(Part):
                                                 and self.distance_bias is None)):
             raise ValueError("attention: pooled blocks need a sliding window, keys of the layer's own "
                              "and no convolution, bias or slope by distance")
-        self.headwise = self.conv is None and bool(
-            self.bias_names or self.head_gate or self.head_norm or self.vd != self.hd
+        self.headwise = self.qk_norm is not None if self.conv is not None else bool(
+            self.out_gate or self.bias_names or self.head_gate or self.head_norm or self.vd != self.hd
             or self.chunk or self.slope_spec or not self.own_kv or self.pool
             or self.out_scale != 1.0 or (self.qk_norm is not None and has_position))
         # norms over the whole projections in the kernel that stores keys and values
@@ -258,6 +264,13 @@ class Attention(Part):
                              "(give `conv`)")
         if self.conv is not None and (self.bias_names or self.head_gate):
             raise ValueError("attention: bias and head_gate are built without a convolution")
+        if self.out_gate and (self.head_gate or not self.headwise):
+            raise ValueError("attention: out_gate comes without head_gate, and with a convolution only "
+                             "where qk_norm norms it")
+        if self.conv is not None and self.headwise and (
+                not self.own_kv or self.query_gain or self.distance_bias or self.chunk or self.slope_spec):
+            raise ValueError("attention: convolved projections normed as a whole are built with keys of "
+                             "the layer's own and without gain, bias, slope or chunks")
         if self.headwise:
             if self.values_are_keys or (self.qk_norm is not None
                                         and (self.head_norm is not None or not self.own_kv)):
@@ -271,10 +284,10 @@ class Attention(Part):
             if not 1 <= self.vd <= 512:
                 raise ValueError("attention: value_dim must be in [1, 512]")
         if self.conv is not None:
-            if self.head_norm is None or self.qk_norm is not None or self.values_are_keys \
-                    or (params.get("position") or {}).get("kind", "none") != "none":
-                raise ValueError("attention: convolved projections are built with head_norm, "
-                                 "without qk_norm, position encoding or keys as values")
+            if not self.headwise and (self.head_norm is None or self.values_are_keys
+                                      or has_position):
+                raise ValueError("attention: convolved projections are built with head_norm (without "
+                                 "position encoding or keys as values) or with qk_norm")
             if int(self.conv["taps"]) < 1 or not 1 <= self.vd <= 512:
                 raise ValueError("attention: conv.taps must be >= 1 and value_dim in [1, 512]")
             self.taps = int(self.conv["taps"])
@@ -322,6 +335,8 @@ class Attention(Part):
         if hn and not conv and hn.get("q"):
             out["q_head_norm"] = (hn["q"], WeightSpec((params["head_dim"],), init=(1.0, 0.1)))
             out["k_head_norm"] = (hn["k"], WeightSpec((params["head_dim"],), init=(1.0, 0.1)))
+        if params.get("out_gate"):
+            out["out_gate"] = (params["out_gate"], WeightSpec((o_in, hidden_size)))
         if params.get("head_gate"):
             out["head_gate"] = (params["head_gate"],
                                 WeightSpec((params["num_heads"], hidden_size)))
@@ -331,8 +346,8 @@ class Attention(Part):
         # one product for q, k and v: rows [q | k | v] of the stacked matrix
         stacked = [tensors["q"]] + ([tensors["k"]] if self.own_kv else []) \
             + ([tensors["v"]] if self.own_kv and not self.values_are_keys else [])
-        if self.head_gate:
-            stacked.append(tensors["head_gate"])              # rows [q | k | v | gates | zeros]
+        if self.head_gate or self.out_gate:                   # rows [q | k | v | gates | zeros]
+            stacked.append(tensors["head_gate" if self.head_gate else "out_gate"])
             self.w_qkv = self._stacked(stacked)
         elif self.headwise:
             self.w_qkv = self._stacked(stacked)               # rows [q | k | v | zeros]
@@ -349,7 +364,8 @@ class Attention(Part):
         if self.conv is not None:
             taps = [tensors["q_conv"]] + ([tensors["k_conv"], tensors["v_conv"]]
                                           if self.own_kv else [])
-            self.conv_w = self._vector32(torch.cat(taps, dim=0))
+            taps = torch.cat(taps, dim=0)                      # [C, taps]; headwise: [taps, C]
+            self.conv_w = self._vector32(taps.t() if self.headwise else taps)
         if self.distance_bias is not None:
             self.bias = self._vector32(tensors["rel"])
             edges = distance_edges(self.bias.shape[0], float(self.distance_bias["far"]))
@@ -393,7 +409,10 @@ class Attention(Part):
         if self.conv is None or self.taps == 1:
             return kv
         # the last taps - 1 projected rows of every convolved channel
-        state = StateRequest((self.conv_channels * (self.taps - 1),), torch.float32)
+        floats = self.conv_channels * (self.taps - 1)
+        if self.headwise:                     # every slot's inputs start at a 16-byte boundary
+            floats = -(-floats // 4) * 4
+        state = StateRequest((floats,), torch.float32)
         return state if kv is None else (kv, state)
 
     def _forward_convolved(self, x, ctx, cache, into=None):
@@ -446,8 +465,9 @@ class Attention(Part):
         return self.headwise
 
     def mix(self, proj, ctx, cache, out) -> None:
-        """From the input product's rows (32-bit sums) to the output product's: bias, norms, rotation
-        and the cache write in one kernel, pooled entries, attention, the per-head gate."""
+        """From the input product's rows (32-bit sums) to the output product's: bias or convolution,
+        norms, rotation and the cache write in one kernel, pooled entries or saved inputs, attention,
+        the gate."""
         kv = cache.kv
         rot = getattr(self.position, "rotary_table", None)
         if rot is not None:
@@ -471,7 +491,12 @@ class Attention(Part):
             ops.projnorm_rope_kv_append(
                 proj, self.in_bias, self.q_norm_w, self.k_norm_w, self.qk_eps, cos, sin, pairing,
                 rot_dim, ctx.tok_pos, ctx.tok_seq, ctx.seq_slot, self.nh, self.nkv, self.hd, self.vd,
-                q, v_scale=self.out_scale, pool=pool if ctx.is_decode else None, **common)
+                q, v_scale=self.out_scale, pool=pool if ctx.is_decode else None,
+                conv=None if self.conv is None else (self.conv_w, cache.state, ctx.seq_start,
+                                                     ctx.is_decode), **common)
+            if self.conv is not None and self.taps > 1 and not ctx.is_decode:
+                ops.delta_conv_state(proj, cache.state, self.taps, self.conv_channels,
+                                     ctx.cu_seqlens, ctx.seq_slot, ctx.B)
         else:
             ops.headnorm_rope_kv_append(
                 proj, self.in_bias, self.q_head_w, self.k_head_w,
@@ -482,9 +507,9 @@ class Attention(Part):
             ops.pool_kv(kv.k, kv.v, kv.table, pool, ctx.cu_seqlens, ctx.seq_start, ctx.seq_slot,
                         self.nkv, self.hd, self.vd, kv.block_tokens, ctx.B, ctx.max_new, ctx.fault)
         self.attend(q, out, ctx, kv)
-        if self.head_gate:
-            ops.gate_heads(out, proj[:, self.q_dim + (self.kv_dim + self.v_dim if own else 0):],
-                           self.nh, self.vd)
+        if self.head_gate or self.out_gate:           # a number per head, or per channel
+            gates = proj[:, self.q_dim + (self.kv_dim + self.v_dim if own else 0):]
+            ops.gate_heads(out, gates, *((self.nh, self.vd) if self.head_gate else (self.o_dim, 1)))
 
     def _forward_headwise(self, x, ctx, cache, into=None, alpha: float = 1.0, proj=None):
         """One product for q|k|v|gates with 32-bit sums (``proj``, where the caller made it
@@ -569,7 +594,7 @@ class Attention(Part):
         kernel and the tensor-core products.  Projections normed head by head: few tokens take
         the input product that norms the rows in its prologue, and ``alpha`` times the output
         product is added into ``h``.  False if the step does not qualify."""
-        if norm is not None and self.headwise and self.conv is None:
+        if norm is not None and self.headwise:
             from .linear import normed_linear_few
             proj = normed_linear_few(h, norm, self.w_qkv, torch.float32)
             if proj is None:

@@ -1,7 +1,7 @@
 """Interfaces of the parts a model is assembled from, and their registries.
 
 A part is a small class that owns its constants (given as ``params``) and its
-weights, and knows nothing about the model it sits in.  There are six kinds:
+weights, and knows nothing about the model it sits in.  There are these kinds:
 
 ===============  =============================================================
 kind             interface
@@ -16,11 +16,14 @@ position         used by a mixer; ``rotate_and_store(qkv, ctx, kv_view, ...)``
 head             ``forward(n[R, H], ctx) -> logits[R, V] float32``
 shift            ``forward(h[T, H] float32, norm, ctx, state) -> x[T, H]``: the normed rows,
                  each blended with the row of the token before it
+merge            ``begin(h) -> rows`` once a step, ``forward(h, rows)`` in front of every pass over a
+                 span of layers: the model's input enters the stream ``h`` again, in place
 
 ===============  =============================================================
 
 Every part class also has ``weight_specs(params, hidden_size)``: a dict from a
-short key to ``(tensor name relative to the part's prefix, WeightSpec)``, which is
+short key to ``(tensor name relative to the part's prefix, WeightSpec)`` (a name that begins with
+"/" is the model's own, without the prefix: a tensor that layers share), which is
 how the loader learns the names and shapes a checkpoint must have, and
 ``load(tensors)`` which receives the CPU tensors under the same short keys.
 
@@ -38,7 +41,7 @@ from ..config.spec import PartSpec
 from ..weights.loader import WeightSpec
 
 _KINDS = ("embedding", "norm", "mixer", "feed_forward", "position", "head", "arrangement",
-          "shift")
+          "shift", "merge")
 _REGISTRY: Dict[str, Dict[str, Any]] = {k: {} for k in _KINDS}
 
 

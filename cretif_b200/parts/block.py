@@ -20,6 +20,12 @@ the residual stream itself, applies the given norm inside its first kernel and a
 output into ``h`` inside its last one (the fused few-token kernels do this).  It returns
 False when it cannot take the step, and the arrangement falls back to the separate norm
 and the returned branch.  Parts without the method just use that path.
+
+A part with ``adds_scaled`` also takes ``into=h`` in its ``forward`` and adds its output there, and
+one with ``adds_into_stream`` takes ``into=h, emit=...``: it adds into ``h`` and hands back the new rows
+in the compute type, which a branch without a norm behind it reads.  Copies of the stream in the
+compute type are made only where somebody reads them: the next branch, or, behind the last branch,
+whoever set ``ctx.extras["copy_wanted"]`` (absent: a copy is left).
 """
 from __future__ import annotations
 
@@ -50,7 +56,13 @@ def run_residual(layer, h, pending, ctx, caches):
     # a copy of the stream in the compute type, left by the kernel that last added to it
     extras = getattr(ctx, "extras", None)
     lowp = extras.pop("stream_copy", None) if extras is not None else None
-    for branch, cache in zip(layer.branches, caches):
+    for k, (branch, cache) in enumerate(zip(layer.branches, caches)):
+        # whether what follows reads the stream itself
+        follows = layer.branches[k + 1] if k + 1 < len(layer.branches) else None
+        if follows is not None:
+            emit = follows.norm is None and getattr(follows, "shift", None) is None
+        else:
+            emit = extras.get("copy_wanted", True) if extras is not None else True
         part = branch.part
         scale = float(getattr(branch, "scale", 1.0))
         if scale != 1.0 and branch.post_norm is None:
@@ -110,6 +122,18 @@ def run_residual(layer, h, pending, ctx, caches):
                 pending, lowp = None, None
             # the part reads the stream itself
             x = lowp if lowp is not None and lowp.dtype == part.dtype else stream_as(h, part.dtype)
+        # (a part that reads the stream itself may not write into what it reads)
+        adds = branch.post_norm is None and branch.norm is not None
+        if adds and follows is not None and emit and getattr(part, "adds_into_stream", False):
+            lowp = part.forward(x, ctx, into=h, emit=True)
+            continue
+        if adds and getattr(part, "adds_scaled", False):
+            if branch.role == "mixer":
+                part.forward(x, ctx, cache, into=h)
+            else:
+                part.forward(x, ctx, into=h)
+            lowp = None
+            continue
         y = call_part(branch, x, ctx, cache)
         if branch.post_norm is not None:
             if scale != 1.0:
@@ -118,7 +142,7 @@ def run_residual(layer, h, pending, ctx, caches):
                 continue
             if hasattr(branch.post_norm, "add_into"):
                 # h += norm(y), 32-bit, one kernel, which also leaves the next reader's copy
-                lowp = branch.post_norm.add_into(h, y, emit=True)
+                lowp = branch.post_norm.add_into(h, y, emit=emit)
                 continue
             y = branch.post_norm.forward(y.to(h.dtype).contiguous())
         pending = y

@@ -14,7 +14,7 @@ import torch
 from ..csrc import ops
 from ..weights.loader import WeightSpec
 from .base import Part, register_part
-from .linear import linear
+from .linear import linear, norm_prologue
 
 
 @register_part("embedding", "token_embedding")
@@ -110,14 +110,16 @@ class LinearHead(Part):
         step does not qualify."""
         from .attention import FUSED_MAX_TOKENS, fused_steps_enabled
         R = h.shape[0] if rows is None else rows.numel()
-        rms = getattr(norm, "rms_params", None)
+        params = norm_prologue(norm)
         if (pending is not None or not fused_steps_enabled() or self.dtype != torch.bfloat16
-                or R > FUSED_MAX_TOKENS or rms is None
-                or not ops.fused_supported(R, self.hidden_size, self.weight)):
+                or R > FUSED_MAX_TOKENS or params is None
+                or not ops.fused_supported(R, self.hidden_size, self.weight,
+                                           norm=1 if params[1] is None else 2)):
             return None
         logits = torch.empty((R, self.weight.shape[0]), dtype=torch.float32, device=h.device)
-        norm_w, eps = rms()
-        ops.fused_norm_linear(h, norm_w, eps, self.weight, logits, rows=rows, alpha=self.scale)
+        norm_w, norm_b, eps = params
+        ops.fused_norm_linear(h, norm_w, eps, self.weight, logits, rows=rows, alpha=self.scale,
+                              norm_b=norm_b)
         return self._capped(logits, scaled=True)
 
     def weight_bytes(self):

@@ -12,11 +12,13 @@ kernels' unary activations; ``groups`` (``{"count", "keep"}``) lets the experts 
 equal groups of neighbours, scores a group by the sum of its two largest scores and allows only
 experts of the ``keep`` best groups; ``sum_eps`` is added to the sum that ``renormalize`` divides
 by; ``scores: "softmax"`` takes the softmax over all router outputs instead of the logistic
-function; ``correction`` names a tensor with a number per router output that is added to the scores
+function, ``"softmax_chosen"`` over the chosen ones alone; ``router_bias`` names a tensor with a number
+per router output that is added to the logits; ``clamp`` (``{"limit", "slope", "offset"}``) clamps the
+gates of gated experts (parts/mlp.py); ``correction`` names a tensor with a number per router output that is added to the scores
 for the choice alone; a group's score is then that of its choice scores, and ``groups`` may say
 ``"score": "best"`` for the largest instead of the sum of two; ``identities`` appends that many router
 outputs that are no experts: their output is the input itself; ``shared``
-(``{"intermediate_size", "names"}``) is one more expert of the same form that every token uses with
+(``{"intermediate_size", "names"[, "clamp"]}``) is one more expert of the same form that every token uses with
 weight one.
 
 The step's (token, choice) pairs are sorted by expert on the device and each expert's rows
@@ -34,6 +36,7 @@ from ..csrc import ops
 from ..weights.loader import WeightSpec
 from ..config.spec import PartSpec
 from .base import Part, build_part, register_part
+from .mlp import gate_rule
 from .side_stream import Fork, forks
 
 
@@ -61,23 +64,28 @@ class RoutedExperts(Part):
     ("input" | "output"), ``renormalize`` (default False), ``names``: ``router`` and the
     patterns ``gate``, ``up``, ``down`` with ``{e}`` for the expert's number.  Optional:
     ``gated`` (default True), ``activation``, ``groups``, ``sum_eps``, ``scores`` ("sigmoid" |
-    "softmax"), ``correction``, ``identities``, ``shared``."""
+    "softmax" | "softmax_chosen"), ``router_bias``, ``clamp``, ``correction``, ``identities``,
+    ``shared``."""
 
     graph_safe = True
+    # forward takes ``into`` (the stream) and ``emit``: see parts/block.py
+    adds_into_stream = True
 
     def __init__(self, params, hidden_size, dtype, device):
         super().__init__(params, hidden_size, dtype, device)
         self.E = int(params["num_experts"])
         self.identities = int(params.get("identities") or 0)
         self.outputs = self.E + self.identities              # of the router
-        self.softmax = params.get("scores", "sigmoid") == "softmax"
-        if params.get("scores", "sigmoid") not in ("sigmoid", "softmax") or self.identities < 0:
-            raise ValueError("routed_experts: scores must be 'sigmoid' or 'softmax' and identities "
-                             "not below zero")
+        scores = params.get("scores", "sigmoid")
+        if scores not in ("sigmoid", "softmax", "softmax_chosen") or self.identities < 0:
+            raise ValueError("routed_experts: scores must be 'sigmoid', 'softmax' or 'softmax_chosen' "
+                             "and identities not below zero")
+        self.softmax = {"sigmoid": False, "softmax": True, "softmax_chosen": "chosen"}[scores]
         self.top = int(params["top"])
         self.inter = int(params["intermediate_size"])
         self.weight_on = params.get("weight_on", "output")
-        self.renorm = bool(params.get("renormalize", False))
+        self.renorm = bool(params.get("renormalize", False)) or self.softmax == "chosen"
+        self.gate = gate_rule(params.get("clamp"))
         if self.weight_on not in ("input", "output"):
             raise ValueError(f"routed_experts: weight_on must be 'input' or 'output', got "
                              f"{self.weight_on!r}")
@@ -87,6 +95,11 @@ class RoutedExperts(Part):
         if self.identities and self.weight_on == "input":
             raise ValueError("routed_experts: identities are built with the weight on the output")
         self.gated = bool(params.get("gated", True))
+        if self.gate is not None and not self.gated:
+            raise ValueError("routed_experts: experts without a gate have none to clamp")
+        if self.softmax == "chosen" and (params.get("correction") or params.get("groups")):
+            raise ValueError("routed_experts: the softmax over the chosen experts alone is built without "
+                             "correction and groups")
         self.activation = params.get("activation", "silu")
         if self.gated and self.activation != "silu":
             raise ValueError("routed_experts: gated experts have a kernel for 'silu' only")
@@ -108,15 +121,18 @@ class RoutedExperts(Part):
         sh = params.get("shared")
         if sh:
             kind = "gated_mlp" if self.gated else "dense_mlp"
+            extra = {"clamp": sh["clamp"]} if sh.get("clamp") else {}
             self.shared = build_part("feed_forward", PartSpec(kind, {
                 "intermediate_size": int(sh["intermediate_size"]), "activation": self.activation,
-                "names": sh["names"]}), hidden_size, dtype, device)
+                "names": sh["names"], **extra}), hidden_size, dtype, device)
 
     @classmethod
     def weight_specs(cls, params, hidden_size):
         E, F, n = params["num_experts"], params["intermediate_size"], params["names"]
         outputs = E + int(params.get("identities") or 0)
         out = {"router": (n["router"], WeightSpec((outputs, hidden_size), init=(0.0, 0.5)))}
+        if params.get("router_bias"):
+            out["router_bias"] = (params["router_bias"], WeightSpec((outputs,), init=(0.0, 0.5)))
         if params.get("correction"):
             out["correction"] = (params["correction"], WeightSpec((outputs,), init=(0.0, 0.05)))
         for e in range(E):
@@ -143,6 +159,8 @@ class RoutedExperts(Part):
             self.router_matrix = None
         self.correction = (self._vector32(tensors["correction"]) if "correction" in tensors
                            else None)
+        self.router_bias = (self._vector32(tensors["router_bias"]) if "router_bias" in tensors
+                            else None)
         if self.shared is not None:
             self.shared.load({k[len("shared_"):]: v for k, v in tensors.items()
                               if k.startswith("shared_")})
@@ -163,10 +181,12 @@ class RoutedExperts(Part):
                  tensors[f"up{e}"].reshape(F // 64, 64, -1)], dim=1).reshape(2 * F, -1)
                 for e in range(E)]))
 
-    def forward(self, x, ctx):
+    def forward(self, x, ctx, into=None, emit: bool = False):
+        """``into``: a float32 matrix that the output is added to (the residual stream) instead of
+        being returned; with ``emit`` (and a compute type other than float32) its new rows are returned
+        in the compute type, for the sublayer that reads the stream next."""
         T, H = x.shape
         dev = x.device
-        P = T * self.top
         # the shared expert: in a step of few tokens beside the routed ones, its output then joins
         # where the choices are summed; otherwise added to their sum
         fork = beside = None
@@ -183,28 +203,38 @@ class RoutedExperts(Part):
             ops.moe_topk(logits, self.top, ids, wts, **self._rule())
         else:
             ops.moe_route(x, self.router, self.top, ids, wts, **self._rule())
+        if into is not None:
+            # (the combination comes last, so that it leaves the finished rows)
+            if self.shared is not None and beside is None:
+                self.shared.forward(x, ctx, into=into)
+            x_out = (torch.empty((T, H), dtype=self.dtype, device=dev)
+                     if emit and self.dtype == torch.bfloat16 else None)
+            self._experts(x, ids, wts, into, fork, beside, add=True, x_out=x_out)
+            return x_out
         y = torch.empty((T, H), dtype=torch.float32, device=dev)
-        if self.gated:
-            self._gated_experts(x, ids, wts, y, fork, beside)
-        else:
-            self._plain_experts(x, ids, wts, y, fork, beside)
+        self._experts(x, ids, wts, y, fork, beside)
         if self.shared is not None and beside is None:
             self.shared.forward(x, ctx, into=y)
         return y
 
+    def _experts(self, x, ids, wts, y, fork, beside, **how):
+        (self._gated_experts if self.gated else self._plain_experts)(x, ids, wts, y, fork, beside, how)
+
     def _rule(self) -> dict:
         return dict(renorm=self.renorm, groups=self.groups, keep=self.keep, sum_eps=self.sum_eps,
-                    softmax=self.softmax, group_best=self.group_best, correction=self.correction)
+                    softmax=self.softmax, group_best=self.group_best, correction=self.correction,
+                    bias=self.router_bias)
 
-    def _combine(self, rows, place, y, x, ids, wts, scaled: bool, fork, beside):
+    def _combine(self, rows, place, y, x, ids, wts, scaled: bool, fork, beside, how):
         """The choices (and what ran beside them) summed; ``scaled``: the rows carry their weights
         already."""
         if fork is not None:
             fork.join()
         ops.moe_combine(rows, place, self.top, y, wts=None if scaled else wts,
-                        identity=(ids, self.E, wts, x) if self.identities else None, plus=beside)
+                        identity=(ids, self.E, wts, x) if self.identities else None, plus=beside,
+                        **how)
 
-    def _plain_experts(self, x, ids, wts, y, fork, beside):
+    def _plain_experts(self, x, ids, wts, y, fork, beside, how):
         """Experts without a gate: the activation sits in the first product's epilogue."""
         T, H = x.shape
         dev, P = x.device, T * self.top
@@ -215,7 +245,7 @@ class RoutedExperts(Part):
             rows = torch.empty((P, H), dtype=torch.float32, device=dev)
             ops.moe_gemv(x, self.w_up, act, self.top, mode, 1 if on_input else 0, ids, wts)
             ops.moe_gemv(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, ids, wts)
-            self._combine(rows, None, y, x, ids, wts, True, fork, beside)
+            self._combine(rows, None, y, x, ids, wts, True, fork, beside, how)
             return
         if self.dtype == torch.bfloat16 and ops.moe_tc_supported(x, self.w_up, self.w_down,
                                                                  gated=False):
@@ -230,7 +260,7 @@ class RoutedExperts(Part):
             ops.gemm_tc_act_grouped(xs, self.w_up, act, tile_expert, used, self.activation)
             rows = torch.empty((rows_pad, H), dtype=torch.float32, device=dev)
             ops.gemm_tc_grouped(act, self.w_down, rows, tile_expert, used)
-            self._combine(rows, place, y, x, ids, wts, on_input, fork, beside)
+            self._combine(rows, place, y, x, ids, wts, on_input, fork, beside, how)
             return
         tiles = ops.moe_max_tiles(P, self.E)
         idx = torch.empty(self.E + 1 + 2 * P + 2 * tiles, dtype=torch.int32, device=dev)
@@ -245,9 +275,9 @@ class RoutedExperts(Part):
                      tile_expert, tile_row0)
         ops.moe_gemm(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, wts, order,
                      offsets, tile_expert, tile_row0)
-        self._combine(rows, place, y, x, ids, wts, True, fork, beside)
+        self._combine(rows, place, y, x, ids, wts, True, fork, beside, how)
 
-    def _gated_experts(self, x, ids, wts, y, fork, beside):
+    def _gated_experts(self, x, ids, wts, y, fork, beside, how):
         T, H = x.shape
         dev, P = x.device, T * self.top
         on_input = self.weight_on == "input"
@@ -255,9 +285,10 @@ class RoutedExperts(Part):
             # a handful of pairs: every pair streams its expert's rows, nothing is sorted
             act = torch.empty((P, self.inter), dtype=self.dtype, device=dev)
             rows = torch.empty((P, H), dtype=torch.float32, device=dev)
-            ops.moe_gemv(x, self.w_gu, act, self.top, 0, 1 if on_input else 0, ids, wts)
+            ops.moe_gemv(x, self.w_gu, act, self.top, 0, 1 if on_input else 0, ids, wts,
+                         gate=self.gate)
             ops.moe_gemv(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, ids, wts)
-            self._combine(rows, None, y, x, ids, wts, True, fork, beside)
+            self._combine(rows, None, y, x, ids, wts, True, fork, beside, how)
             return
         if self.w_gu_blocks is not None and ops.moe_tc_supported(x, self.w_gu_blocks, self.w_down):
             # many pairs, bfloat16: the tcgen05 product in its grouped mode over rows sorted
@@ -270,10 +301,10 @@ class RoutedExperts(Part):
             xs = torch.empty((rows_pad, H), dtype=self.dtype, device=dev)
             ops.moe_gather_rows(x, xs, place, wts if on_input else None, self.top)
             act = torch.empty((rows_pad, self.inter), dtype=self.dtype, device=dev)
-            ops.gemm_tc_silu_grouped(xs, self.w_gu_blocks, act, tile_expert, used)
+            ops.gemm_tc_silu_grouped(xs, self.w_gu_blocks, act, tile_expert, used, gate=self.gate)
             rows = torch.empty((rows_pad, H), dtype=torch.float32, device=dev)
             ops.gemm_tc_grouped(act, self.w_down, rows, tile_expert, used)
-            self._combine(rows, place, y, x, ids, wts, on_input, fork, beside)
+            self._combine(rows, place, y, x, ids, wts, on_input, fork, beside, how)
             return
         tiles = ops.moe_max_tiles(P, self.E)
         idx = torch.empty(self.E + 1 + 2 * P + 2 * tiles, dtype=torch.int32, device=dev)
@@ -285,10 +316,10 @@ class RoutedExperts(Part):
         act = torch.empty((P, self.inter), dtype=self.dtype, device=dev)
         rows = torch.empty((P, H), dtype=torch.float32, device=dev)
         ops.moe_gemm(x, self.w_gu, act, self.top, 0, 1 if on_input else 0, wts, order, offsets,
-                     tile_expert, tile_row0)
+                     tile_expert, tile_row0, gate=self.gate)
         ops.moe_gemm(act, self.w_down, rows, self.top, 1, 0 if on_input else 2, wts, order,
                      offsets, tile_expert, tile_row0)
-        self._combine(rows, place, y, x, ids, wts, True, fork, beside)
+        self._combine(rows, place, y, x, ids, wts, True, fork, beside, how)
 
     def weight_bytes(self):
         # (the blocked copy of gate|up serves the many-pairs path and is not counted twice)

@@ -86,21 +86,33 @@ def linear_few(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype
     return linear(x, w, out_dtype=out_dtype, out=out, accumulate=accumulate)
 
 
+def norm_prologue(norm):
+    """(weight, bias or None, eps) of a norm that a product may apply in its prologue, or None."""
+    params = getattr(norm, "prologue_params", None)
+    if params is not None:
+        return params()
+    rms = getattr(norm, "rms_params", None)
+    if rms is None:
+        return None
+    weight, eps = rms()
+    return weight, None, eps
+
+
 def normed_linear_few(h: torch.Tensor, norm, w: torch.Tensor, out_dtype,
                       unary: Optional[str] = None) -> Optional[torch.Tensor]:
-    """``[act](rmsnorm(h) · Wᵀ)`` by the few-token kernel that norms the residual rows in its
+    """``[act](norm(h) · Wᵀ)`` (an RMS or a layer norm) by the few-token kernel that norms the residual rows in its
     own prologue (and rounds them to bfloat16 as the norm's kernel would), or None where the
     step, the norm or the sizes do not allow it."""
     from .attention import fused_steps_enabled
-    rms = getattr(norm, "rms_params", None)
     M, K = h.shape
-    if (rms is None or not 0 < M <= FEW_ROWS or w.dtype != torch.bfloat16 or _force_plain
+    params = norm_prologue(norm)
+    if (params is None or not 0 < M <= FEW_ROWS or w.dtype != torch.bfloat16 or _force_plain
             or not fused_steps_enabled() or h.dtype != torch.float32 or not h.is_contiguous()
-            or not ops.fused_supported(M, K, w)):
+            or not ops.fused_supported(M, K, w, norm=1 if params[1] is None else 2)):
         return None
-    norm_w, eps = rms()
+    norm_w, norm_b, eps = params
     out = torch.empty((M, w.shape[0]), dtype=out_dtype, device=h.device)
-    ops.fused_norm_linear(h, norm_w, eps, w, out, unary=unary)
+    ops.fused_norm_linear(h, norm_w, eps, w, out, unary=unary, norm_b=norm_b)
     return out
 
 
@@ -124,19 +136,22 @@ def linear_scaled_add(x: torch.Tensor, w: torch.Tensor, h: torch.Tensor, alpha: 
     ops.axpy_rows(h, y, float(alpha))
 
 
-def linear_activation(x: torch.Tensor, w: torch.Tensor, kind: str, dtype) -> torch.Tensor:
+def linear_activation(x: torch.Tensor, w: torch.Tensor, kind: str, dtype, mul=None) -> torch.Tensor:
     """``act(x · Wᵀ)`` in ``dtype``, the activation on the product's 32-bit sums: in the
     epilogue of the tensor-core product or of the few-token kernels where they take the step,
-    else as a kernel of its own over a 32-bit result."""
+    else as a kernel of its own over a 32-bit result.  ``mul`` (``(table, ids)``): times row ids[m]
+    of the table, there as well."""
     M = x.shape[0]
     act = torch.empty((M, w.shape[0]), dtype=dtype, device=x.device)
     if (M > FEW_ROWS and x.dtype == torch.bfloat16 and not _force_plain
-            and ops.gemm_tc_supported(x, w, act)):
-        ops.gemm_tc(x, w, act, unary=kind)
+            and ops.gemm_tc_supported(x, w, act)
+            and (mul is None or (w.shape[0] % 8 == 0 and mul[0].stride(0) % 8 == 0
+                                 and mul[0].data_ptr() % 16 == 0))):
+        ops.gemm_tc(x, w, act, unary=kind, mul=mul)
         return act
     if act.dtype == torch.bfloat16 and _few_rows(x, w):
-        ops.fused_linear_x(x, w, act, unary=kind)
+        ops.fused_linear_x(x, w, act, unary=kind, mul=mul)
         return act
     up = linear_few(x, w, out_dtype=torch.float32)
-    ops.activation(up, act, kind)
+    ops.activation(up, act, kind, mul=mul)
     return act

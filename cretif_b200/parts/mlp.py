@@ -14,15 +14,28 @@ from .base import Part, register_part
 from .linear import linear, linear_scaled_add, plain_forced, skinny_max_rows as SKINNY_ROWS
 
 
+def gate_rule(clamp):
+    """``clamp`` (``{"limit", "slope", "offset"}``, or None) as the kernels take it: with g at most
+    ``limit`` and u within ±``limit``, g · sigmoid(slope · g) · (u + offset) instead of silu(g) · u."""
+    if not clamp:
+        return None
+    rule = (float(clamp["limit"]), float(clamp.get("slope", 1.0)), float(clamp.get("offset", 0.0)))
+    if not rule[0] > 0:
+        raise ValueError(f"a clamped gate needs a limit above zero, got {clamp!r}")
+    return rule
+
+
 @register_part("feed_forward", "gated_mlp")
 class GatedMLP(Part):
-    """params: ``intermediate_size``, ``activation`` ("silu"), ``names`` (gate, up, down)."""
+    """params: ``intermediate_size``, ``activation`` ("silu"), ``clamp`` (optional: a clamped gate,
+    see :func:`gate_rule`), ``names`` (gate, up, down)."""
 
     graph_safe = True
 
     def __init__(self, params, hidden_size, dtype, device):
         super().__init__(params, hidden_size, dtype, device)
         self.inter = int(params["intermediate_size"])
+        self.gate = gate_rule(params.get("clamp"))
         if params.get("activation", "silu") != "silu":
             raise ValueError(f"gated_mlp: activation {params['activation']!r} has no kernel "
                              "(only 'silu')")
@@ -62,16 +75,16 @@ class GatedMLP(Part):
                 and ops.fused_supported(T, self.hidden_size, self.w_gate_up, norm=False)
                 and ops.fused_supported(T, self.inter, self.w_down, norm=False)):
             # few tokens that are already in bfloat16 (no norm in front of this part)
-            ops.fused_gate_up_silu_x(x, self.w_gate_up, act, self.gu_block)
+            ops.fused_gate_up_silu_x(x, self.w_gate_up, act, self.gu_block, gate=self.gate)
             y = linear_few(act, self.w_down, out_dtype=torch.float32, out=into,
                            accumulate=into is not None)
             return None if into is not None else y
         if (self.gu_block == 64 and T > SKINNY_ROWS() and not plain_forced()
                 and ops.gemm_tc_supported(x, self.w_gate_up, act)):
-            ops.gemm_tc_silu(x, self.w_gate_up, act)                  # product + SiLU·mul
+            ops.gemm_tc_silu(x, self.w_gate_up, act, gate=self.gate)  # product + SiLU·mul
         else:
             gu = linear(x, self.w_gate_up)                            # [T, 2 I]
-            ops.silu_mul(gu, act, self.gu_block)
+            ops.silu_mul(gu, act, self.gu_block, gate=self.gate)
         if into is not None:
             linear(act, self.w_down, out=into, accumulate=True)
             return None
@@ -96,7 +109,7 @@ class GatedMLP(Part):
             return False
         act = torch.empty((T, self.inter), dtype=self.dtype, device=h.device)
         norm_w, eps = rms()
-        ops.fused_gate_up_silu(h, norm_w, eps, self.w_gate_up, act, self.gu_block)
+        ops.fused_gate_up_silu(h, norm_w, eps, self.w_gate_up, act, self.gu_block, gate=self.gate)
         ops.fused_linear_add(act, self.w_down, h)
         return True
 

@@ -1,4 +1,4 @@
-"""RMSNorm, fused with the residual addition that precedes it.
+"""RMSNorm and layer norm, fused with the residual addition that precedes it.
 
 ``forward(h, delta)`` performs ``h ← h + delta`` in place on the 32-bit residual
 stream and returns ``norm(h)`` in the compute dtype, which is the reference's fused
@@ -6,6 +6,9 @@ kernel (src/kernels/elementwise.cu:463-506; the plain norm is :30-72).  The weig
 multiplies directly unless ``offset`` is given: a checkpoint that stores its norm weights
 around zero is read with ``offset = 1`` (the factor is ``offset + w``, added once at loading in
 32-bit).  All arithmetic is 32-bit.
+
+A norm may offer ``rms_params() -> (weight, eps)``, or in general ``prologue_params() -> (weight,
+bias or None, eps)``, so that a product applies it in its own prologue.
 
 ``add_into(h, y)`` is the norm on a sublayer's OUTPUT: ``h += norm(y)`` in one kernel, the
 normed rows never leaving 32-bit.
@@ -67,6 +70,39 @@ class RMSNorm(Part):
 
     def weight_bytes(self):
         return self.weight.numel() * 4
+
+
+@register_part("norm", "layernorm")
+class LayerNorm(Part):
+    """``(x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b``.  params: ``eps``, ``name`` (the weight;
+    the bias is stored beside it as ``<name>.b``)."""
+
+    graph_safe = True
+
+    @classmethod
+    def weight_specs(cls, params, hidden_size):
+        n = params["name"]
+        return {"weight": (n, WeightSpec((hidden_size,), init=(1.0, 0.02))),
+                "bias": (n + ".b", WeightSpec((hidden_size,), init=(0.0, 0.02)))}
+
+    def load(self, tensors):
+        self.weight = self._vector32(tensors["weight"])
+        self.bias = self._vector32(tensors["bias"])
+        self.eps = float(self.params["eps"])
+
+    def prologue_params(self):
+        """(weight, bias, eps): a promise that ``forward`` is exactly this layer norm."""
+        return self.weight, self.bias, self.eps
+
+    def forward(self, h, delta=None, rows=None, write_h=True):
+        R = h.shape[0] if rows is None else rows.numel()
+        out = torch.empty((R, h.shape[1]), dtype=self.dtype, device=h.device)
+        ops.add_layernorm(h, delta, self.weight, self.bias, out, self.eps, rows=rows,
+                          write_h=write_h and rows is None and delta is not None)
+        return out
+
+    def weight_bytes(self):
+        return 8 * self.weight.numel()
 
 
 @register_part("norm", "dynamic_tanh")
