@@ -21,7 +21,8 @@ fraction for each); ``prefill_b8`` and ``prefill_b64`` are steps over 8 and 64 p
 ``--dtype float32`` measures the true 32-bit path.
 Every weight plus the cache exceed the L2 cache, so no flush is needed between steps.
 
-    python bench.py --design rigozen|losorax|virorax|mipurax|gibipel [--design-size s|m] [--layers L]
+    python bench.py --design rigozen|losorax|virorax|mipurax|gibipel|pudorax [--design-size s|m]
+                    [--layers L]
 
 measures another thing and leaves the line above as it is: prefill (1 and 8 prompts of 2,048
 tokens) and decode (batch 1, 8, 64 from a context of 2,048) of Rigozen models whose layers
@@ -40,8 +41,11 @@ a mixture in which every fourth layer reads an earlier layer's keys and values) 
 with a window as long as the chunk, Rigozen's latent attention and Losorax's routed experts.
 ``--design gibipel`` does it for Gibipel models (attention with pooled blocks beside a matrix memory
 in every layer, without and with its routed feed-forward) beside Virorax's attention and retention
-layers, whose sizes its two mixers have, and Losorax's routed experts; ``--models NAME,...`` measures
-only the named ones of any of these lists.
+layers, whose sizes its two mixers have, and Losorax's routed experts.  ``--design pudorax`` does it for
+Pudorax models (all layers attention, all layers mamba2, and a mixture whose second half runs twice,
+each with routed experts and a shared one and a token side) beside Losorax's routed attention,
+Virorax's retention, as many channels and as long a state as its mamba2, and Gibipel.
+``--models NAME,...`` measures only the named ones of any of these lists.
 """
 from __future__ import annotations
 
@@ -325,10 +329,10 @@ def run_e2e(engine, batch, steps, prompt_len):
 DESIGN_SIZES = {
     "s": dict(width=576, ff=1536, vocab=49152, heads=9, kv=3, dim=64, rank=128,
               d_heads=9, d_dim=64, d_vdim=64, window=1024,
-              experts=8, top=2, expert_ff=384, decay_rank=32),
+              experts=8, top=2, expert_ff=384, decay_rank=32, ssm_groups=3),
     "m": dict(width=2048, ff=8192, vocab=49152, heads=32, kv=8, dim=64, rank=128,
               d_heads=16, d_dim=128, d_vdim=128, window=1024,
-              experts=32, top=4, expert_ff=1024, decay_rank=64),
+              experts=32, top=4, expert_ff=1024, decay_rank=64, ssm_groups=4),
 }
 
 
@@ -482,6 +486,41 @@ def gibipel_configs(z, layers):
     }
 
 
+def pudorax_configs(z, layers):
+    """name -> config.json of the models --design pudorax measures: the attention has Losorax's sizes,
+    mamba2 as many channels as Virorax's retention and its head size as the state's, the experts are
+    Losorax's with a shared one of the same width."""
+    inner, vdim = z["d_heads"] * z["d_vdim"], 64
+    heads = inner // vdim
+    att = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"],
+           "scale": z["dim"] ** -0.5, "conv": 4, "rot": {"base": 250000.0, "dims": z["dim"] // 2}}
+    ssm = {"heads": heads, "vdim": vdim, "state": z["d_dim"], "groups": z["ssm_groups"],
+           "norm_groups": z["ssm_groups"], "conv": 4}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"], "limit": 7.0},
+           "router": {"experts": z["experts"], "top": z["top"]},
+           "shared": {"ff": z["expert_ff"], "limit": 7.0}}
+    mixers = {"attention": att, "mamba2": ssm}
+
+    def pudorax(order, loop=None):
+        cfg = {"architecture": "Pudorax", "vocab": z["vocab"], "width": z["width"],
+               "norm": {"eps": 1e-5}, "max_positions": CONTEXT, "embedding": {"scale": 3.0},
+               "logit_softcap": 30.0, "token_side": {"dim": 128},
+               "layers": [{"type": k, "mixer": mixers[k], "mlp": moe} for k in order]}
+        if loop is not None:
+            cfg["loop"] = loop
+        return cfg
+    mixed = (["mamba2", "mamba2", "mamba2", "attention"] * layers)[:layers]
+    gib = gibipel_configs(z, layers)
+    return {
+        "losorax attention routed": gib["losorax attention routed"],
+        "virorax retention": gib["virorax retention"],
+        "gibipel routed": gib["gibipel routed"],
+        "pudorax attention": pudorax(["attention"] * layers),
+        "pudorax mamba2": pudorax(["mamba2"] * layers),
+        "pudorax mixed looped": pudorax(mixed, {"start": layers // 2, "stop": layers, "times": 2}),
+    }
+
+
 def design_configs(z, layers):
     """name -> config.json of the models --design measures."""
     att = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"],
@@ -532,6 +571,7 @@ def design_bench(args) -> int:
                else virorax_configs(z, layers) if args.design == "virorax"
                else mipurax_configs(z, layers) if args.design == "mipurax"
                else gibipel_configs(z, layers) if args.design == "gibipel"
+               else pudorax_configs(z, layers) if args.design == "pudorax"
                else design_configs(z, layers))
     if args.models:
         wanted = [n.strip() for n in args.models.split(",")]
@@ -555,19 +595,22 @@ def design_bench(args) -> int:
                 else T
             kinds = ([l["type"] for l in cfg["layers"]] if "layers" in cfg
                      else ["llama"] * layers)
-            if cfg.get("architecture") == "Virorax":
+            if cfg.get("architecture") in ("Virorax", "Pudorax"):
                 # a span of layers may run several times: products and what is kept count per
                 # run, the tensors once
                 runs = [e.layer for e in engine.spec.schedule]
-                kinds = [cfg["layers"][i]["type"] for i in runs]
+                run_layers = [cfg["layers"][i] for i in runs]
+                kinds = [l["type"] for l in run_layers]
                 per_layer = [sum(p.weight_bytes() for br in l.branches for p in br.parts())
                              / (2 if args.dtype == "bfloat16" else 4)
                              for l in engine.model.layers]
-                params_run = params + sum(per_layer[i] for i in runs) - sum(per_layer)
+                params += sum(per_layer[i] for i in runs) - sum(per_layer)
+                passes = sum(e.merge_input for e in engine.spec.schedule)
+                params += 2 * W * W * max(0, passes - 1)
             else:
-                params_run = None
+                run_layers = cfg.get("layers", [])
             # routed experts: a token multiplies by `top` of them, a step reads those it uses
-            routed = [l["mlp"] for l in cfg.get("layers", [])
+            routed = [l["mlp"] for l in run_layers
                       if (l.get("mlp") or {}).get("kind") == "moe"]
             # (an expert is three matrices with a gate, two without)
             mats = 2 if cfg.get("architecture") == "Mipurax" else 3
@@ -580,8 +623,6 @@ def design_bench(args) -> int:
             active_params = params - expert_params + sum(
                 mats * W * m["expert"]["ff"] * m["router"]["top"] * used(m["router"])
                 for m in routed)
-            if params_run is not None:
-                active_params = params_run
 
             def read_params(b):
                 return params - expert_params + sum(
@@ -590,8 +631,9 @@ def design_bench(args) -> int:
                     for m in routed)
             # the embedding table is read a row at a time; an output matrix of its own is
             # multiplied on the last rows only
-            untied = cfg.get("architecture") in ("Losorax", "Gibipel")
-            tables = V * W * (2 if untied else 1)
+            untied = cfg.get("architecture") in ("Losorax", "Gibipel", "Pudorax")
+            side = V * (cfg.get("token_side") or {}).get("dim", 0) * len(run_layers)
+            tables = V * W * (2 if untied else 1) + side
             attn_flops = kept = 0.0
             for i, k in enumerate(kinds):
                 if k == "parallel":
@@ -617,6 +659,10 @@ def design_bench(args) -> int:
                 elif k == "general_delta":
                     attn_flops += T * z["d_heads"] * 8 * z["d_dim"] * z["d_dim"]
                     kept += 2 * 4 * z["d_heads"] * z["d_dim"] * z["d_dim"]
+                elif k == "mamba2":
+                    m = run_layers[i]["mixer"]
+                    attn_flops += T * m["heads"] * 4 * m["state"] * m["vdim"]
+                    kept += 2 * 4 * m["heads"] * m["state"] * m["vdim"]
                 elif k == "retention":          # two multiply-adds a state element and token
                     attn_flops += T * z["d_heads"] * 4 * z["d_dim"] * z["d_vdim"]
                     kept += 2 * 4 * z["d_heads"] * z["d_dim"] * z["d_vdim"]
@@ -641,7 +687,7 @@ def design_bench(args) -> int:
                                              seed=b)
                 rec[f"decode_b{b}_ms"] = ms
                 rec[f"decode_b{b}_tok_s"] = b / (ms * 1e-3)
-                rbytes = (read_params(b) - (V * W if untied else 0)) \
+                rbytes = (read_params(b) - (V * W if untied else 0) - side) \
                     * (2 if args.dtype == "bfloat16" else 4)
                 rec[f"decode_b{b}_frac_hbm"] = ((rbytes + b * kept) / (ms * 1e-3) / 1e9
                                                 / pk["hbm_gbs"])
@@ -751,7 +797,7 @@ def main() -> int:
     ap.add_argument("--unequal", action="store_true",
                     help="prompts of unequal lengths 256..2,048 instead of 2,048 each")
     ap.add_argument("--design", default=None,
-                    choices=["rigozen", "losorax", "virorax", "mipurax", "gibipel"],
+                    choices=["rigozen", "losorax", "virorax", "mipurax", "gibipel", "pudorax"],
                     help="measure this design at real layer sizes beside Llama at the same "
                          "sizes instead of the headline (another JSON line)")
     ap.add_argument("--models", default=None,
