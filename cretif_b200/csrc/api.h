@@ -475,7 +475,7 @@ int cretif_matrix_memory(const float* proj, int ldp, const float* bias_i, const 
 // The Mamba-2 recurrence (state_space.cu): proj rows (float32) [z (H e) | x (H e) | B (G N) | C (G N) |
 // dt (H) | ...] -> out [T, H e], the gated and normed read-outs.  conv_w [taps, C'], conv_b [C'],
 // C' = H e + 2 G N.  A slot's state: S [H, N, e] and, at inputs_at, the last taps - 1 inputs of every
-// convolved channel.  Scratch: y [T, H e]; for chunks xbc [T, ldx >= C'], dts [H, T], sums [H, T]
+// convolved channel.  Scratch: y [T, H e], xbc [T, ldx >= C'], dts [H, T]; for chunks sums [H, T]
 // (float64).  parts: equal parts of the H e channels that are normed on their own.  save_inputs: a step
 // of one token a sequence, whose inputs are saved here.  form: 0 chooses, 1 token by token, 2 chunks.
 int cretif_state_space(const float* proj, int ldp, const float* conv_w, const float* conv_b, int taps,

@@ -69,6 +69,13 @@ __device__ __forceinline__ float gate_mul_bf16_path(float g, float u, const Gate
   }
   return silu_bf16_path(g) * u;
 }
+// ... for kernels that are compiled for a clamped gate: the exponential's two factors are one
+__device__ __forceinline__ float gate_clamped_bf16_path(float g, float u, const GateRule& r) {
+  gate_clamp(g, u, r);
+  float e;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(g * (-1.4426950408889634f * r.slope)));
+  return __fdividef(g, 1.0f + e) * u;
+}
 inline bool gate_rule_ok(float limit) { return limit >= 0.f; }
 
 __device__ __forceinline__ float warp_sum(float v) {

@@ -73,11 +73,12 @@ struct TcSmem {
 //   kTcStore  store as bfloat16 / float32, or add into a float32 matrix;
 //   kTcSilu   the stacked gate|up product whose weight rows are interleaved in blocks of 64
 //             (64 gate rows, then the 64 up rows that belong to them): a 128-wide tile holds
-//             matching gate and up columns, and act = silu(gate) * up, or what another GateRule
-//             makes of the two, is stored (BN = 128);
+//             matching gate and up columns, and act = silu(gate) * up is stored (BN = 128);
+//   kTcGate   the same with a clamped gate (GateRule) instead of SiLU;
 //   kTcRope   the stacked q|k|v product with one head per tile (BN = head_dim): rotary on q and
 //             k, q to the query buffer, k and v into the block cache at the token's position.
-enum TcEpilogue : int { kTcStore = 0, kTcSilu = 1, kTcRope = 2, kTcStoreEx = 3 };
+enum TcEpilogue : int { kTcStore = 0, kTcSilu = 1, kTcRope = 2, kTcStoreEx = 3, kTcGate = 4 };
+__host__ __device__ constexpr bool tc_is_gated(int epi) { return epi == kTcSilu || epi == kTcGate; }
 // kTcStoreEx is kTcStore with a factor on the product and an optional activation: a kind of its
 // own, so that the plain store's code and registers stay what they were.
 __host__ __device__ constexpr bool tc_is_store(int epi) {
@@ -110,6 +111,11 @@ struct TcEpi {
   GateRule gate;                                           // silu
 };
 
+template <int EPI>
+__device__ __forceinline__ float tc_gate(float g, float u, const GateRule& rule) {
+  return EPI == kTcGate ? gate_clamped_bf16_path(g, u, rule) : silu_bf16_path(g) * u;
+}
+
 __device__ __forceinline__ float round_bf16(float x) {
   return __bfloat162float(__float2bfloat16_rn(x));
 }
@@ -138,7 +144,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
       (reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   using L = TcSmem<BN>;
   constexpr bool kBulk = tc_is_store(EPI) && sizeof(TC) == 4;
-  constexpr bool kBulkSilu = EPI == kTcSilu && EW == 8 && BN == 256;
+  constexpr bool kBulkSilu = tc_is_gated(EPI) && EW == 8 && BN == 256;
   constexpr int kSlabs = kBulk ? EW / 2 : (kBulkSilu ? 2 : 0);     // two a group of four warps
   unsigned char* staging = smem + kTcStages * L::kStage;
   uint64_t* full = reinterpret_cast<uint64_t*>(staging + (kSlabs && ep.bulk ? kSlabs * L::kSlab : 0));
@@ -454,8 +460,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
               const float g1 = round_bf16(__uint_as_float(g[j + e + 1]));
               const float u0 = round_bf16(__uint_as_float(u[j + e]));
               const float u1 = round_bf16(__uint_as_float(u[j + e + 1]));
-              __nv_bfloat162 h2 = __floats2bfloat162_rn(gate_mul_bf16_path(g0, u0, ep.gate),
-                                                        gate_mul_bf16_path(g1, u1, ep.gate));
+              __nv_bfloat162 h2 = __floats2bfloat162_rn(tc_gate<EPI>(g0, u0, ep.gate),
+                                                        tc_gate<EPI>(g1, u1, ep.gate));
               w4[e >> 1] = *reinterpret_cast<uint32_t*>(&h2);
             }
             const int piece = chalf * 4 + (j >> 3);
@@ -469,7 +475,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
             tc::bulk_commit_group();
           }
         }
-      } else if (ok && EPI == kTcSilu) {
+      } else if (ok && tc_is_gated(EPI)) {
         // every 128 tile columns are 64 gate columns and the 64 up columns that belong to
         // them: act[:, n0/2 + 64 pair ..]
 #pragma unroll 1
@@ -491,7 +497,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                   // gate and up pass through bfloat16 as they do when stored separately
                   const float gg = round_bf16(__uint_as_float(g[j + e]));
                   const float uu = round_bf16(__uint_as_float(u[j + e]));
-                  v[e] = gate_mul_bf16_path(gg, uu, ep.gate);
+                  v[e] = tc_gate<EPI>(gg, uu, ep.gate);
                 }
                 if (col0 + c0 + j + 8 <= ep.I) store8(out + j, v);
               }
@@ -809,8 +815,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
               const float g1 = round_bf16(__uint_as_float(g[j + e + 1]));
               const float u0 = round_bf16(__uint_as_float(u[j + e]));
               const float u1 = round_bf16(__uint_as_float(u[j + e + 1]));
-              __nv_bfloat162 h2 = __floats2bfloat162_rn(gate_mul_bf16_path(g0, u0, ep.gate),
-                                                        gate_mul_bf16_path(g1, u1, ep.gate));
+              __nv_bfloat162 h2 = __floats2bfloat162_rn(tc_gate<EPI>(g0, u0, ep.gate),
+                                                        tc_gate<EPI>(g1, u1, ep.gate));
               w4[e >> 1] = *reinterpret_cast<uint32_t*>(&h2);
             }
             const int piece = chalf * 4 + (j >> 3);
@@ -1082,7 +1088,7 @@ static int launch_tc(const void* A, const void* W, const TcEpi& ep_in, int M, in
     smem = TcSmem<BN>::total(stages, epi_warps / 2);
     count_variant(kVarTcBulkAdd);
   }
-  if (EPI == kTcSilu && epi_warps == 8 && BN == 256 && g_tc_bulk_add &&
+  if (tc_is_gated(EPI) && epi_warps == 8 && BN == 256 && g_tc_bulk_add &&
       make_box_map(&map_c, ep.act, M, ep.I, ep.I, kTcBM, 64, true, false) == 0) {
     ep.bulk = 1;
     stages = TcSmem<BN>::stages_with_staging(stages, 2);
@@ -1214,14 +1220,16 @@ extern "C" int cretif_gemm_tc_silu(const void* A, const void* Wgu, void* act, in
   // wide tiles (two gate|up pairs, one CTA per SM) once there are four waves of them for the
   // whole chip; with fewer, the last wave's empty seats cost more than the wide tile saves
   const long long wide_tiles = (long long)((2 * I + 255) / 256) * ((M + kTcBM - 1) / kTcBM);
-  if (g_tc_pair != 0 && g_tc_bulk_add && (2 * I) % 256 == 0 &&
-      (g_tc_pair > 0 || (wide_tiles >= 4 * 148 && pair_pays(2 * I, K))))
-    return launch_tc_pair<256, kTcSilu>(A, Wgu, ep, M, 2 * I, K, lda, ldw, fault, (cudaStream_t)stream);
-  if (wide_tiles >= 4 * 148)
-    return launch_tc<256, kTcSilu, __nv_bfloat16>(A, Wgu, ep, M, 2 * I, K, lda, ldw, fault,
-                                                  (cudaStream_t)stream);
-  return launch_tc<128, kTcSilu, __nv_bfloat16>(A, Wgu, ep, M, 2 * I, K, lda, ldw, fault,
-                                                (cudaStream_t)stream);
+  cudaStream_t st = (cudaStream_t)stream;
+  const bool pair = g_tc_pair != 0 && g_tc_bulk_add && (2 * I) % 256 == 0 &&
+                    (g_tc_pair > 0 || (wide_tiles >= 4 * 148 && pair_pays(2 * I, K)));
+#define CRETIF_TC_GATED(EPI)                                                                       \
+  (pair ? launch_tc_pair<256, EPI>(A, Wgu, ep, M, 2 * I, K, lda, ldw, fault, st)                   \
+        : wide_tiles >= 4 * 148                                                                    \
+              ? launch_tc<256, EPI, __nv_bfloat16>(A, Wgu, ep, M, 2 * I, K, lda, ldw, fault, st)   \
+              : launch_tc<128, EPI, __nv_bfloat16>(A, Wgu, ep, M, 2 * I, K, lda, ldw, fault, st))
+  return limit > 0.f ? CRETIF_TC_GATED(kTcGate) : CRETIF_TC_GATED(kTcSilu);
+#undef CRETIF_TC_GATED
 }
 
 // Grouped products: A [M, K] with M a multiple of 128 whose row tiles belong to groups
@@ -1292,11 +1300,15 @@ extern "C" int cretif_gemm_tc_silu_grouped(const void* A, const void* Wgu, void*
   ep.gate = GateRule{limit, slope, offset};
   ep.tile_group = tile_group; ep.group_rows = 2 * I; ep.used_m_tiles = used_m_tiles;
   const long long wide_tiles = (long long)((2 * I + 255) / 256) * (M / kTcBM);
-  if (wide_tiles >= 4 * 148)
-    return launch_tc<256, kTcSilu, __nv_bfloat16>(A, Wgu, ep, M, 2 * I, K, lda, ldw, fault,
-                                                  (cudaStream_t)stream, groups * 2 * I);
-  return launch_tc<128, kTcSilu, __nv_bfloat16>(A, Wgu, ep, M, 2 * I, K, lda, ldw, fault,
-                                                (cudaStream_t)stream, groups * 2 * I);
+  cudaStream_t st = (cudaStream_t)stream;
+#define CRETIF_TC_GATED(EPI)                                                                       \
+  (wide_tiles >= 4 * 148                                                                           \
+       ? launch_tc<256, EPI, __nv_bfloat16>(A, Wgu, ep, M, 2 * I, K, lda, ldw, fault, st,          \
+                                            groups * 2 * I)                                        \
+       : launch_tc<128, EPI, __nv_bfloat16>(A, Wgu, ep, M, 2 * I, K, lda, ldw, fault, st,          \
+                                            groups * 2 * I))
+  return limit > 0.f ? CRETIF_TC_GATED(kTcGate) : CRETIF_TC_GATED(kTcSilu);
+#undef CRETIF_TC_GATED
 }
 
 // q|k|v = A·Wqkv^T with rotary on q and k; q to Q, k and v into the block cache.

@@ -819,18 +819,16 @@ def state_space(proj, conv_w, conv_b, a_log, dt_bias, d_skip, state, inputs_at: 
     chunks = form == "chunk" or (form == "auto" and T >= 16 * B)
     ldx = -(-C // 4) * 4
     y = torch.empty((T, inner), dtype=torch.float32, device=proj.device)
-    xbc = dts = sums = None
-    if chunks:
-        xbc = torch.empty((T, ldx), dtype=torch.float32, device=proj.device)
-        dts = torch.empty(H * T, dtype=torch.float32, device=proj.device)
-        sums = torch.empty(H * T, dtype=torch.float64, device=proj.device)
+    xbc = torch.empty((T, ldx), dtype=torch.float32, device=proj.device)
+    dts = torch.empty(H * T, dtype=torch.float32, device=proj.device)
+    sums = torch.empty(H * T, dtype=torch.float64, device=proj.device) if chunks else None
     _check(lib().cretif_state_space(
         _p(proj), _rows(proj, "proj"), _p(conv_w), _p(conv_b), taps, _p(a_log), _p(dt_bias),
         _p(d_skip), _p(state), ctypes.c_longlong(state.stride(0)), ctypes.c_longlong(inputs_at),
         _p(cu_seqlens), _p(seq_slot), _p(tok_seq), B, H, G, N, e, _p(y), _p(xbc), ldx, _p(dts),
         _p(sums), parts, _p(norm_w), ctypes.c_float(eps), _p(out), _dt(out), _rows(out, "out"),
         int(write_state), int(save_inputs), T, {"auto": 0, "token": 1, "chunk": 2}[form], _stream()),
-        "state_space", kernels=4 if chunks else 2)
+        "state_space", kernels=4 if chunks else 3)
 
 
 def heads_out_norm(o_raw, gate, norm_w, eps: float, out, H: int, e: int,

@@ -10,12 +10,14 @@
 // per channel.  Everything is 32-bit; sums of a dt are carried in 64-bit, because what enters the
 // exponentials are differences of them.
 //
+// * ssm_prepare_kernel: the convolved channels and the step sizes.  A thread has a channel and eight
+//   tokens in turn, so that a projected row is read once, or (few tokens) a channel and one token.  In a
+//   step of one token a sequence it also brings the convolution's saved inputs up to date: each is read
+//   and replaced by one thread.  After any other step delta_conv_state (delta_rule.cu) does.
 // * ssm_token_kernel (a CTA per (sequence, head, slice of columns)): token by token, the thread layout
-//   of the retention's recurrence (retention.cu).  It convolves what it reads itself.
-// * ssm_prepare_kernel + ssm_intra_kernel + ssm_carry_kernel: 64 tokens at a time, below.
-// * ssm_out_kernel: the gate, the norms and the weight.  In a step of one token a sequence further
-//   CTAs of it bring the convolution's saved inputs up to date (every reader of the old ones has
-//   finished); after any other step delta_conv_state (delta_rule.cu) does.
+//   of the retention's recurrence (retention.cu).
+// * ssm_intra_kernel + ssm_carry_kernel: 64 tokens at a time, below.
+// * ssm_out_kernel: the gate, the norms and the weight.
 //
 // A slot's state: [S (H N e) | the last taps - 1 inputs of every convolved channel (C' (taps - 1))].
 #include "api.h"
@@ -48,9 +50,9 @@ struct SsmArgs {
   const int* tok_seq;
   int B, H, G, N, e, T;
   float* y;                 // [T, H e]
-  float* xbc;               // chunks: [T, ldx] the convolved channels
+  float* xbc;               // [T, ldx] the convolved channels
   int ldx;
-  float* dts;               // chunks: [H, T] step sizes
+  float* dts;               // [H, T] step sizes
   double* sums;             // chunks: [H, T] sums of a dt from the chunk's start
   int write_state;
   __device__ int inner() const { return H * e; }
@@ -63,19 +65,97 @@ struct SsmArgs {
   __device__ float* S(int b, int h) const {
     return state + (size_t)slot[b] * stride + (size_t)h * N * e;
   }
-  __device__ const float* saved(int b) const { return state + (size_t)slot[b] * stride + inputs; }
-  // channel c of token t (lt tokens after the first of its sequence in the step), convolved
-  __device__ float conv(int t, int lt, const float* st, int c) const {
-    const int keep = taps - 1, C = channels();
-    float acc = conv_b[c];
-    for (int j = 0; j <= keep; ++j) {
-      const int back = keep - j;
-      const float v = back <= lt ? u(t - back)[c] : st[(size_t)c * keep + keep - (back - lt)];
-      acc = fmaf(conv_w[(size_t)j * C + c], v, acc);
-    }
-    return ssm_silu(acc);
+  // a sequence's last taps - 1 inputs of channel c, the oldest first
+  __device__ float* saved(int b, int c) const {
+    return state + (size_t)slot[b] * stride + inputs + (size_t)c * (taps - 1);
   }
 };
+
+constexpr int kSpTokens = 8;
+
+// TAPS: the number of taps when it is 2, 3 or 4, 0 for any number.  NT: tokens a thread.
+template <int TAPS, int NT>
+__global__ void __launch_bounds__(256)
+ssm_prepare_kernel(const SsmArgs a, int save) {
+  const int C = a.channels();
+  const int c = blockIdx.y * 256 + threadIdx.x;
+  const int first = blockIdx.x * NT, last = min(first + NT, a.T);
+  if (c >= C) {                         // behind the channels: the heads' step sizes
+    const int h = c - C;
+    if (h < a.H)
+      for (int t = first; t < last; ++t) a.dts[(size_t)h * a.T + t] = a.step(t, h);
+    return;
+  }
+  if (TAPS == 0) {
+    const int keep = a.taps - 1;
+    for (int t = first; t < last; ++t) {
+      const int b = a.tok_seq[t], lt = t - a.cu[b];
+      float* st = a.saved(b, c);
+      float acc = a.conv_b[c];
+      for (int j = 0; j <= keep; ++j) {
+        const int back = keep - j;
+        const float v = back <= lt ? a.u(t - back)[c] : st[keep - (back - lt)];
+        acc = fmaf(a.conv_w[(size_t)j * C + c], v, acc);
+      }
+      a.xbc[(size_t)t * a.ldx + c] = ssm_silu(acc);
+      if (save && keep) {
+        for (int j = 0; j + 1 < keep; ++j) st[j] = st[j + 1];
+        st[keep - 1] = a.u(t)[c];
+      }
+    }
+    return;
+  }
+  constexpr int K = TAPS > 1 ? TAPS - 1 : 1;
+  float w[TAPS > 0 ? TAPS : 1], back[K];          // back[k]: the input k + 1 tokens before
+  float in[NT];
+#pragma unroll
+  for (int i = 0; i < NT; ++i) in[i] = first + i < last ? a.u(first + i)[c] : 0.f;
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) w[j] = a.conv_w[(size_t)j * C + c];
+  const float bias = a.conv_b[c];
+#pragma unroll
+  for (int i = 0; i < NT; ++i) {
+    const int t = first + i;
+    if (t >= last) break;
+    const int b = a.tok_seq[t], lt = t - a.cu[b];
+    if (i == 0 || lt == 0) {
+      const float* st = a.saved(b, c);
+#pragma unroll
+      for (int k = 0; k < K; ++k) back[k] = k + 1 <= lt ? a.u(t - k - 1)[c] : st[K - (k + 1 - lt)];
+    }
+    float acc = bias;
+#pragma unroll
+    for (int k = K; k >= 1; --k) acc = fmaf(w[TAPS > 0 ? TAPS - 1 - k : 0], back[k - 1], acc);
+    acc = fmaf(w[TAPS > 0 ? TAPS - 1 : 0], in[i], acc);
+    a.xbc[(size_t)t * a.ldx + c] = ssm_silu(acc);
+#pragma unroll
+    for (int k = K - 1; k > 0; --k) back[k] = back[k - 1];
+    back[0] = in[i];
+    if (save) {
+      float* st = a.saved(b, c);
+#pragma unroll
+      for (int k = 0; k < K; ++k) st[K - 1 - k] = back[k];
+    }
+  }
+}
+
+int launch_ssm_prepare(const SsmArgs& a, int save, cudaStream_t st) {
+  const bool few = a.T <= 256;
+  const int tokens = few ? 1 : kSpTokens;
+  const dim3 grid((a.T + tokens - 1) / tokens, (a.H * a.e + 2 * a.G * a.N + a.H + 255) / 256);
+  if (grid.y > 65535) return kBadArgument;
+#define CRETIF_SSM_PREP(TAPS)                                                        \
+  do {                                                                               \
+    if (few) ssm_prepare_kernel<TAPS, 1><<<grid, 256, 0, st>>>(a, save);             \
+    else ssm_prepare_kernel<TAPS, kSpTokens><<<grid, 256, 0, st>>>(a, save);         \
+  } while (0)
+  if (a.taps == 4) CRETIF_SSM_PREP(4);
+  else if (a.taps == 3) CRETIF_SSM_PREP(3);
+  else if (a.taps == 2) CRETIF_SSM_PREP(2);
+  else CRETIF_SSM_PREP(0);
+#undef CRETIF_SSM_PREP
+  return launch_status();
+}
 
 constexpr int kSsmChunk = 16;
 
@@ -99,7 +179,6 @@ ssm_token_kernel(const SsmArgs a, int P, int ecols) {
   float* sk = so + kSsmChunk * ecols;            // [chunk] decay
   float* sd = sk + kSsmChunk;                    // [chunk] step size
   float* M = a.S(b, h);
-  const float* st = a.saved(b);
   float S[R];
 #pragma unroll
   for (int r = 0; r < R; ++r) {
@@ -110,21 +189,22 @@ ssm_token_kernel(const SsmArgs a, int P, int ecols) {
   const int grp = h / (a.H / a.G);
   const int cb = a.inner() + grp * N, cc = cb + a.G * N, cx = h * e;
   const float rate = a.rate(h), skip = a.d_skip[h];
+  auto value = [&](int t, int c) { return a.xbc[(size_t)t * a.ldx + c]; };
   for (int c0 = t0; c0 < t1; c0 += kSsmChunk) {
     const int nt = min(kSsmChunk, t1 - c0);
+    const float dt = threadIdx.x < nt ? a.dts[(size_t)h * a.T + c0 + threadIdx.x] : 0.f;
     __syncthreads();                             // the chunk before has been read and written out
     for (int idx = threadIdx.x; idx < nt * rows_padded; idx += blockDim.x) {
       const int tt = idx / rows_padded, i = idx - tt * rows_padded;
       const int p = i / R, r = i - p * R, t = c0 + tt;
-      sc[(tt * P + p) * slice + r] = i < N ? a.conv(t, t - t0, st, cc + i) : 0.f;
-      sb[(tt * P + p) * slice + r] = i < N ? a.conv(t, t - t0, st, cb + i) : 0.f;
+      sc[(tt * P + p) * slice + r] = i < N ? value(t, cc + i) : 0.f;
+      sb[(tt * P + p) * slice + r] = i < N ? value(t, cb + i) : 0.f;
     }
     for (int idx = threadIdx.x; idx < nt * ecols; idx += blockDim.x) {
       const int tt = idx / ecols, j = idx - tt * ecols, t = c0 + tt;
-      sx[idx] = col0 + j < e ? a.conv(t, t - t0, st, cx + col0 + j) : 0.f;
+      sx[idx] = col0 + j < e ? value(t, cx + col0 + j) : 0.f;
     }
     if (threadIdx.x < nt) {
-      const float dt = a.step(c0 + threadIdx.x, h);
       sd[threadIdx.x] = dt;
       sk[threadIdx.x] = expf(rate * dt);
     }
@@ -197,8 +277,6 @@ int launch_ssm_token(const SsmArgs& a, int P, int ecols, cudaStream_t st) {
 //     S_n = exp(F_n) S0 + sum_s exp(F_n - F_s) dt_s B_s x_s^T
 // and no exponent is ever above zero.
 //
-// * ssm_prepare_kernel: the convolved channels (a thread a channel, eight tokens in turn, so that a
-//   projected row is read once) and the step sizes.
 // * ssm_intra_kernel (a CTA per (chunk, few heads of one group); the chunks of all sequences at once):
 //   the second and third term to y, the sums F to memory.  The scores C . B are computed once for the
 //   CTA's heads.  Nothing here depends on the state, so a long prompt fills the chip.
@@ -231,6 +309,12 @@ __device__ __forceinline__ void ssm_cp16(float* dst, const float* src) {
   const unsigned a = (unsigned)__cvta_generic_to_shared(dst);
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(src) : "memory");
 }
+template <typename T>
+__device__ __forceinline__ void ssm_cp_one(T* dst, const T* src) {      // 4 or 8 bytes
+  const unsigned a = (unsigned)__cvta_generic_to_shared(dst);
+  asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(a), "l"(src), "n"(sizeof(T))
+               : "memory");
+}
 __device__ __forceinline__ void ssm_cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N>
 __device__ __forceinline__ void ssm_cp_wait() {
@@ -252,60 +336,23 @@ inline size_t ssm_intra_smem(int n) {
   return sizeof(double) * kScHeads * kScTokens + sizeof(float) * (kScHeads * kScTokens +
                                                                   ssm_intra_floats(n));
 }
+// (the 64-bit sums come first, so that they are 8-byte aligned)
 inline size_t ssm_carry_smem(int n, int ec, int nbuf) {
-  return sizeof(float) * (nbuf * (2 * (size_t)kScTokens * ssm_chunk_ld(n) + (size_t)kScTokens * ec) +
-                          (size_t)n * ec + 2 * kScTokens);
+  return nbuf * kScTokens * (sizeof(double) + sizeof(float)) +
+         sizeof(float) * (nbuf * (2 * (size_t)kScTokens * ssm_chunk_ld(n) + (size_t)kScTokens * ec) +
+                          (size_t)n * ec);
 }
-
-constexpr int kSpTokens = 8;
-
-template <int TAPS>
-__global__ void __launch_bounds__(256)
-ssm_prepare_kernel(const SsmArgs a) {
-  const int C = a.channels();
-  const int c = blockIdx.y * 256 + threadIdx.x;
-  const int first = blockIdx.x * kSpTokens, last = min(first + kSpTokens, a.T);
-  if (c >= C) {                         // behind the channels: the heads' step sizes
-    const int h = c - C;
-    if (h < a.H)
-      for (int t = first; t < last; ++t) a.dts[(size_t)h * a.T + t] = a.step(t, h);
-    return;
+// The pieces tid, tid + kScThreads, ... of a [rows][n4] block without a division a piece.
+struct SsmWalk {
+  int row, col, n4, dr, dc;
+  __device__ SsmWalk(int tid, int n4_)
+      : row(tid / n4_), col(tid % n4_), n4(n4_), dr(kScThreads / n4_), dc(kScThreads % n4_) {}
+  __device__ void next() {
+    row += dr;
+    col += dc;
+    if (col >= n4) { col -= n4; ++row; }
   }
-  if (TAPS == 0) {
-    for (int t = first; t < last; ++t) {
-      const int b = a.tok_seq[t];
-      a.xbc[(size_t)t * a.ldx + c] = a.conv(t, t - a.cu[b], a.saved(b), c);
-    }
-    return;
-  }
-  constexpr int K = TAPS > 1 ? TAPS - 1 : 1;
-  float w[TAPS > 0 ? TAPS : 1], back[K];          // back[k]: the input k + 1 tokens before
-#pragma unroll
-  for (int j = 0; j < TAPS; ++j) w[j] = a.conv_w[(size_t)j * C + c];
-  const float bias = a.conv_b[c];
-  float in[kSpTokens];
-#pragma unroll
-  for (int i = 0; i < kSpTokens; ++i) in[i] = first + i < last ? a.u(first + i)[c] : 0.f;
-#pragma unroll
-  for (int i = 0; i < kSpTokens; ++i) {
-    const int t = first + i;
-    if (t >= last) break;
-    const int b = a.tok_seq[t], lt = t - a.cu[b];
-    if (i == 0 || lt == 0) {
-      const float* st = a.saved(b) + (size_t)c * K;
-#pragma unroll
-      for (int k = 0; k < K; ++k) back[k] = k + 1 <= lt ? a.u(t - k - 1)[c] : st[K - (k + 1 - lt)];
-    }
-    float acc = bias;
-#pragma unroll
-    for (int k = K; k >= 1; --k) acc = fmaf(w[TAPS > 0 ? TAPS - 1 - k : 0], back[k - 1], acc);
-    acc = fmaf(w[TAPS > 0 ? TAPS - 1 : 0], in[i], acc);
-    a.xbc[(size_t)t * a.ldx + c] = ssm_silu(acc);
-#pragma unroll
-    for (int k = K - 1; k > 0; --k) back[k] = back[k - 1];
-    back[0] = in[i];
-  }
-}
+};
 
 __global__ void __launch_bounds__(kScThreads)
 ssm_intra_kernel(const SsmArgs a, int heads) {
@@ -341,11 +388,10 @@ ssm_intra_kernel(const SsmArgs a, int heads) {
   const int cb = a.inner() + grp * N, cc = cb + a.G * N;
   // Rows beyond the chunk's last token stay as they are: they reach only scores of rows that are
   // not stored, or of keys after the row, which are set to zero.
-  for (int idx = tid; idx < nt * n4; idx += kScThreads) {
-    const int tt = idx / n4, i4 = idx - tt * n4;
-    const float* row = a.xbc + (size_t)(c0 + tt) * a.ldx + 4 * i4;
-    ssm_cp16(sC + tt * ldq + 4 * i4, row + cc);
-    ssm_cp16(sB + tt * ldq + 4 * i4, row + cb);
+  for (SsmWalk w(tid, n4); w.row < nt; w.next()) {
+    const float* row = a.xbc + (size_t)(c0 + w.row) * a.ldx + 4 * w.col;
+    ssm_cp16(sC + w.row * ldq + 4 * w.col, row + cc);
+    ssm_cp16(sB + w.row * ldq + 4 * w.col, row + cb);
   }
   ssm_cp_commit();
   for (int hh = tid >> 5; hh < heads; hh += kScThreads / 32) {
@@ -484,9 +530,10 @@ ssm_carry_kernel(const SsmArgs a, int nbuf) {
   const int ldq = ssm_chunk_ld(N);
   const int n4 = N >> 2;
   const int buf_floats = 2 * C * ldq + C * EC;   // C [C][ldq] | B [C][ldq] | x [C][EC]
-  float* sS = smem + nbuf * buf_floats;          // [N][EC]
-  float* sR = sS + N * EC;                       // [C] what the state before the chunk weighs at a token
-  float* sW = sR + C;                            // [C] a token's weight in the state's update
+  double* sums = reinterpret_cast<double*>(smem);           // [nbuf][C] F
+  float* steps = reinterpret_cast<float*>(sums + nbuf * C); // [nbuf][C] dt
+  float* bufs = steps + nbuf * C;
+  float* sS = bufs + nbuf * buf_floats;          // [N][EC]
   const int grp = h / (H / a.G);
   const int cb = a.inner() + grp * N, cc = cb + a.G * N, cx = h * e + col0;
   float* M = a.S(b, h) + col0;
@@ -501,13 +548,18 @@ ssm_carry_kernel(const SsmArgs a, int nbuf) {
   const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
   // Rows beyond a chunk's last token are not copied: of C they reach only read-outs that are not
   // stored, of B and x nothing (the update stops at the last token).
-  auto stage = [&](int c0, float* buf) {
+  auto stage = [&](int c0, int which) {
     const int nt = min(C, t1 - c0);
-    for (int idx = tid; idx < nt * n4; idx += kScThreads) {
-      const int tt = idx / n4, i4 = idx - tt * n4;
-      const float* row = a.xbc + (size_t)(c0 + tt) * a.ldx + 4 * i4;
-      ssm_cp16(buf + tt * ldq + 4 * i4, row + cc);
-      ssm_cp16(buf + C * ldq + tt * ldq + 4 * i4, row + cb);
+    float* buf = bufs + which * buf_floats;
+    for (SsmWalk w(tid, n4); w.row < nt; w.next()) {
+      const float* row = a.xbc + (size_t)(c0 + w.row) * a.ldx + 4 * w.col;
+      float* to = buf + w.row * ldq + 4 * w.col;
+      ssm_cp16(to, row + cc);
+      ssm_cp16(to + C * ldq, row + cb);
+    }
+    if (tid < nt) {
+      ssm_cp_one(sums + which * C + tid, F + c0 + tid);
+      ssm_cp_one(steps + which * C + tid, dts + c0 + tid);
     }
     for (int idx = tid; idx < nt * CG; idx += kScThreads) {
       const int tt = idx / CG, jg = idx - tt * CG;
@@ -516,23 +568,21 @@ ssm_carry_kernel(const SsmArgs a, int nbuf) {
     }
     ssm_cp_commit();
   };
-  stage(t0, smem);
+  stage(t0, 0);
   int turn = 0;
   for (int c0 = t0; c0 < t1; c0 += C, ++turn) {
     const int nt = min(C, t1 - c0);
     const bool last = c0 + C >= t1;
-    float* sC = smem + (nbuf == 2 ? (turn & 1) * buf_floats : 0);
+    const int which = nbuf == 2 ? (turn & 1) : 0;
+    float* sC = bufs + which * buf_floats;
     float* sB = sC + C * ldq;
     float* sX = sB + C * ldq;
-    const double Fn = F[c0 + nt - 1];
-    if (tid < nt) {                        // (read by others after the barrier below; by nobody still)
-      const double Ft = F[c0 + tid];
-      sR[tid] = expf((float)Ft);
-      sW[tid] = expf((float)(Fn - Ft)) * dts[c0 + tid];
-    }
+    const double* sF = sums + which * C;
+    const float* sD = steps + which * C;
     ssm_cp_wait<0>();
     __syncthreads();                       // the chunk is in place; the chunk before is done
-    if (nbuf == 2 && !last) stage(c0 + C, smem + ((turn + 1) & 1) * buf_floats);
+    if (nbuf == 2 && !last) stage(c0 + C, which ^ 1);
+    const double Fn = sF[nt - 1];
     const float keep = expf((float)Fn);
     {
       // what the state before the chunk gives every row: rows tr + NR r, columns 4 tj .. + 3
@@ -545,7 +595,7 @@ ssm_carry_kernel(const SsmArgs a, int nbuf) {
                               a.y + (size_t)(c0 + t) * a.inner() + cx + 4 * tj))
                         : zero4;
       }
-#pragma unroll 2
+#pragma unroll (RT == 1 ? 4 : 2)
       for (int i = 0; i < N; i += 4) {
         const float4 s0 = *reinterpret_cast<const float4*>(sS + (i + 0) * EC + 4 * tj);
         const float4 s1 = *reinterpret_cast<const float4*>(sS + (i + 1) * EC + 4 * tj);
@@ -565,7 +615,7 @@ ssm_carry_kernel(const SsmArgs a, int nbuf) {
         const int t = tr + NR * r;
         if (t < nt) {
           float4 o = old[r];
-          fma4(o, sR[t], acc[r]);
+          fma4(o, expf((float)sF[t]), acc[r]);
           *reinterpret_cast<float4*>(a.y + (size_t)(c0 + t) * a.inner() + cx + 4 * tj) = o;
         }
       }
@@ -575,11 +625,29 @@ ssm_carry_kernel(const SsmArgs a, int nbuf) {
     for (int idx = tid; idx < nt * CG; idx += kScThreads) {
       const int tt = idx / CG, jg = idx - tt * CG;
       float4 v4 = *reinterpret_cast<float4*>(sX + tt * EC + 4 * jg);
-      scale4(v4, sW[tt]);
+      scale4(v4, expf((float)(Fn - sF[tt])) * sD[tt]);
       *reinterpret_cast<float4*>(sX + tt * EC + 4 * jg) = v4;
     }
     __syncthreads();                       // everybody has read the old state; x is weighted
-    for (int ig = tr; ig < n4; ig += NR) {
+    // (few rows for many threads: two rows a thread, so that all have some)
+    if (n4 < NR) {
+      for (int ig = tr; ig < 2 * n4; ig += NR) {
+        float* srow = sS + (2 * ig) * EC + 4 * tj;
+        float4 a0 = *reinterpret_cast<float4*>(srow);
+        float4 a1 = *reinterpret_cast<float4*>(srow + EC);
+        scale4(a0, keep);
+        scale4(a1, keep);
+#pragma unroll 8
+        for (int s = 0; s < nt; ++s) {
+          const float2 k2 = *reinterpret_cast<const float2*>(sB + s * ldq + 2 * ig);
+          const float4 v4 = *reinterpret_cast<const float4*>(sX + s * EC + 4 * tj);
+          fma4(a0, k2.x, v4);
+          fma4(a1, k2.y, v4);
+        }
+        *reinterpret_cast<float4*>(srow) = a0;
+        *reinterpret_cast<float4*>(srow + EC) = a1;
+      }
+    } else for (int ig = tr; ig < n4; ig += NR) {
       float* srow = sS + (4 * ig) * EC + 4 * tj;
       float4 a0 = *reinterpret_cast<float4*>(srow);
       float4 a1 = *reinterpret_cast<float4*>(srow + EC);
@@ -605,7 +673,7 @@ ssm_carry_kernel(const SsmArgs a, int nbuf) {
     }
     if (nbuf != 2 && !last) {
       __syncthreads();                     // the one buffer has been read
-      stage(c0 + C, smem);
+      stage(c0 + C, 0);
     }
   }
   if (a.write_state) {
@@ -653,23 +721,12 @@ int launch_ssm_intra(const SsmArgs& a, int sm_count, cudaStream_t st) {
 
 // out[t, part] = v / sqrt(mean(v^2) + eps) * w,  v = y silu(z) over the part's channels.  NT threads a
 // (token, part): 32 or 256; VEC: four channels at a time, 16 NT of them kept in registers between the
-// sum and the store, what lies beyond is computed again.  Blocks from `norm_blocks` on: the saved inputs of the convolution of a
-// step of one token a sequence, a thread a (sequence, channel).
+// sum and the store, what lies beyond is computed again.
 template <int NT, bool VEC, typename TO>
 __global__ void __launch_bounds__(256)
 ssm_out_kernel(const SsmArgs a, int parts, const float* __restrict__ norm_w, float eps,
-               TO* __restrict__ out, int ldo, long long items, unsigned norm_blocks) {
+               TO* __restrict__ out, int ldo, long long items) {
   __shared__ float scratch[33];
-  if (blockIdx.x >= norm_blocks) {
-    const long long idx = (long long)(blockIdx.x - norm_blocks) * 256 + threadIdx.x;
-    const int C = a.channels(), keep = a.taps - 1;
-    const int b = (int)(idx / C), c = (int)(idx - (long long)b * C);
-    if (b >= a.B) return;
-    float* s = a.state + (size_t)a.slot[b] * a.stride + a.inputs + (size_t)c * keep;
-    for (int j = 0; j + 1 < keep; ++j) s[j] = s[j + 1];
-    s[keep - 1] = a.u(a.cu[b])[c];
-    return;
-  }
   const long long item = (long long)blockIdx.x * (256 / NT) + threadIdx.x / NT;
   const int tid = threadIdx.x % NT;
   if (item >= items) return;             // (whole warps; with a CTA an item there is none beyond)
@@ -735,23 +792,21 @@ inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 
 
 template <typename TO>
 int launch_ssm_out(const SsmArgs& a, int parts, const float* norm_w, float eps, TO* out, int ldo,
-                   int save_inputs, cudaStream_t st) {
+                   cudaStream_t st) {
   const int inner = a.H * a.e, n = inner / parts;
   const bool vec = n % 4 == 0 && a.ldp % 4 == 0 && ldo % 4 == 0 && inner % 4 == 0 && aligned16(a.y) &&
                    aligned16(a.proj) && aligned16(norm_w) && aligned16(out);
   const long long items = (long long)a.T * parts;
-  const bool warps = n <= 512 || (n <= 1024 && items >= 1024);
+  const bool warps = n <= 1024 && items >= 1024;
   const long long blocks = warps ? (items + 7) / 8 : items;
-  const int C = inner + 2 * a.G * a.N;
-  const long long more = save_inputs && a.taps > 1 ? ((long long)a.B * C + 255) / 256 : 0;
-  if (blocks + more > 0x7fffffffLL) return kBadArgument;
-  const unsigned grid = (unsigned)(blocks + more), nb = (unsigned)blocks;
+  if (blocks > 0x7fffffffLL) return kBadArgument;
+  const unsigned grid = (unsigned)blocks;
   if (warps) {
-    if (vec) ssm_out_kernel<32, true, TO><<<grid, 256, 0, st>>>(a, parts, norm_w, eps, out, ldo, items, nb);
-    else ssm_out_kernel<32, false, TO><<<grid, 256, 0, st>>>(a, parts, norm_w, eps, out, ldo, items, nb);
+    if (vec) ssm_out_kernel<32, true, TO><<<grid, 256, 0, st>>>(a, parts, norm_w, eps, out, ldo, items);
+    else ssm_out_kernel<32, false, TO><<<grid, 256, 0, st>>>(a, parts, norm_w, eps, out, ldo, items);
   } else {
-    if (vec) ssm_out_kernel<256, true, TO><<<grid, 256, 0, st>>>(a, parts, norm_w, eps, out, ldo, items, nb);
-    else ssm_out_kernel<256, false, TO><<<grid, 256, 0, st>>>(a, parts, norm_w, eps, out, ldo, items, nb);
+    if (vec) ssm_out_kernel<256, true, TO><<<grid, 256, 0, st>>>(a, parts, norm_w, eps, out, ldo, items);
+    else ssm_out_kernel<256, false, TO><<<grid, 256, 0, st>>>(a, parts, norm_w, eps, out, ldo, items);
   }
   return launch_status();
 }
@@ -761,8 +816,7 @@ int launch_ssm_out(const SsmArgs& a, int parts, const float* norm_w, float eps, 
 using namespace cretif;
 
 // form 0 chooses, 1 token by token, 2 chunks (refused where the sizes or addresses rule out 16-byte
-// accesses).  xbc [T, ldx], dts [H, T] and sums (float64) [H, T]: scratch of the chunks, may be null
-// with form 1.  save_inputs: the step brings one token a sequence and the saved inputs are brought up to
+// accesses).  Scratch: y [T, H e], xbc [T, ldx] and dts [H, T]; sums (float64) [H, T] for the chunks.  save_inputs: the step brings one token a sequence and the saved inputs are brought up to
 // date here.
 extern "C" int cretif_state_space(const float* proj, int ldp, const float* conv_w, const float* conv_b,
                                   int taps, const float* a_log, const float* dt_bias,
@@ -774,12 +828,13 @@ extern "C" int cretif_state_space(const float* proj, int ldp, const float* conv_
                                   int write_state, int save_inputs, int T, int form, void* stream) {
   if (B <= 0 || T <= 0) return kOk;
   if (H <= 0 || G <= 0 || H % G || N <= 0 || e <= 0 || taps < 1 || parts <= 0 || (H * e) % parts ||
-      !proj || !conv_w || !conv_b || !a_log || !dt_bias || !d_skip || !state || !norm_w || !y ||
+      !proj || !conv_w || !conv_b || !a_log || !dt_bias || !d_skip || !state || !norm_w || !y || !xbc || !dts ||
       form < 0 || form > 2)
     return kBadArgument;
   const int inner = H * e, C = inner + 2 * G * N;
   if (ldp < inner + C + H || ldo < inner || inputs_at < (long long)H * N * e ||
-      state_stride < inputs_at + (long long)C * (taps - 1) || (save_inputs && T != B))
+      state_stride < inputs_at + (long long)C * (taps - 1) || ldx < C ||
+      (save_inputs && T != B))
     return kBadArgument;
   static int sm_count = 0;
   if (!sm_count) {
@@ -792,31 +847,28 @@ extern "C" int cretif_state_space(const float* proj, int ldp, const float* conv_
   const SsmArgs a{proj, ldp, conv_w, conv_b, taps, a_log, dt_bias, d_skip, state, (size_t)state_stride,
                   (size_t)inputs_at, cu_seqlens, seq_slot, tok_seq, B, H, G, N, e, T, y, xbc, ldx, dts,
                   sums, write_state};
-  int rc = kBadArgument;
+  int rc = launch_ssm_prepare(a, save_inputs && taps > 1, st);
+  if (rc != kOk) return rc;
   bool done = false;
   // 64 tokens at a time where the step brings a sequence 16 tokens or more on average and the
   // sizes allow 16-byte accesses throughout; token by token otherwise.
   if (form == 2 || (form == 0 && (long long)T >= 16LL * B)) {
-    const bool fits = N % 4 == 0 && e % 16 == 0 && state_stride % 4 == 0 && xbc && dts && sums &&
-                      ldx >= C && ldx % 4 == 0 && aligned16(xbc) && aligned16(state) && aligned16(y) &&
+    const bool fits = N % 4 == 0 && e % 16 == 0 && state_stride % 4 == 0 && sums && ldx % 4 == 0 && aligned16(xbc) && aligned16(state) && aligned16(y) &&
                       H <= 65535 && ssm_carry_smem(N, 16, 1) <= 220 * 1024 &&
                       ssm_intra_smem(N) <= 220 * 1024;
     if (fits) {
-      const dim3 grid((T + kSpTokens - 1) / kSpTokens, (C + H + 255) / 256);
-      if (grid.y > 65535) return kBadArgument;
-      if (taps == 4) ssm_prepare_kernel<4><<<grid, 256, 0, st>>>(a);
-      else if (taps == 3) ssm_prepare_kernel<3><<<grid, 256, 0, st>>>(a);
-      else if (taps == 2) ssm_prepare_kernel<2><<<grid, 256, 0, st>>>(a);
-      else ssm_prepare_kernel<0><<<grid, 256, 0, st>>>(a);
-      rc = launch_status();
-      if (rc != kOk) return rc;
       rc = launch_ssm_intra(a, sm_count, st);
       if (rc != kOk) return rc;
-      // columns a CTA: as many as divide e and fit, fewer while the chip is not filled
-      int ec = e % 64 == 0 ? 64 : e % 32 == 0 ? 32 : 16;
-      while (ec > 16 && (ssm_carry_smem(N, ec, 1) > 220 * 1024 ||
-                         (long long)B * H * (e / ec) < (long long)sm_count))
-        ec /= 2;
+      // columns a CTA: a chunk takes about 40 + columns units of time, a wave of CTAs (one an SM) a
+      // chunk after the other (measured with N = 128: 205, 250 and 390 us for 2,048 tokens at 16, 32
+      // and 64 columns)
+      int ec = 16;
+      double best = 0.0;
+      for (int n = 16; n <= 64 && e % n == 0 && ssm_carry_smem(N, n, 1) <= 220 * 1024; n *= 2) {
+        const double waves = (double)B * H * (e / n) / sm_count;
+        const double cost = (waves > 1.0 ? waves : 1.0) * (40 + n);
+        if (n == 16 || cost < best) { best = cost; ec = n; }
+      }
       rc = ec == 64   ? launch_ssm_carry<64>(a, st)
            : ec == 32 ? launch_ssm_carry<32>(a, st)
                       : launch_ssm_carry<16>(a, st);
@@ -847,8 +899,8 @@ extern "C" int cretif_state_space(const float* proj, int ldp, const float* conv_
     if (rc != kOk) return rc;
   }
   if (out_dt == kF32)
-    return launch_ssm_out(a, parts, norm_w, eps, (float*)out, ldo, save_inputs, st);
+    return launch_ssm_out(a, parts, norm_w, eps, (float*)out, ldo, st);
   if (out_dt == kBF16)
-    return launch_ssm_out(a, parts, norm_w, eps, (__nv_bfloat16*)out, ldo, save_inputs, st);
+    return launch_ssm_out(a, parts, norm_w, eps, (__nv_bfloat16*)out, ldo, st);
   return kBadDType;
 }
