@@ -27,7 +27,8 @@ namespace cretif {
 
 namespace {
 
-__device__ __forceinline__ float ssm_silu(float z) { return z / (1.0f + expf(-z)); }
+// (the quotient by an approximate reciprocal: two units in the last place of 32 bits)
+__device__ __forceinline__ float ssm_silu(float z) { return __fdividef(z, 1.0f + expf(-z)); }
 __device__ __forceinline__ float ssm_softplus(float z) {
   return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
 }
@@ -73,7 +74,8 @@ struct SsmArgs {
 
 constexpr int kSpTokens = 8;
 
-// TAPS: the number of taps when it is 2, 3 or 4, 0 for any number.  NT: tokens a thread.
+// TAPS: the number of taps when it is 2, 3 or 4, 0 for any number.  NT: tokens a thread (one where
+// the inputs are saved).
 template <int TAPS, int NT>
 __global__ void __launch_bounds__(256)
 ssm_prepare_kernel(const SsmArgs a, int save) {
@@ -113,15 +115,18 @@ ssm_prepare_kernel(const SsmArgs a, int save) {
 #pragma unroll
   for (int j = 0; j < TAPS; ++j) w[j] = a.conv_w[(size_t)j * C + c];
   const float bias = a.conv_b[c];
+  const bool one = a.tok_seq[first] == a.tok_seq[last - 1];       // all of one sequence
 #pragma unroll
   for (int i = 0; i < NT; ++i) {
     const int t = first + i;
     if (t >= last) break;
-    const int b = a.tok_seq[t], lt = t - a.cu[b];
-    if (i == 0 || lt == 0) {
-      const float* st = a.saved(b, c);
+    if (i == 0 || !one) {
+      const int b = a.tok_seq[t], lt = t - a.cu[b];
+      if (i == 0 || lt == 0) {
+        const float* st = a.saved(b, c);
 #pragma unroll
-      for (int k = 0; k < K; ++k) back[k] = k + 1 <= lt ? a.u(t - k - 1)[c] : st[K - (k + 1 - lt)];
+        for (int k = 0; k < K; ++k) back[k] = k + 1 <= lt ? a.u(t - k - 1)[c] : st[K - (k + 1 - lt)];
+      }
     }
     float acc = bias;
 #pragma unroll
@@ -131,8 +136,8 @@ ssm_prepare_kernel(const SsmArgs a, int save) {
 #pragma unroll
     for (int k = K - 1; k > 0; --k) back[k] = back[k - 1];
     back[0] = in[i];
-    if (save) {
-      float* st = a.saved(b, c);
+    if (NT == 1 && save) {
+      float* st = a.saved(a.tok_seq[t], c);
 #pragma unroll
       for (int k = 0; k < K; ++k) st[K - 1 - k] = back[k];
     }
@@ -140,7 +145,7 @@ ssm_prepare_kernel(const SsmArgs a, int save) {
 }
 
 int launch_ssm_prepare(const SsmArgs& a, int save, cudaStream_t st) {
-  const bool few = a.T <= 256;
+  const bool few = a.T <= 256 || save;
   const int tokens = few ? 1 : kSpTokens;
   const dim3 grid((a.T + tokens - 1) / tokens, (a.H * a.e + 2 * a.G * a.N + a.H + 255) / 256);
   if (grid.y > 65535) return kBadArgument;
